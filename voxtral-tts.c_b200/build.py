@@ -17,7 +17,7 @@ LIBDIR = os.path.join(HERE, "lib")
 LIB = os.path.join(LIBDIR, "libvoxtral_b200.so")
 OBJDIR = os.path.join(LIBDIR, "obj")
 
-CU_SOURCES = ["vb_engine.cu", "vb_simple.cu", "vb_model.cu", "vb_prefill.cu", "vb_abi.cu", "vb_noalloc.cu",
+CU_SOURCES = ["vb_upload.cu", "vb_engine.cu", "vb_simple.cu", "vb_model.cu", "vb_prefill.cu", "vb_abi.cu", "vb_noalloc.cu",
               "vb_tc.cu", "vb_acoustic_tc.cu", "vb_batch.cu", "vb_stream.cu", "vb_codec.cu"]
 CPP_SOURCES = ["vb_synth.cpp"]
 NVCC = os.environ.get("NVCC", "nvcc")

@@ -8,6 +8,7 @@
 #include "vb_model.cuh"
 #include "vb_simple.cuh"
 #include "vb_tc.cuh"
+#include "vb_upload.cuh"
 
 #include <math.h>
 #include <stddef.h>
@@ -16,7 +17,6 @@
 #include <string.h>
 
 #include <chrono>
-#include <thread>
 #include <vector>
 
 namespace vb {
@@ -191,91 +191,10 @@ static void drop(T **p) {
     if (*p) { dev_release(*p); *p = nullptr; }
 }
 
-/* Host -> device copies of the weights go through a small ring of pinned staging buffers:
- * a few host threads fill buffer n + 1 from the caller's (pageable, usually memory-mapped:
- * voxtral_tts_safetensors.c:400-405) memory while the copy engine drains buffer n, and the
- * repacking kernels run behind the copies on the same stream. Nothing waits for the device
- * except a buffer that is still being drained; the upload call synchronises once at its end.
- * The reference copies every matrix with a blocking cudaMemcpy (voxtral_tts_cuda.cu:223-310). */
-struct Stager {
-    static const int kBufs = 3;
-    size_t cap = (size_t)64 << 20;
-    void *pin[kBufs] = {};
-    cudaEvent_t drained[kBufs] = {};
-    bool busy[kBufs] = {};
-    int next = 0, threads = 4;
-    bool ok = false;
-};
+/* Host -> device copies of the weights go through the pinned staging ring (vb_upload.cuh). */
 static Stager g_stage;
 
-static void stage_open() {
-    Stager &s = g_stage;
-    if (s.ok) return;
-    const char *env = getenv("VB200_UPLOAD_THREADS");
-    unsigned hc = std::thread::hardware_concurrency();
-    s.threads = env ? atoi(env) : (hc >= 4 ? 4 : 1);   /* four saturate the host's copy bandwidth where measured */
-    if (s.threads < 1) s.threads = 1;
-    if (s.threads > 32) s.threads = 32;
-    for (int i = 0; i < Stager::kBufs; i++) {
-        if (cudaHostAlloc(&s.pin[i], s.cap, cudaHostAllocDefault) != cudaSuccess ||
-            cudaEventCreateWithFlags(&s.drained[i], cudaEventDisableTiming) != cudaSuccess) {
-            cudaGetLastError();
-            return;   /* no pinned memory: stage_copy() falls back to plain copies */
-        }
-        s.busy[i] = false;
-    }
-    s.ok = true;
-}
-
-static void stage_close() {
-    Stager &s = g_stage;
-    for (int i = 0; i < Stager::kBufs; i++) {
-        if (s.pin[i]) cudaFreeHost(s.pin[i]);
-        if (s.drained[i]) cudaEventDestroy(s.drained[i]);
-        s.pin[i] = nullptr; s.drained[i] = nullptr; s.busy[i] = false;
-    }
-    s.ok = false;
-}
-
-static void fill_parallel(char *dst, const char *src, size_t n, int threads) {
-    const size_t min_part = (size_t)4 << 20;
-    int parts = (int)((n + min_part - 1) / min_part);
-    if (parts > threads) parts = threads;
-    if (parts <= 1) { memcpy(dst, src, n); return; }
-    const size_t per = ((n / parts) + 4095) & ~(size_t)4095;
-    std::vector<std::thread> pool;
-    for (int i = 1; i < parts; i++) {
-        const size_t off = per * i;
-        if (off >= n) break;
-        const size_t len = off + per < n ? per : n - off;
-        pool.emplace_back([=] { memcpy(dst + off, src + off, len); });
-    }
-    memcpy(dst, src, per < n ? per : n);
-    for (auto &t : pool) t.join();
-}
-
-/* Asynchronous on m.st as far as the device goes; the source may be reused on return. */
-static int stage_copy(void *dst, const void *src, size_t bytes) {
-    Model &m = g_model;
-    Stager &s = g_stage;
-    m.upload_bytes += (double)bytes;
-    if (!s.ok) {
-        VB_CHECK(cudaMemcpyAsync(dst, src, bytes, cudaMemcpyHostToDevice, m.st));
-        VB_CHECK(cudaStreamSynchronize(m.st));
-        return 0;
-    }
-    for (size_t off = 0; off < bytes; off += s.cap) {
-        const size_t n = bytes - off < s.cap ? bytes - off : s.cap;
-        const int b = s.next;
-        s.next = (s.next + 1) % Stager::kBufs;
-        if (s.busy[b]) VB_CHECK(cudaEventSynchronize(s.drained[b]));
-        fill_parallel((char *)s.pin[b], (const char *)src + off, n, s.threads);
-        VB_CHECK(cudaMemcpyAsync((char *)dst + off, s.pin[b], n, cudaMemcpyHostToDevice, m.st));
-        VB_CHECK(cudaEventRecord(s.drained[b], m.st));
-        s.busy[b] = true;
-    }
-    return 0;
-}
+static int stage_copy(void *dst, const void *src, size_t bytes) { return g_stage.copy(dst, src, bytes, g_model.st); }
 
 static int upload_bf16(uint16_t **dst, const uint16_t *src, size_t n) {
     if (!src) return -1;
@@ -319,10 +238,12 @@ static int upload_layer(LayerDev &L, const vb200_layer_weights_t &w, uint16_t *t
  * once, releases the ring and adds the call's wall-clock time to the model's upload record. */
 struct UploadScope {
     std::chrono::steady_clock::time_point t0;
-    UploadScope() : t0(std::chrono::steady_clock::now()) { stage_open(); }
+    UploadScope() : t0(std::chrono::steady_clock::now()) { g_stage.open(); }
     int finish(int rc) {
         if (cudaStreamSynchronize(g_model.st) != cudaSuccess) rc = -1;
-        stage_close();
+        g_stage.close();
+        g_model.upload_bytes += g_stage.bytes_copied;
+        g_stage.bytes_copied = 0.0;
         g_model.upload_seconds += std::chrono::duration<double>(std::chrono::steady_clock::now() - t0).count();
         return rc;
     }

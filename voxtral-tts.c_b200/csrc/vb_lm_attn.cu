@@ -1,0 +1,527 @@
+/*
+ * vb_lm_attn.cu - decoder language models: softmax attention over a ring cache. Query and key
+ * norm over the whole projection, rotary positions on a part of the head, optional softcap,
+ * optional sliding window with kept first tokens; any head sizes, separate key and value sizes.
+ *
+ *   lm_attn_prepare  one row per CTA: sums the projection's split-K partials, norms and rotates q
+ *                    and k, appends k and v to the cache
+ *   lm_attn_generic  fp32 pipes: decode (keys split over CTAs, last arrival merges) and the 32-bit mode
+ *   lm_attn_mma      prompts: mma.sync on hi + lo BF16 halves of q, k, v and the weights
+ *
+ * Keys are visited in two stretches, the kept first tokens and the window; a stretch that is out
+ * of reach of all of a CTA's rows is never loaded.
+ */
+#include "vb_lm_kernels.cuh"
+#include "vb_tc.cuh"
+
+namespace vb {
+
+namespace {
+
+inline int ok(cudaError_t e) { return e == cudaSuccess ? 0 : -1; }
+
+/* ------------------------------------------------------------------ q, k, v of a row */
+constexpr int kPrepThreads = 512;
+
+__global__ void __launch_bounds__(kPrepThreads) lm_attn_prepare_kernel(const LmAttn a) {
+    extern __shared__ float prep_smem[];
+    __shared__ float red[2][kPrepThreads / 32];
+    const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim;
+    float *buf = prep_smem;                       /* [nq + nk] */
+    float *cs = buf + nq + nk;                    /* [rot / 2] cos, then [rot / 2] sin */
+    pdl_launch_dependents();
+    pdl_wait();
+    const int m = blockIdx.x, tid = threadIdx.x, half = a.rot / 2;
+    const int pos = a.dyn->pos + m;
+    const size_t row = (size_t)lm_ring_row(a.ring, pos);
+    for (int i = tid; i < half; i += kPrepThreads) {
+        /* the angle pos * f to twice fp32's precision: sine and cosine of its leading part, and the
+         * remainder as a first-order correction */
+        const float p = (float)pos, f = a.freq[i];
+        const float hi = p * f, lo = fmaf(p, f, -hi) + p * a.freq[half + i];
+        float s, c;
+        sincosf(hi, &s, &c);
+        cs[i] = (c - s * lo) * a.mag;
+        cs[half + i] = (s + c * lo) * a.mag;
+    }
+    float sq = 0.0f, sk = 0.0f;
+    for (int c = tid; c < nq + nk; c += kPrepThreads) {
+        const float v = lm_sum(a.qkv, m, c);
+        buf[c] = v;
+        if (c < nq) sq += v * v; else sk += v * v;
+    }
+    float *Vr = lm_state(a.v, a.dyn) + row * nv;
+    for (int c = tid; c < nv; c += kPrepThreads) Vr[c] = lm_sum(a.qkv, m, nq + nk + c);
+    sq = vb_warp_sum(sq);
+    sk = vb_warp_sum(sk);
+    if ((tid & 31) == 0) { red[0][tid >> 5] = sq; red[1][tid >> 5] = sk; }
+    __syncthreads();
+    sq = sk = 0.0f;
+#pragma unroll
+    for (int w = 0; w < kPrepThreads / 32; w++) { sq += red[0][w]; sk += red[1][w]; }
+    const float rq = 1.0f / sqrtf(sq / (float)nq + a.eps), rk = 1.0f / sqrtf(sk / (float)nk + a.eps);
+    float *Kr = lm_state(a.k, a.dyn) + row * nk, *Q = a.q + (size_t)m * nq;
+    for (int c = tid; c < nq + nk; c += kPrepThreads) {
+        const bool isq = c < nq;
+        const int j = isq ? c : c - nq, d = j % a.dim;
+        const float *gain = isq ? a.q_gain : a.k_gain;
+        const float r = isq ? rq : rk;
+        float v = buf[c] * r * __ldg(gain + j);
+        if (d < a.rot) {
+            const int i = d < half ? d : d - half, other = d < half ? half : -half;
+            const float u = buf[c + other] * r * __ldg(gain + j + other);
+            v = d < half ? v * cs[i] - u * cs[half + i] : v * cs[i] + u * cs[half + i];
+        }
+        (isq ? Q : Kr)[j] = v;
+    }
+}
+
+/* ------------------------------------------------------------------ which keys */
+/* Keys that rows at positions [imin, imax] may see: [0, a_end) and [b0, b_end), in tiles of KT. */
+struct KeyTiles {
+    int a_end, b0, b_end, a_tiles, n_tiles;
+};
+template <int KT>
+VB_DEVINL KeyTiles key_tiles(int imin, int imax, int window, int keep) {
+    KeyTiles t;
+    t.b_end = imax + 1;
+    if (window <= 0) { t.a_end = 0; t.b0 = 0; }
+    else {
+        t.a_end = keep < t.b_end ? keep : t.b_end;
+        t.b0 = imin - window + 1 > t.a_end ? imin - window + 1 : t.a_end;
+    }
+    t.a_tiles = (t.a_end + KT - 1) / KT;
+    t.n_tiles = t.a_tiles + (t.b_end > t.b0 ? (t.b_end - t.b0 + KT - 1) / KT : 0);
+    return t;
+}
+/* First key of tile t and how many keys it has. */
+template <int KT>
+VB_DEVINL void key_tile(const KeyTiles &k, int t, int *j0, int *n) {
+    const bool first = t < k.a_tiles;
+    const int s = first ? t * KT : k.b0 + (t - k.a_tiles) * KT, e = first ? k.a_end : k.b_end;
+    *j0 = s;
+    *n = e - s < KT ? e - s : KT;
+}
+VB_DEVINL bool key_seen(int i, int j, int window, int keep) {
+    return j <= i && (window <= 0 || i - j < window || j < keep);
+}
+
+/* ------------------------------------------------------------------ generic kernel */
+constexpr int kGaThreads = 256, kGaKeys = 32, kGaPairs = kLmAttnPairs;
+
+inline size_t ga_smem(int dim, int vdim) {
+    return sizeof(float) * ((size_t)kGaPairs * dim + (size_t)kGaKeys * (dim + 1) + (size_t)kGaKeys * vdim +
+                            (size_t)kGaPairs * vdim + kGaPairs * (kGaKeys + 1) + 4 * kGaPairs + kLmAttnSplits * kGaPairs);
+}
+
+/* grid = (tiles of 16 (row, head) pairs, KV heads, key splits) */
+__global__ void __launch_bounds__(kGaThreads) lm_attn_generic_kernel(const LmAttn a, int M) {
+    extern __shared__ float ga[];
+    __shared__ int last_flag;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int dim = a.dim, vdim = a.vdim, group = a.heads / a.kv_heads;
+    float *Q = ga, *K = Q + kGaPairs * dim, *V = K + kGaKeys * (dim + 1), *O = V + kGaKeys * vdim;
+    float *S = O + kGaPairs * vdim, *mx = S + kGaPairs * (kGaKeys + 1), *den = mx + kGaPairs, *cor = den + kGaPairs,
+          *wgt = cor + 2 * kGaPairs;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int g = blockIdx.y, p0 = blockIdx.x * kGaPairs;
+    const int np = M * group - p0 < kGaPairs ? M * group - p0 : kGaPairs;
+    const int pos0 = a.dyn->pos;
+    const KeyTiles kt = key_tiles<kGaKeys>(pos0 + p0 / group, pos0 + (p0 + np - 1) / group, a.window, a.keep);
+    const int S_eff = (int)gridDim.z < kt.n_tiles ? (int)gridDim.z : kt.n_tiles;
+    const int sp = blockIdx.z;
+    if (sp >= S_eff) return;
+    const int t0 = (int)((long long)kt.n_tiles * sp / S_eff), t1 = (int)((long long)kt.n_tiles * (sp + 1) / S_eff);
+    const float *Kc = lm_state(a.k, a.dyn), *Vc = lm_state(a.v, a.dyn);
+    const int ldk = a.kv_heads * dim, ldv = a.kv_heads * vdim;
+
+    for (int i = tid; i < np * dim; i += kGaThreads) {
+        const int p = p0 + i / dim, d = i % dim;
+        Q[i] = a.q[(size_t)(p / group) * a.heads * dim + (size_t)(g * group + p % group) * dim + d];
+    }
+    for (int i = tid; i < np * vdim; i += kGaThreads) O[i] = 0.0f;
+    if (tid < kGaPairs) { mx[tid] = -INFINITY; den[tid] = 0.0f; }
+
+    for (int t = t0; t < t1; t++) {
+        int j0, n;
+        key_tile<kGaKeys>(kt, t, &j0, &n);
+        __syncthreads();
+        for (int i = tid; i < n * dim; i += kGaThreads) {
+            const int j = i / dim, d = i % dim;
+            K[j * (dim + 1) + d] = __ldcg(Kc + (size_t)lm_ring_row(a.ring, j0 + j) * ldk + g * dim + d);
+        }
+        for (int i = tid; i < n * vdim; i += kGaThreads) {
+            const int j = i / vdim, d = i % vdim;
+            V[i] = __ldcg(Vc + (size_t)lm_ring_row(a.ring, j0 + j) * ldv + g * vdim + d);
+        }
+        __syncthreads();
+        for (int p = warp; p < np; p += kGaThreads / 32) {
+            const int i = pos0 + (p0 + p) / group;
+            float s = -INFINITY;
+            if (lane < n && key_seen(i, j0 + lane, a.window, a.keep)) {
+                const float *q = Q + p * dim, *k = K + lane * (dim + 1);
+                float e0 = 0.0f, e1 = 0.0f, e2 = 0.0f, e3 = 0.0f;
+                int d = 0;
+                for (; d + 3 < dim; d += 4) {
+                    e0 = fmaf(q[d], k[d], e0);
+                    e1 = fmaf(q[d + 1], k[d + 1], e1);
+                    e2 = fmaf(q[d + 2], k[d + 2], e2);
+                    e3 = fmaf(q[d + 3], k[d + 3], e3);
+                }
+                for (; d < dim; d++) e0 = fmaf(q[d], k[d], e0);
+                s = ((e0 + e1) + (e2 + e3)) * a.scale;
+                if (a.softcap > 0.0f) s = a.softcap * tanhf(s / a.softcap);
+            }
+            float top = s;
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
+            const float old = mx[p], now = fmaxf(old, top);
+            const float w = s > -INFINITY ? expf(s - now) : 0.0f;
+            const float sum = vb_warp_sum(w);
+            S[p * (kGaKeys + 1) + lane] = w;
+            __syncwarp();
+            if (lane == 0) {
+                const float c = old > -INFINITY ? expf(old - now) : 0.0f;
+                cor[p] = c;
+                mx[p] = now;
+                den[p] = den[p] * c + sum;
+            }
+        }
+        __syncthreads();
+        for (int i = tid; i < np * vdim; i += kGaThreads) {
+            const int p = i / vdim, d = i % vdim;
+            float o = O[i] * cor[p];
+            const float *w = S + p * (kGaKeys + 1);
+            for (int j = 0; j < n; j++) o = fmaf(w[j], V[j * vdim + d], o);
+            O[i] = o;
+        }
+    }
+    __syncthreads();
+
+    float *po = nullptr;
+    if (S_eff > 1) {
+        /* several CTAs share these pairs: publish the slice, the last arrival merges in slice order */
+        const int stride = vdim + 2;
+        const size_t tile = (size_t)blockIdx.y * gridDim.x + blockIdx.x;
+        po = a.scratch + tile * gridDim.z * kGaPairs * stride;
+        float *mine = po + (size_t)sp * kGaPairs * stride;
+        for (int i = tid; i < np * vdim; i += kGaThreads) mine[(i / vdim) * stride + i % vdim] = O[i];
+        if (tid < np) { mine[tid * stride + vdim] = mx[tid]; mine[tid * stride + vdim + 1] = den[tid]; }
+        __threadfence();
+        __syncthreads();
+        if (tid == 0) {
+            const unsigned t = atomicAdd(&a.tickets[tile], 1u);
+            last_flag = t == (unsigned)(S_eff - 1);
+            if (last_flag) a.tickets[tile] = 0u;
+        }
+        __syncthreads();
+        if (!last_flag) return;
+        __threadfence();
+        if (tid < np) {
+            float M0 = -INFINITY, L = 0.0f;
+            for (int u = 0; u < S_eff; u++) M0 = fmaxf(M0, __ldcg(po + ((size_t)u * kGaPairs + tid) * stride + vdim));
+            for (int u = 0; u < S_eff; u++) {
+                const float mu = __ldcg(po + ((size_t)u * kGaPairs + tid) * stride + vdim);
+                const float w = mu > -INFINITY ? expf(mu - M0) : 0.0f;
+                wgt[u * kGaPairs + tid] = w;
+                L += w * __ldcg(po + ((size_t)u * kGaPairs + tid) * stride + vdim + 1);
+            }
+            den[tid] = L;
+        }
+        __syncthreads();
+        for (int i = tid; i < np * vdim; i += kGaThreads) {
+            const int p = i / vdim, d = i % vdim;
+            float o = 0.0f;
+            for (int u = 0; u < S_eff; u++) o = fmaf(wgt[u * kGaPairs + p], __ldcg(po + ((size_t)u * kGaPairs + p) * stride + d), o);
+            O[i] = o;
+        }
+        __syncthreads();
+    }
+    for (int i = tid; i < np * vdim; i += kGaThreads) {
+        const int p = i / vdim, d = i % vdim, P = p0 + p;
+        lm_put(a.out, P / group, (g * group + P % group) * vdim + d, O[i] / den[p]);
+    }
+}
+
+/* ------------------------------------------------------------------ prompts on the warp-level tensor cores */
+VB_DEVINL void hilo(float v, uint32_t &hi, uint32_t &lo) {
+    const __nv_bfloat16 h = __float2bfloat16_rn(v);
+    hi = __bfloat16_as_ushort(h);
+    lo = __bfloat16_as_ushort(__float2bfloat16_rn(v - __bfloat162float(h)));
+}
+VB_DEVINL void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+VB_DEVINL void ldsm(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+VB_DEVINL void ldsm_t(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+/* Byte offset of the 16-byte chunk `chunk` of key row `key` in a [keys][16 * STEPS] BF16 tile; chunks are
+ * XOR-swizzled by the key so that eight rows of one chunk column hit eight different banks. */
+template <int STEPS>
+VB_DEVINL uint32_t tile_off(int key, int chunk) {
+    return (uint32_t)(key * STEPS * 32 + (((chunk & ~7) | ((chunk ^ key) & 7)) << 4));
+}
+
+constexpr int kMaThreads = 256, kMaWarps = 8, kMaKeys = 32;
+
+/* Stages 32 keys of one KV head: fp32 rows of the cache -> hi and lo BF16 tiles, zero beyond the
+ * keys and beyond the head's size. */
+template <int STEPS>
+VB_DEVINL void stage_tile(unsigned char *hi_t, unsigned char *lo_t, const float *cache, int ld, int col0, int size, int j0, int n,
+                          const LmRing &ring) {
+    constexpr int kQuads = STEPS * 4;                   /* groups of four values per row */
+    for (int i = threadIdx.x; i < kMaKeys * kQuads; i += kMaThreads) {
+        const int key = i / kQuads, f = i % kQuads;
+        float e[4] = {0.f, 0.f, 0.f, 0.f};
+        if (key < n && 4 * f < size) {
+            const float *src = cache + (size_t)lm_ring_row(ring, j0 + key) * ld + col0 + 4 * f;
+            if ((size & 3) == 0) {
+                const float4 v = __ldcg(reinterpret_cast<const float4 *>(src));
+                e[0] = v.x; e[1] = v.y; e[2] = v.z; e[3] = v.w;
+            } else {
+#pragma unroll
+                for (int u = 0; u < 4; u++)
+                    if (4 * f + u < size) e[u] = __ldcg(src + u);
+            }
+        }
+        uint32_t h[4], l[4];
+#pragma unroll
+        for (int u = 0; u < 4; u++) hilo(e[u], h[u], l[u]);
+        const uint32_t off = tile_off<STEPS>(key, f >> 1) + (uint32_t)(f & 1) * 8u;
+        *reinterpret_cast<uint2 *>(hi_t + off) = make_uint2(h[0] | (h[1] << 16), h[2] | (h[3] << 16));
+        *reinterpret_cast<uint2 *>(lo_t + off) = make_uint2(l[0] | (l[1] << 16), l[2] | (l[3] << 16));
+    }
+}
+
+/* A CTA serves one KV head; each of its eight warps owns 16 query rows of one query head of the
+ * group (consecutive (row block, head) tiles), so that the staged keys are shared by up to eight
+ * warps. Every product a.b is taken as a_hi.b_hi + a_hi.b_lo + a_lo.b_hi, accumulated in fp32;
+ * scores, softcap, weights and the running maximum are fp32. DK, DV: 16-wide steps of the key
+ * and value sizes (padded with zeros). */
+template <int DK, int DV>
+__global__ void __launch_bounds__(kMaThreads) lm_attn_mma_kernel(const LmAttn a, int M) {
+    extern __shared__ __align__(128) unsigned char ma_tiles[];
+    unsigned char *Kh = ma_tiles, *Kl = Kh + kMaKeys * DK * 32, *Vh = Kl + kMaKeys * DK * 32, *Vl = Vh + kMaKeys * DV * 32;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int group = a.heads / a.kv_heads, g = blockIdx.y;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3;
+    const int n_tiles_q = (M + 15) / 16 * group;
+    /* the latest rows see the most keys: they go first */
+    const int T0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * kMaWarps, T1 = T0 + kMaWarps < n_tiles_q ? T0 + kMaWarps : n_tiles_q;
+    const int T = T0 + warp;
+    const bool active = T < T1;
+    const int r0 = active ? T / group * 16 : 0, h = g * group + (active ? T % group : 0);
+    const int pos0 = a.dyn->pos;
+    const int rowA = r0 + gq, rowB = rowA + 8;
+    const bool validA = active && rowA < M, validB = active && rowB < M;
+    const int iA = pos0 + rowA, iB = pos0 + rowB;
+    const int last_row = T1 > T0 ? ((T1 - 1) / group * 16 + 15 < M - 1 ? (T1 - 1) / group * 16 + 15 : M - 1) : 0;
+    const KeyTiles kt = key_tiles<kMaKeys>(pos0 + T0 / group * 16, pos0 + last_row, a.window, a.keep);
+    const int w_imin = pos0 + r0, w_imax = pos0 + (r0 + 15 < M - 1 ? r0 + 15 : M - 1);
+    const float *Kc = lm_state(a.k, a.dyn), *Vc = lm_state(a.v, a.dyn);
+    const int ldk = a.kv_heads * a.dim, ldv = a.kv_heads * a.vdim;
+
+    /* Q as A fragments: (row A, k 2t..), (row B, k 2t..), (row A, k 8 + 2t..), (row B, k 8 + 2t..) */
+    uint32_t qh[DK][4], ql[DK][4];
+#pragma unroll
+    for (int ks = 0; ks < DK; ks++)
+#pragma unroll
+        for (int hf = 0; hf < 2; hf++)
+#pragma unroll
+            for (int rr = 0; rr < 2; rr++) {
+                const int d = ks * 16 + hf * 8 + 2 * tq;
+                const float *q = a.q + (size_t)(rr ? rowB : rowA) * a.heads * a.dim + (size_t)h * a.dim + d;
+                const bool v = rr ? validB : validA;
+                uint32_t h0, l0, h1, l1;
+                hilo(v && d < a.dim ? q[0] : 0.0f, h0, l0);
+                hilo(v && d + 1 < a.dim ? q[1] : 0.0f, h1, l1);
+                qh[ks][hf * 2 + rr] = h0 | (h1 << 16);
+                ql[ks][hf * 2 + rr] = l0 | (l1 << 16);
+            }
+    float o[2 * DV][4];
+#pragma unroll
+    for (int i = 0; i < 2 * DV; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
+    float mA = -INFINITY, mB = -INFINITY, lA = 0.0f, lB = 0.0f;
+    const uint32_t sKh = vb_smem_u32(Kh), sKl = vb_smem_u32(Kl), sVh = vb_smem_u32(Vh), sVl = vb_smem_u32(Vl);
+    const int mat = lane >> 3, mr = lane & 7;
+    const float inv_cap = a.softcap > 0.0f ? 1.0f / a.softcap : 0.0f;
+
+    for (int t = 0; t < kt.n_tiles; t++) {
+        int j0, n;
+        key_tile<kMaKeys>(kt, t, &j0, &n);
+        __syncthreads();
+        stage_tile<DK>(Kh, Kl, Kc, ldk, g * a.dim, a.dim, j0, n, a.ring);
+        stage_tile<DV>(Vh, Vl, Vc, ldv, g * a.vdim, a.vdim, j0, n, a.ring);
+        __syncthreads();
+        /* nothing of this tile for this warp's rows: later than all of them, or behind every window and not kept */
+        if (!active || j0 > w_imax || (a.window > 0 && w_imin - (j0 + n - 1) >= a.window && j0 >= a.keep)) continue;
+
+        float s[4][4];
+#pragma unroll
+        for (int i = 0; i < 4; i++) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
+#pragma unroll
+        for (int ks = 0; ks < DK; ks++) {
+#pragma unroll
+            for (int kp = 0; kp < 2; kp++) {           /* 16 keys each */
+                const uint32_t off = tile_off<DK>(kp * 16 + (mat >> 1) * 8 + mr, ks * 2 + (mat & 1));
+                uint32_t bh[4], bl[4];
+                ldsm(bh, sKh + off);
+                ldsm(bl, sKl + off);
+                mma_bf16(s[kp * 2], qh[ks], bh[0], bh[1]);
+                mma_bf16(s[kp * 2 + 1], qh[ks], bh[2], bh[3]);
+                mma_bf16(s[kp * 2], qh[ks], bl[0], bl[1]);
+                mma_bf16(s[kp * 2 + 1], qh[ks], bl[2], bl[3]);
+                mma_bf16(s[kp * 2], ql[ks], bh[0], bh[1]);
+                mma_bf16(s[kp * 2 + 1], ql[ks], bh[2], bh[3]);
+            }
+        }
+        float tA = -INFINITY, tB = -INFINITY;
+#pragma unroll
+        for (int nt = 0; nt < 4; nt++)
+#pragma unroll
+            for (int c = 0; c < 4; c++) {
+                const int key = nt * 8 + 2 * tq + (c & 1);
+                float v = s[nt][c] * a.scale;
+                if (a.softcap > 0.0f) v = a.softcap * tanhf(v * inv_cap);
+                if (key >= n || !key_seen(c < 2 ? iA : iB, j0 + key, a.window, a.keep)) v = -INFINITY;
+                s[nt][c] = v;
+                if (c < 2) tA = fmaxf(tA, v); else tB = fmaxf(tB, v);
+            }
+        tA = fmaxf(tA, __shfl_xor_sync(0xffffffffu, tA, 1));
+        tA = fmaxf(tA, __shfl_xor_sync(0xffffffffu, tA, 2));
+        tB = fmaxf(tB, __shfl_xor_sync(0xffffffffu, tB, 1));
+        tB = fmaxf(tB, __shfl_xor_sync(0xffffffffu, tB, 2));
+        /* a row that has seen no key yet keeps a finite reference, so that every weight below is exp(-inf) = 0 */
+        const float nA = fmaxf(mA, tA), nB = fmaxf(mB, tB);
+        const float fA = nA > -INFINITY ? nA : 0.0f, fB = nB > -INFINITY ? nB : 0.0f;
+        const float cA = expf(mA - fA), cB = expf(mB - fB);
+        mA = nA; mB = nB;
+        float sumA = 0.0f, sumB = 0.0f;
+        uint32_t ph[2][4], pl[2][4];
+#pragma unroll
+        for (int nt = 0; nt < 4; nt++) {
+            const float p0 = expf(s[nt][0] - fA), p1 = expf(s[nt][1] - fA), p2 = expf(s[nt][2] - fB), p3 = expf(s[nt][3] - fB);
+            sumA += p0 + p1;
+            sumB += p2 + p3;
+            uint32_t h0, l0, h1, l1;
+            hilo(p0, h0, l0); hilo(p1, h1, l1);
+            ph[nt >> 1][(nt & 1) * 2] = h0 | (h1 << 16);
+            pl[nt >> 1][(nt & 1) * 2] = l0 | (l1 << 16);
+            hilo(p2, h0, l0); hilo(p3, h1, l1);
+            ph[nt >> 1][(nt & 1) * 2 + 1] = h0 | (h1 << 16);
+            pl[nt >> 1][(nt & 1) * 2 + 1] = l0 | (l1 << 16);
+        }
+        lA = lA * cA + sumA;
+        lB = lB * cB + sumB;
+#pragma unroll
+        for (int i = 0; i < 2 * DV; i++) { o[i][0] *= cA; o[i][1] *= cA; o[i][2] *= cB; o[i][3] *= cB; }
+#pragma unroll
+        for (int dp = 0; dp < DV; dp++) {
+#pragma unroll
+            for (int kp = 0; kp < 2; kp++) {
+                const uint32_t off = tile_off<DV>(kp * 16 + (mat & 1) * 8 + mr, dp * 2 + (mat >> 1));
+                uint32_t vh[4], vl[4];
+                ldsm_t(vh, sVh + off);
+                ldsm_t(vl, sVl + off);
+                mma_bf16(o[2 * dp], ph[kp], vh[0], vh[1]);
+                mma_bf16(o[2 * dp + 1], ph[kp], vh[2], vh[3]);
+                mma_bf16(o[2 * dp], ph[kp], vl[0], vl[1]);
+                mma_bf16(o[2 * dp + 1], ph[kp], vl[2], vl[3]);
+                mma_bf16(o[2 * dp], pl[kp], vh[0], vh[1]);
+                mma_bf16(o[2 * dp + 1], pl[kp], vh[2], vh[3]);
+            }
+        }
+    }
+    lA += __shfl_xor_sync(0xffffffffu, lA, 1);
+    lA += __shfl_xor_sync(0xffffffffu, lA, 2);
+    lB += __shfl_xor_sync(0xffffffffu, lB, 1);
+    lB += __shfl_xor_sync(0xffffffffu, lB, 2);
+    const float rA = 1.0f / lA, rB = 1.0f / lB;
+#pragma unroll
+    for (int nt = 0; nt < 2 * DV; nt++)
+#pragma unroll
+        for (int u = 0; u < 2; u++) {
+            const int d = nt * 8 + 2 * tq + u;
+            if (d >= a.vdim) continue;
+            if (validA) lm_put(a.out, rowA, h * a.vdim + d, o[nt][u] * rA);
+            if (validB) lm_put(a.out, rowB, h * a.vdim + d, o[nt][2 + u] * rB);
+        }
+}
+
+template <int DK, int DV>
+int launch_mma(const LmAttn &a, int M, cudaStream_t st) {
+    constexpr size_t smem = (size_t)kMaKeys * 64 * (DK + DV);
+    static bool attr = false;
+    if (!attr) {
+        if (cudaFuncSetAttribute(lm_attn_mma_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+            cudaGetLastError();
+            return -1;
+        }
+        attr = true;
+    }
+    const int tiles = (M + 15) / 16 * (a.heads / a.kv_heads);
+    return ok(launch_pdl(lm_attn_mma_kernel<DK, DV>, dim3((tiles + kMaWarps - 1) / kMaWarps, a.kv_heads), dim3(kMaThreads), smem, st, a, M));
+}
+
+constexpr int kSplitBudget = 296;        /* two CTAs per SM */
+
+} // namespace
+
+size_t lm_attn_scratch_floats(int heads, int kv_heads, int vdim) {
+    (void)heads; (void)kv_heads;
+    return (size_t)kSplitBudget * kLmAttnPairs * (vdim + 2);
+}
+int lm_attn_ticket_count(int heads, int kv_heads) {
+    (void)heads; (void)kv_heads;
+    return kSplitBudget;
+}
+
+int lm_attn_prepare(const LmAttn &a, int M, cudaStream_t st) {
+    const size_t smem = sizeof(float) * ((size_t)(a.heads + a.kv_heads) * a.dim + a.rot);
+    if (smem > 200 * 1024) return -1;
+    static size_t set = 48 * 1024;
+    if (smem > set) {
+        if (cudaFuncSetAttribute(lm_attn_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+            cudaGetLastError();
+            return -1;
+        }
+        set = smem;
+    }
+    return ok(launch_pdl(lm_attn_prepare_kernel, dim3(M), dim3(kPrepThreads), smem, st, a));
+}
+
+int lm_attn_generic(const LmAttn &a, int M, cudaStream_t st) {
+    const size_t smem = ga_smem(a.dim, a.vdim);
+    if (smem > 200 * 1024) return -1;
+    static size_t set = 48 * 1024;
+    if (smem > set) {
+        if (cudaFuncSetAttribute(lm_attn_generic_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+            cudaGetLastError();
+            return -1;
+        }
+        set = smem;
+    }
+    const int tiles = (M * (a.heads / a.kv_heads) + kGaPairs - 1) / kGaPairs;
+    int splits = kSplitBudget / (tiles * a.kv_heads);
+    splits = splits < 1 ? 1 : splits > kLmAttnSplits ? kLmAttnSplits : splits;
+    return ok(launch_pdl(lm_attn_generic_kernel, dim3(tiles, a.kv_heads, splits), dim3(kGaThreads), smem, st, a, M));
+}
+
+bool lm_attn_mma_ok(const LmAttn &a) { return a.dim <= 128 && a.vdim <= 128; }
+
+int lm_attn_mma(const LmAttn &a, int M, cudaStream_t st) {
+    const bool k4 = a.dim <= 64, v4 = a.vdim <= 64;
+    if (k4) return v4 ? launch_mma<4, 4>(a, M, st) : launch_mma<4, 8>(a, M, st);
+    return v4 ? launch_mma<8, 4>(a, M, st) : launch_mma<8, 8>(a, M, st);
+}
+
+} // namespace vb

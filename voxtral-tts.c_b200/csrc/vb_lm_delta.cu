@@ -1,0 +1,217 @@
+/*
+ * vb_lm_delta.cu - decoder language models: gated delta-rule mixer.
+ *
+ *   q, k, v = silu(short causal convolution of the projections), q and k made unit vectors
+ *   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q        (per head, fp32)
+ *   out = rmsnorm(o) * silu(gate)
+ *
+ *   lm_delta_inputs  convolution, unit norms, step sizes beta, log decays: 16 rows per CTA
+ *   lm_delta_scan    the recurrence token by token; columns of S are independent, so a CTA owns 32
+ *                    of a head's value columns, four lanes per column
+ *   lm_delta_gate    head norm and gate of a row; saves the raw convolution inputs of the last rows
+ *
+ * The convolution's memory is a ring of `taps` rows indexed by position, the state S a matrix per
+ * head; both read as zero at the start of a sequence, so a slot needs no clearing.
+ */
+#include "vb_lm_kernels.cuh"
+#include "vb_tc.cuh"
+
+namespace vb {
+
+namespace {
+
+inline int ok(cudaError_t e) { return e == cudaSuccess ? 0 : -1; }
+
+VB_DEVINL float silu(float z) { return z / (1.0f + expf(-z)); }
+VB_DEVINL float softplus(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
+
+/* ------------------------------------------------------------------ inputs of the recurrence */
+constexpr int kInThreads = 128, kInRows = 16;
+
+/* grid = (row tiles, 2 * kv_heads + heads + 1): one head of q, k or v per CTA; the last column of
+ * CTAs works out step sizes and decays. */
+__global__ void __launch_bounds__(kInThreads) lm_delta_inputs_kernel(const LmDelta a, int M) {
+    extern __shared__ float in_smem[];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int r0 = blockIdx.x * kInRows, rows = M - r0 < kInRows ? M - r0 : kInRows;
+    const int tid = threadIdx.x, G = a.kv_heads, H = a.heads;
+    const int nqk = G * a.dim, ch = 2 * nqk + H * a.vdim;
+    int unit = blockIdx.y;
+    if (unit == 2 * G + H) {
+        for (int i = tid; i < rows * H; i += kInThreads) {
+            const int r = r0 + i / H, h = i % H;
+            const int cb = ch + H * a.vdim;           /* columns: q, k, v, gate, b, a */
+            a.beta[(size_t)r * H + h] = 1.0f / (1.0f + expf(-lm_sum(a.in, r, cb + h)));
+            a.ldecay[(size_t)r * H + h] = -__ldg(a.decay + h) * softplus(lm_sum(a.in, r, cb + H + h) + __ldg(a.dt_bias + h));
+        }
+        return;
+    }
+    const int kind = unit < G ? 0 : unit < 2 * G ? 1 : 2;     /* q, k, v */
+    const int head = kind == 2 ? unit - 2 * G : unit % G;
+    const int size = kind == 2 ? a.vdim : a.dim;
+    const int c0 = kind == 2 ? 2 * nqk + head * a.vdim : kind * nqk + head * a.dim;   /* first channel */
+    const int past = a.taps - 1;
+    float *raw = in_smem, *out = raw + (kInRows + past) * size;      /* [past + rows][size], [rows][size] */
+    const int pos0 = a.dyn->pos;
+    const float *tail = lm_state(a.tail, a.dyn);
+    for (int i = tid; i < (past + rows) * size; i += kInThreads) {
+        const int r = r0 - past + i / size, c = c0 + i % size;       /* row of this launch, may be an earlier token */
+        float v = 0.0f;
+        if (r >= 0) v = lm_sum(a.in, r, c);
+        else if (pos0 + r >= 0) v = tail[(size_t)((pos0 + r) % a.taps) * ch + c];
+        raw[i] = v;
+    }
+    __syncthreads();
+    for (int i = tid; i < rows * size; i += kInThreads) {
+        const int r = i / size, d = i % size;
+        const float *w = a.conv + (size_t)(c0 + d) * a.taps;
+        float v = 0.0f;
+        for (int j = 0; j < a.taps; j++) v = fmaf(__ldg(w + j), raw[(r + j) * size + d], v);
+        v = silu(v);
+        if (kind == 2) a.v[(size_t)(r0 + r) * H * a.vdim + head * a.vdim + d] = v;
+        else out[i] = v;
+    }
+    if (kind == 2) return;
+    __syncthreads();
+    const int warp = tid >> 5, lane = tid & 31;
+    float *dst = kind == 0 ? a.q : a.k;
+    const float post = kind == 0 ? 1.0f / sqrtf((float)a.dim) : 1.0f;
+    for (int r = warp; r < rows; r += kInThreads / 32) {
+        float s = 0.0f;
+        for (int d = lane; d < size; d += 32) s += out[r * size + d] * out[r * size + d];
+        s = vb_warp_sum(s);
+        const float f = 1.0f / sqrtf(s + 1e-6f) * post;
+        for (int d = lane; d < size; d += 32) dst[(size_t)(r0 + r) * nqk + head * a.dim + d] = out[r * size + d] * f;
+    }
+}
+
+/* ------------------------------------------------------------------ the recurrence, token by token */
+constexpr int kScThreads = 128, kScCols = 32, kScTok = 16;
+
+/* grid = (value column tiles, heads). Lane rg of a column's four lanes holds rows 4 i + rg of S. */
+template <int NR>
+__global__ void __launch_bounds__(kScThreads) lm_delta_scan_kernel(const LmDelta a, int M) {
+    __shared__ float ks[kScTok][4 * NR], qs[kScTok][4 * NR], vs[kScTok][kScCols], bs[kScTok], gs[kScTok];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int tid = threadIdx.x, h = blockIdx.y, kv = h / (a.heads / a.kv_heads);
+    const int rg = tid & 3, cl = tid >> 2, c = blockIdx.x * kScCols + cl;
+    const bool live = c < a.vdim;
+    const int nqk = a.kv_heads * a.dim, nv = a.heads * a.vdim;
+    float *S = lm_state(a.s, a.dyn) + (size_t)h * a.dim * a.vdim;
+    float s[NR];
+    const bool fresh = a.dyn->pos == 0;
+#pragma unroll
+    for (int i = 0; i < NR; i++) {
+        const int r = 4 * i + rg;
+        s[i] = (!fresh && live && r < a.dim) ? S[(size_t)r * a.vdim + c] : 0.0f;
+    }
+    for (int t0 = 0; t0 < M; t0 += kScTok) {
+        const int nt = M - t0 < kScTok ? M - t0 : kScTok;
+        __syncthreads();
+        for (int i = tid; i < nt * 4 * NR; i += kScThreads) {
+            const int t = i / (4 * NR), d = i % (4 * NR);
+            const size_t at = (size_t)(t0 + t) * nqk + kv * a.dim + d;
+            ks[t][d] = d < a.dim ? a.k[at] : 0.0f;
+            qs[t][d] = d < a.dim ? a.q[at] : 0.0f;
+        }
+        for (int i = tid; i < nt * kScCols; i += kScThreads) {
+            const int t = i / kScCols, cc = blockIdx.x * kScCols + i % kScCols;
+            vs[t][i % kScCols] = cc < a.vdim ? a.v[(size_t)(t0 + t) * nv + h * a.vdim + cc] : 0.0f;
+        }
+        if (tid < nt) {
+            bs[tid] = a.beta[(size_t)(t0 + tid) * a.heads + h];
+            gs[tid] = expf(a.ldecay[(size_t)(t0 + tid) * a.heads + h]);
+        }
+        __syncthreads();
+        for (int t = 0; t < nt; t++) {
+            const float g = gs[t];
+            float e0 = 0.0f, e1 = 0.0f;
+#pragma unroll
+            for (int i = 0; i < NR; i++) {
+                s[i] *= g;
+                if (i & 1) e1 = fmaf(s[i], ks[t][4 * i + rg], e1); else e0 = fmaf(s[i], ks[t][4 * i + rg], e0);
+            }
+            float e = e0 + e1;
+            e += __shfl_xor_sync(0xffffffffu, e, 1);
+            e += __shfl_xor_sync(0xffffffffu, e, 2);
+            const float u = bs[t] * (vs[t][cl] - e);
+            float o0 = 0.0f, o1 = 0.0f;
+#pragma unroll
+            for (int i = 0; i < NR; i++) {
+                s[i] = fmaf(ks[t][4 * i + rg], u, s[i]);
+                if (i & 1) o1 = fmaf(s[i], qs[t][4 * i + rg], o1); else o0 = fmaf(s[i], qs[t][4 * i + rg], o0);
+            }
+            float o = o0 + o1;
+            o += __shfl_xor_sync(0xffffffffu, o, 1);
+            o += __shfl_xor_sync(0xffffffffu, o, 2);
+            if (rg == 0 && live) a.o[(size_t)(t0 + t) * nv + h * a.vdim + c] = o;
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < NR; i++) {
+        const int r = 4 * i + rg;
+        if (live && r < a.dim) S[(size_t)r * a.vdim + c] = s[i];
+    }
+}
+
+/* ------------------------------------------------------------------ head norm, gate, convolution memory */
+constexpr int kGtThreads = 256;
+
+/* grid = rows; a warp per head. The CTAs of the last `taps` rows also save their raw convolution
+ * inputs (everything that reads the memory's old content ran in earlier launches). */
+__global__ void __launch_bounds__(kGtThreads) lm_delta_gate_kernel(const LmDelta a, int M) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int m = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int nv = a.heads * a.vdim, ch = 2 * a.kv_heads * a.dim + nv;
+    for (int h = warp; h < a.heads; h += kGtThreads / 32) {
+        const float *o = a.o + (size_t)m * nv + h * a.vdim;
+        float s = 0.0f;
+        for (int d = lane; d < a.vdim; d += 32) s += o[d] * o[d];
+        const float r = 1.0f / sqrtf(vb_warp_sum(s) / (float)a.vdim + a.eps);
+        for (int d = lane; d < a.vdim; d += 32)
+            lm_put(a.out, m, h * a.vdim + d, o[d] * r * __ldg(a.norm + d) * silu(lm_sum(a.in, m, ch + h * a.vdim + d)));
+    }
+    if (m >= M - a.taps) {
+        float *tail = lm_state(a.tail, a.dyn) + (size_t)((a.dyn->pos + m) % a.taps) * ch;
+        for (int c = tid; c < ch; c += kGtThreads) tail[c] = lm_sum(a.in, m, c);
+    }
+}
+
+} // namespace
+
+int lm_delta_channels(int heads, int kv_heads, int dim, int vdim) { return 2 * kv_heads * dim + heads * vdim; }
+bool lm_delta_supported(int dim, int vdim) { return dim >= 1 && dim <= 256 && vdim >= 1; }
+
+int lm_delta_inputs(const LmDelta &a, int M, cudaStream_t st) {
+    const int size = a.dim > a.vdim ? a.dim : a.vdim;
+    const size_t smem = sizeof(float) * (size_t)(2 * kInRows + a.taps - 1) * size;
+    if (smem > 200 * 1024) return -1;
+    static size_t set = 48 * 1024;
+    if (smem > set) {
+        if (cudaFuncSetAttribute(lm_delta_inputs_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+            cudaGetLastError();
+            return -1;
+        }
+        set = smem;
+    }
+    return ok(launch_pdl(lm_delta_inputs_kernel, dim3((M + kInRows - 1) / kInRows, 2 * a.kv_heads + a.heads + 1), dim3(kInThreads), smem,
+                         st, a, M));
+}
+
+int lm_delta_scan(const LmDelta &a, int M, cudaStream_t st) {
+    const dim3 g((a.vdim + kScCols - 1) / kScCols, a.heads), b(kScThreads);
+    if (a.dim <= 32) return ok(launch_pdl(lm_delta_scan_kernel<8>, g, b, 0, st, a, M));
+    if (a.dim <= 64) return ok(launch_pdl(lm_delta_scan_kernel<16>, g, b, 0, st, a, M));
+    if (a.dim <= 128) return ok(launch_pdl(lm_delta_scan_kernel<32>, g, b, 0, st, a, M));
+    if (a.dim <= 256) return ok(launch_pdl(lm_delta_scan_kernel<64>, g, b, 0, st, a, M));
+    return -1;
+}
+
+int lm_delta_gate(const LmDelta &a, int M, cudaStream_t st) {
+    return ok(launch_pdl(lm_delta_gate_kernel, dim3(M), dim3(kGtThreads), 0, st, a, M));
+}
+
+} // namespace vb

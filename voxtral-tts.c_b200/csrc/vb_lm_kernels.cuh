@@ -1,0 +1,166 @@
+/*
+ * vb_lm_kernels.cuh - device side of the decoder language models: argument blocks and launchers
+ * of the kernels between the GEMMs (vb_lm_kernels.cu, vb_lm_attn.cu, vb_lm_delta.cu).
+ *
+ * A kernel reads the result of a GEMM as split-K partials (LmPart), and leaves rows for the next
+ * one in an LmSink: BF16 terms for the tensor-core GEMM, or plain fp32 rows for the fp32 one.
+ * Everything in between is fp32. Where a sequence stands, and in which slot, is read from device
+ * memory (LmDyn), so that a captured graph serves every position and slot.
+ */
+#ifndef VB_LM_KERNELS_CUH
+#define VB_LM_KERNELS_CUH
+
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+#include "vb_common.cuh"
+
+namespace vb {
+
+struct LmDyn {
+    int slot;      /* whose cache and state */
+    int pos;       /* position of the first row of this launch sequence */
+    int logged;    /* tokens written by the generation loop */
+    int pad;
+};
+
+/* Split-K partials of a GEMM: n buffers [M][ld], stride floats apart; their sum is the result. */
+struct LmPart {
+    const float *p;
+    int n, ld;
+    size_t stride;
+};
+
+VB_DEVINL float lm_sum(const LmPart &g, int m, int c) {
+    const float *q = g.p + (size_t)m * g.ld + c;
+    float v = __ldcg(q);
+    for (int i = 1; i < g.n; i++) v += __ldcg(q + (size_t)i * g.stride);
+    return v;
+}
+
+/* Activation rows of the next GEMM. */
+struct LmSink {
+    float *rows;        /* fp32 rows [M][ld], or null */
+    uint16_t *terms;    /* BF16 terms [n_terms][rows_pad][ld], or null */
+    int rows_pad, ld, n_terms;
+};
+
+VB_DEVINL void lm_put(const LmSink &s, int m, int c, float v) {
+    if (s.rows) {
+        s.rows[(size_t)m * s.ld + c] = v;
+    } else {
+        uint16_t t0, t1, t2;
+        vb_split3(v, t0, t1, t2);
+        uint16_t *o = s.terms + (size_t)m * s.ld + c;
+        const size_t term = (size_t)s.rows_pad * s.ld;
+        o[0] = t0;
+        if (s.n_terms > 1) o[term] = t1;
+        if (s.n_terms > 2) o[2 * term] = t2;
+    }
+}
+
+/* State of one layer run: `base` + slot * `slab` floats. */
+struct LmState {
+    float *base;
+    size_t slab;
+};
+VB_DEVINL float *lm_state(const LmState &s, const LmDyn *dyn) { return s.base + (size_t)dyn->slot * s.slab; }
+
+/* Where position p of a windowed layer lives: the first `keep` positions have rows of their own,
+ * the others share a ring. (An unwindowed layer is a ring that never wraps.) */
+struct LmRing {
+    int keep, ring;
+};
+VB_DEVINL int lm_ring_row(const LmRing &r, int p) { return p < r.keep ? p : r.keep + (p - r.keep) % r.ring; }
+
+/* ---- residual stream (vb_lm_kernels.cu) ---- */
+enum LmNext { LM_NEXT_NONE = 0, LM_NEXT_NORM = 1, LM_NEXT_CONCAT = 2 };
+
+struct LmResidual {
+    const LmDyn *dyn;
+    const int *tokens;           /* [M] */
+    const uint16_t *embed;       /* [vocab][width] BF16 */
+    int width;
+    float eps;
+    int first;                   /* 1: x = embedding of the row's token (part unused) */
+    LmPart part;                 /* sublayer output */
+    const float *post_gain;      /* x += layernorm(part) * post_gain; null: x = part */
+    float *x;                    /* [M][width] residual stream, in and out */
+    const int *row_of;           /* optional: output row m takes row row_of[m] of part and x (x is then not stored) */
+    float *tap;                  /* optional copy of the new x, [M][width] */
+    int next;                    /* LmNext: what goes to the sink */
+    const float *next_gain;      /* LM_NEXT_NORM */
+    LmSink sink;
+};
+int lm_residual(const LmResidual &a, int M, cudaStream_t st);
+
+/* Weight repacking: row r of src [rows][K] goes to row row0 + r * step of dst [..][Kp], columns
+ * beyond K are zero. */
+int lm_pack_rows(uint16_t *dst, int Kp, int row0, int step, const uint16_t *src, int rows, int K, cudaStream_t st);
+int lm_widen(float *dst, const uint16_t *src, int n, cudaStream_t st);
+int lm_fill_random(uint16_t *dst, size_t n, uint32_t seed, float mean, float scale, cudaStream_t st);
+
+/* fp32 GEMM on the fp32 pipes: y[M][ld_out] = x[M][ldx] . W[N][ldw]^T, BF16 W. swiglu: rows of W
+ * interleaved (gate, up), y[M][N / 2] = silu(gate) * up. */
+int lm_gemm_f32(float *y, int ld_out, const float *x, int ldx, const uint16_t *W, int ldw, int M, int N, int K, bool swiglu,
+                cudaStream_t st);
+
+/* Largest logit of row 0 (first one on a tie) becomes the next token: tokens[0], log[dyn->logged++];
+ * the sequence moves on by the `rows` positions just run. */
+int lm_argmax_advance(LmDyn *dyn, int *tokens, int *log, int log_cap, LmPart logits, int vocab, int rows, cudaStream_t st);
+
+/* ---- attention (vb_lm_attn.cu) ---- */
+struct LmAttn {
+    const LmDyn *dyn;
+    int heads, kv_heads, dim, vdim;
+    int window, keep;            /* window 0: every earlier key */
+    float scale, softcap;        /* softcap 0: none */
+    int rot;                     /* rotated dimensions */
+    const float *freq;           /* [2][rot / 2]: angle per position, high and low part */
+    float mag;
+    const float *q_gain, *k_gain;
+    float eps;
+    LmRing ring;
+    LmState k, v;                /* [ring rows][kv_heads * dim], [..][kv_heads * vdim] */
+    LmPart qkv;
+    float *q;                    /* [M][heads * dim] normed and rotated */
+    float *scratch;              /* key-split partials */
+    unsigned *tickets;
+    LmSink out;
+};
+constexpr int kLmAttnSplits = 32;        /* key splits of one row's attention, at most */
+constexpr int kLmAttnPairs = 16;         /* (row, head) pairs per CTA of the generic kernel */
+size_t lm_attn_scratch_floats(int heads, int kv_heads, int vdim);
+int lm_attn_ticket_count(int heads, int kv_heads);
+int lm_attn_prepare(const LmAttn &a, int M, cudaStream_t st);              /* norm, rotation, cache append */
+int lm_attn_generic(const LmAttn &a, int M, cudaStream_t st);              /* fp32 pipes, any size */
+bool lm_attn_mma_ok(const LmAttn &a);
+int lm_attn_mma(const LmAttn &a, int M, cudaStream_t st);                  /* warp-level tensor cores, prompts */
+
+/* ---- gated delta rule (vb_lm_delta.cu) ---- */
+struct LmDelta {
+    const LmDyn *dyn;
+    int heads, kv_heads, dim, vdim, taps;
+    float eps;
+    const float *conv;           /* [2 * kv_heads * dim + heads * vdim][taps] */
+    const float *decay;          /* [heads]: exp(A_log) */
+    const float *dt_bias;        /* [heads] */
+    const float *norm;           /* [vdim] */
+    LmState s;                   /* [heads][dim][vdim] */
+    LmState tail;                /* [taps][channels] raw convolution inputs, position p in row p % taps */
+    LmPart in;                   /* columns q, k, v, gate, b, a */
+    float *q, *k, *v;            /* [M][kv_heads * dim], same, [M][heads * vdim] */
+    float *beta, *ldecay;        /* [M][heads]; log of the decay */
+    float *o;                    /* [M][heads * vdim] */
+    float *chunk;                /* per-chunk matrices of the chunked form */
+    LmSink out;
+};
+int lm_delta_channels(int heads, int kv_heads, int dim, int vdim);
+int lm_delta_inputs(const LmDelta &a, int M, cudaStream_t st);             /* convolution, unit norms, step sizes, decays */
+int lm_delta_scan(const LmDelta &a, int M, cudaStream_t st);               /* token by token, fp32 pipes */
+int lm_delta_gate(const LmDelta &a, int M, cudaStream_t st);               /* head norm, gate; saves the convolution's tail */
+bool lm_delta_supported(int dim, int vdim);
+
+} // namespace vb
+
+#endif

@@ -457,6 +457,112 @@ def micro_prefill(args):
                       "ms_per_call_median": sorted(t)[len(t) // 2]}))
 
 
+def lm_configs():
+    """Language models of real layer sizes. The first has the layers of the speech decoder: as many, as
+    wide, the same attention heads and feed-forward, nearly the same weights per layer."""
+    def build(width, ff, layers, dh, dkv, ah, akv, dim, vdim, vocab, window, loop=None):
+        mlp = {"kind": "dense", "ff": ff}
+        delta = {"type": "delta", "mlp": mlp, "mixer": {"heads": dh, "kv_heads": dkv, "dim": dim, "vdim": dim, "conv": 4}}
+        att = {"type": "attention", "mlp": mlp, "mixer": {
+            "heads": ah, "kv_heads": akv, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "softcap": 30.0,
+            "mask": {"size": window, "keep_first": 4},
+            "rot": {"dims": dim // 2, "base": 100000.0, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+        c = {"architecture": "Kegizen", "layers": [delta, att] * (layers // 2), "norm": {"eps": 1e-5}, "vocab": vocab, "width": width}
+        if loop:
+            c["loop"] = dict(zip(("start", "stop", "times"), loop))
+        return c
+    return {"w3072_l26": build(3072, 9216, 26, 24, 8, 32, 8, 128, 128, 8320, 1024),
+            "w2048_l16_loop": build(2048, 5632, 16, 16, 8, 16, 4, 128, 128, 32768, 512, (4, 12, 2)),
+            "w4096_l8": build(4096, 14336, 8, 32, 16, 32, 8, 128, 128, 65536, 2048)}
+
+
+def lm_bench(args):
+    """`--lm`: prompt and decoding throughput of the decoder language models (random weights), beside the
+    speech decoder at equal size. Device time (CUDA events); the weights of a step exceed L2 many times.
+    `--lm-only NAME` with `--m` prompt tokens and `--reps` new tokens runs one of them alone (profiling)."""
+    pkg = load_package()
+    from importlib import util
+    spec = util.spec_from_file_location("vb200_lm_binding", os.path.join(ROOT, "voxtral-tts.c_b200", "lm.py"))
+    lm_mod = util.module_from_spec(spec)
+    spec.loader.exec_module(lm_mod)
+    peak, src = measured_hbm_peak()
+    rng = np.random.default_rng(0)
+    configs = lm_configs()
+    if args.lm_only:
+        c = configs[args.lm_only]
+        if args.lm_layers:
+            c["layers"] = c["layers"][:args.lm_layers]
+            c.pop("loop", None)
+        with lm_mod.LanguageModel(config=c, max_tokens=args.m + args.reps + 8) as lm:
+            for _ in range(2):
+                s = lm.open()
+                lm.generate(s, rng.integers(0, c["vocab"], args.m), max(args.reps, 1))
+                lm.release(s)
+            print(json.dumps({"lm": args.lm_only, "prompt": args.m, "new": args.reps, "ms": lm.last_ms()}))
+        return
+    sampler = ClockSampler(int(os.environ.get("VB200_DEVICE", "0")))
+    sampler.start()
+    out = {"bench": "decoder language models", "data": "random weights and tokens", "dtype": "bf16 weights, fp32 activations as BF16 terms",
+           "hbm_gbs": peak, "peak_source": src, "models": {}}
+    time.sleep(1.5)
+    sampler.begin()
+    for name, c in configs.items():
+        with lm_mod.LanguageModel(config=c, max_tokens=8192) as lm:
+            m = {"runs": lm.info.runs, "weight_bytes": lm.info.weight_bytes, "state_bytes": lm.info.state_bytes_per_seq, "prefill": []}
+            embed = c["vocab"] * c["width"] * 2
+            layers = lm.info.weight_bytes - 2 * embed
+            loop = c.get("loop")
+            passes = lm.info.runs / len(c["layers"])
+            m["bytes_per_token"] = layers * passes + embed          # head once, embedding row negligible
+            for n in (256, 1024, 4096):
+                t = []
+                for _ in range(4):
+                    s = lm.open()
+                    lm.generate(s, rng.integers(0, c["vocab"], n), 1)
+                    t.append(lm.last_ms()[0])
+                    lm.release(s)
+                ms = min(t[1:])
+                m["prefill"].append({"tokens": n, "ms": ms, "tokens_per_s": n / ms * 1e3})
+            t = []
+            for _ in range(3):
+                s = lm.open()
+                lm.generate(s, rng.integers(0, c["vocab"], 2048), 129)
+                t.append(lm.last_ms()[1] / 128)
+                lm.release(s)
+            ms = min(t[1:])
+            m["decode"] = {"context": 2048, "ms_per_token": ms, "tokens_per_s": 1e3 / ms,
+                           "weight_gbs": m["bytes_per_token"] / ms / 1e6, "frac_of_measured": m["bytes_per_token"] / ms / 1e6 / peak}
+            m["loop"] = loop
+            out["models"][name] = m
+    sampler.end()
+    out["clocks"] = sampler.stop()
+    # the speech decoder: 26 layers, width 3072
+    import ctypes as C
+    model = pkg.SynthModel(seed=1234)
+    eng = pkg.Engine(kv_cache_max=2304)
+    eng.upload(model, decoder=True, acoustic=True, audio_table=True)
+    rows = prompt_rows(pkg, model, utterance_seeds(0)["prompt"])
+    ref = {"prefill": []}
+    for n in (256, 1024):
+        x = np.resize(rows, (n, rows.shape[1]))
+        t = []
+        for _ in range(4):
+            t0 = time.perf_counter()
+            eng.prefill(x, 0)
+            t.append((time.perf_counter() - t0) * 1e3)
+        ref["prefill"].append({"tokens": n, "ms": min(t[1:]), "tokens_per_s": n / min(t[1:]) * 1e3, "clock": "wall (synchronous call)"})
+    eng.frame(rows[0], np.zeros(36, dtype=np.float32), 300)
+    for pos in (300, 1023):
+        ms = C.c_float(0)
+        assert eng.L.vb200_decoder_step_ms(pos, 50, C.byref(ms)) == 0
+        b = 6052380672.0
+        ref.setdefault("decode", []).append({"context": pos, "ms_per_token": ms.value / 50, "weight_gbs": b / (ms.value / 50) / 1e6,
+                                             "frac_of_measured": b / (ms.value / 50) / 1e6 / peak})
+    eng.close()
+    out["speech_decoder"] = ref
+    print(json.dumps(out))
+
+
 def micro_codec(args):
     """vb200_codec_decode alone on `--m` frames of seeded codes (no decoder upload): `--reps` calls,
     device and wall time per call. The launch list of the codec decoder is taken from this command."""
@@ -566,7 +672,12 @@ def main():
     ap.add_argument("--k", type=int, default=3072)
     ap.add_argument("--n", type=int, default=32768)
     ap.add_argument("--reps", type=int, default=8)
+    ap.add_argument("--lm", action="store_true", help="the decoder language models instead of the frame loop (see lm_bench)")
+    ap.add_argument("--lm-only", default="", help="one language model alone: --m prompt tokens, --reps new tokens")
+    ap.add_argument("--lm-layers", type=int, default=0, help="--lm-only: keep the first layers only")
     args = ap.parse_args()
+    if args.lm or args.lm_only:
+        return lm_bench(args)
     if args.micro:
         return micro(args)
     if args.impl == "gpu_reference_worker":

@@ -20,6 +20,10 @@ extern "C" {
  * (which = 0) or on the open batch (which = 1). Returns the elapsed ms, the weight bytes of
  * one sweep and its launch count. */
 int vb200_gemm_sweep(int which, int iters, float *ms, double *bytes_per_sweep, int *launches_per_sweep);
+/* Measurement aid: the 26 decoder layers and the final norm of one token at cache row `pos`, as the
+ * frame graph runs them, captured alone and replayed `iters` times between two CUDA events. Needs
+ * all weights uploaded. Returns the elapsed ms. */
+int vb200_decoder_step_ms(int pos, int iters, float *ms);
 /* Measurement aid without a model: a generated [N, K] BF16 matrix, M activation rows, `reps`
  * launches of the tensor-core GEMM between two CUDA events on the default stream (split-K
  * partial epilogue, or the SwiGLU epilogue when swiglu != 0; tiled bit 0: tile-contiguous weight

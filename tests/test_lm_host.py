@@ -1,0 +1,114 @@
+"""Decoder language models, host side: configuration reader and registry (no GPU needed), and the plain
+statement's own consistency."""
+import copy
+import importlib.util
+import json
+import os
+
+import numpy as np
+import pytest
+
+import lm_plain as plain
+from lm_models import as_float, attention, config, delta, tokens, weights, write_folder
+
+
+@pytest.fixture(scope="module")
+def lm_mod(pkg):
+    from conftest import PKG_DIR
+    spec = importlib.util.spec_from_file_location("vb200_lm_binding", os.path.join(PKG_DIR, "lm.py"))
+    mod = importlib.util.module_from_spec(spec)
+    spec.loader.exec_module(mod)
+    return mod
+
+
+GOOD = config([delta(), attention(), attention(window=0, rot=0, softcap=0, ff=0)], loop=(1, 2, 2))
+
+
+def test_a_configuration_is_accepted(lm_mod):
+    lm_mod.check_config(GOOD)
+    lm_mod.check_config(json.dumps(GOOD, indent=3))
+    lm_mod.check_config({**GOOD, "loop": None, "something_else": {"x": [1, "a\\\"\\u00e9", None, True]}})
+
+
+@pytest.mark.parametrize("change,what", [
+    (lambda c: c.update(architecture="Other"), "not registered"),
+    (lambda c: c.pop("architecture"), "not registered"),
+    (lambda c: c.pop("vocab"), "vocab"),
+    (lambda c: c.update(width=0), "width"),
+    (lambda c: c.update(width=8.5), "width"),
+    (lambda c: c["norm"].pop("eps"), "eps"),
+    (lambda c: c.update(layers=[]), "layers"),
+    (lambda c: c["layers"][0].update(type="other"), "other"),
+    (lambda c: c["layers"][0]["mixer"].update(kv_heads=2), "kv_heads"),
+    (lambda c: c["layers"][0]["mixer"].pop("conv"), "conv"),
+    (lambda c: c["layers"][0]["mixer"].update(dim=300), "256"),
+    (lambda c: c["layers"][1]["mixer"].pop("scale"), "scale"),
+    (lambda c: c["layers"][1]["mixer"]["mask"].update(size=0), "size"),
+    (lambda c: c["layers"][1]["mixer"]["rot"].update(dims=7), "dims"),
+    (lambda c: c["layers"][1]["mixer"]["rot"].update(dims=34), "dims"),
+    (lambda c: c["layers"][1]["mixer"]["rot"]["scaling"].pop("fast"), "fast"),
+    (lambda c: c["layers"][1]["mlp"].update(kind="sparse"), "kind"),
+    (lambda c: c["layers"][1]["mlp"].pop("ff"), "ff"),
+    (lambda c: c["loop"].update(stop=9), "stop"),
+    (lambda c: c["loop"].update(times=0), "times"),
+])
+def test_a_wrong_configuration_is_named(lm_mod, change, what):
+    c = copy.deepcopy(GOOD)
+    change(c)
+    with pytest.raises(ValueError, match=what):
+        lm_mod.check_config(c)
+
+
+@pytest.mark.parametrize("text", ["", "{", "[1, 2", '{"a" 1}', '{"a": tru}', '{"a": "x', '{"a": 1} x', "[" * 200])
+def test_malformed_json_is_reported(lm_mod, text):
+    with pytest.raises(ValueError, match="config.json"):
+        lm_mod.check_config(text)
+
+
+def test_loading_without_a_gpu_fails_loudly(lm_mod, tmp_path):
+    import torch
+    with pytest.raises(RuntimeError, match="config.json"):
+        lm_mod.LanguageModel(str(tmp_path / "nowhere"))
+    if not torch.cuda.is_available():
+        with pytest.raises(RuntimeError):
+            lm_mod.LanguageModel(write_folder(tmp_path, GOOD, weights(GOOD, 1)))
+
+
+def test_model_folder_round_trip(tmp_path):
+    w = weights(GOOD, 1)
+    cfg, got = plain.load_folder(write_folder(tmp_path, GOOD, w))
+    assert cfg == json.loads(json.dumps(GOOD))
+    want = as_float(w)
+    assert set(got) == set(want) and all(np.array_equal(got[n], want[n]) for n in want)
+
+
+def test_statement_is_causal_and_windowed():
+    """Later tokens change nothing; a token behind the window and not kept changes nothing."""
+    cfg = config([attention(window=8, keep=2, ff=0)], width=48, vocab=50)
+    w = as_float(weights(cfg, 4))
+    t = tokens(cfg, 30, 1)
+    base = plain.forward(w, cfg, t)[0]
+    for at in (0, 1, 2, 21, 22, 29):
+        other = list(t)
+        other[at] = (t[at] + 1) % 50
+        d = np.abs(plain.forward(w, cfg, other)[0] - base).max(axis=1)
+        assert np.all(d[:at] == 0.0)
+        assert (d[29] > 0) == (at < 2 or at >= 22)
+
+
+def test_delta_rule_in_two_pieces():
+    rng = np.random.default_rng(0)
+    q, k, v = rng.standard_normal((20, 6)), rng.standard_normal((20, 6)), rng.standard_normal((20, 5))
+    b, g = rng.uniform(size=20), rng.uniform(size=20)
+    o, S = plain.delta_rule(q, k, v, b, g)
+    o1, S1 = plain.delta_rule(q[:7], k[:7], v[:7], b[:7], g[:7])
+    o2, S2 = plain.delta_rule(q[7:], k[7:], v[7:], b[7:], g[7:], S1)
+    assert np.allclose(np.concatenate([o1, o2]), o) and np.allclose(S, S2)
+
+
+def test_yarn_frequencies():
+    f, m = plain.rope_frequencies({"dims": 16, "base": 10000.0})
+    assert m == 1.0 and np.allclose(f, 10000.0 ** (-np.arange(8) / 8))
+    y, m = plain.rope_frequencies({"dims": 16, "base": 10000.0, "scaling": {"factor": 4.0, "original": 2048, "fast": 32, "slow": 1}})
+    assert np.isclose(m, 0.1 * np.log(4.0) + 1)
+    assert np.allclose(y[0], f[0]) and np.allclose(y[-1], f[-1] / 4) and np.all(y <= f) and np.all(y >= f / 4)

@@ -101,6 +101,7 @@ def lib():
         "vb200_batch_hidden": (C.c_int, [C.c_void_p]),
         "vb200_batch_launches_per_frame": (C.c_int, []),
         "vb200_batch_close": (None, []),
+        "vb200_decoder_step_ms": (C.c_int, [C.c_int, C.c_int, f32p]),
         "vb200_gemm_sweep": (C.c_int, [C.c_int, C.c_int, f32p, C.POINTER(C.c_double), i32p]),
         "vb200_frame_on_tensor_cores": (C.c_int, []),
         "vb200_tp_arena": (C.c_int, [C.c_int, C.c_int, C.c_void_p]),

@@ -174,6 +174,7 @@ int vb200_batch_end(int *codes_out, int *frames_done, int *hit_end, float *devic
 int vb200_batch_hidden(float *out) { return batch_hidden(out); }
 int vb200_batch_launches_per_frame(void) { return batch_launches_per_frame(); }
 void vb200_batch_close(void) { batch_close(); }
+int vb200_decoder_step_ms(int pos, int iters, float *ms) { return decoder_step_time(pos, iters, ms); }
 int vb200_gemm_sweep(int which, int iters, float *ms, double *bytes_per_sweep, int *launches_per_sweep) {
     return gemm_sweep(which, iters, ms, bytes_per_sweep, launches_per_sweep);
 }

@@ -993,8 +993,8 @@ static int ctx_open(Batch &t, bool single, int n_utt, int kv_max, int max_frames
     return 0;
 }
 
-/* One frame of every utterance of the context, enqueued launch by launch. */
-static int enqueue_frame(Batch &t, int embed_mode, bool advance, const float *noise, int *codes_log, int cap) {
+/* The decoder layers and the final norm for the rows in t.X, enqueued launch by launch. */
+static int enqueue_decoder(Batch &t) {
     Model &m = model();
     const BtWeights &w = g_w;
     cudaStream_t st = m.st;
@@ -1002,16 +1002,6 @@ static int enqueue_frame(Batch &t, int embed_mode, bool advance, const float *no
     const float scale = 1.0f / sqrtf((float)kHD);
     const int chunksD = tc_prepare_chunks(D);
     const size_t psD = (size_t)B * D, psQ = (size_t)B * QKV;
-    if (t.stream) {
-        /* decoder step, semantic head + argmax and llm token: one launch */
-        const int variant = embed_mode == EMBED_CODES_AFTER0 ? 0 : embed_mode == EMBED_HOST ? 1 : 2;
-        if (stream_step(t, variant)) return -1;
-        if (acoustic_tc_enqueue_on(t.ac, noise, codes_log, cap, advance, m.ignore_end)) return -1;
-        return cudaGetLastError() == cudaSuccess ? 0 : -1;
-    }
-    if (embed_mode != EMBED_HOST)
-        launch_pdl(bt_embed_kernel, dim3((D + 255) / 256, B), dim3(256), 0, st, t.X, (const uint16_t *)m.audio_table,
-                   (const int *)t.codes, (const VbDyn *)t.dyn, VB200_CODES, 8194, 23, embed_mode);
     /* Tensor parallelism: this rank's tile slice of each layer GEMM, split-K chosen for the slice. */
     const bool tp = t.tp;
     int q0 = 0, qn = 0, o0 = 0, on = 0, h0 = 0, hn = 0;
@@ -1089,6 +1079,27 @@ static int enqueue_frame(Batch &t, int embed_mode, bool advance, const float *no
     else
         launch_pdl(bt_final_kernel<false>, dim3(B), dim3(1024), 0, st, t.hidden, t.bD, 16, (const float *)t.X,
                    (const float *)t.part_w2, s_w2, psD, (const float *)m.dec_norm, VB200_NORM_EPS, last_tap, TcNoWait());
+    return cudaGetLastError() == cudaSuccess ? 0 : -1;
+}
+
+/* One frame of every utterance of the context, enqueued launch by launch. */
+static int enqueue_frame(Batch &t, int embed_mode, bool advance, const float *noise, int *codes_log, int cap) {
+    Model &m = model();
+    const BtWeights &w = g_w;
+    cudaStream_t st = m.st;
+    const int B = t.B;
+    const size_t psD = (size_t)B * D;
+    if (t.stream) {
+        /* decoder step, semantic head + argmax and llm token: one launch */
+        const int variant = embed_mode == EMBED_CODES_AFTER0 ? 0 : embed_mode == EMBED_HOST ? 1 : 2;
+        if (stream_step(t, variant)) return -1;
+        if (acoustic_tc_enqueue_on(t.ac, noise, codes_log, cap, advance, m.ignore_end)) return -1;
+        return cudaGetLastError() == cudaSuccess ? 0 : -1;
+    }
+    if (embed_mode != EMBED_HOST)
+        launch_pdl(bt_embed_kernel, dim3((D + 255) / 256, B), dim3(256), 0, st, t.X, (const uint16_t *)m.audio_table,
+                   (const int *)t.codes, (const VbDyn *)t.dyn, VB200_CODES, 8194, 23, embed_mode);
+    if (enqueue_decoder(t)) return -1;
     TcGemm g;
     g.M = B; g.status = t.status;
     /* semantic head + argmax (voxtral_tts_acoustic.c:283-309), llm token (:204) */
@@ -1280,6 +1291,34 @@ int gemm_sweep(int which, int iters, float *ms_out, double *bytes_per_sweep, int
         *bytes_per_sweep = 2.0 * VB200_DEC_LAYERS * ((double)QKV * D + (double)D * QD + 2.0 * HID * D + (double)D * HID);
     if (launches_per_sweep) *launches_per_sweep = 4 * VB200_DEC_LAYERS;
     return 0;
+}
+
+/* The decoder layers of the single-utterance frame graph alone (no heads, no acoustic part) at cache
+ * row `pos`, captured as a graph and replayed `iters` times between two events. The row `pos` is
+ * rewritten with the same values. */
+int decoder_step_time(int pos, int iters, float *ms_out) {
+    Model &m = model();
+    if (!m.inited || !m.llm_ready || iters < 1 || pos < 0 || pos >= m.kv_max || one_ready(0)) return -1;
+    Batch &t = g_one;
+    if (!t.open || t.stream) return -1;
+    t.h_in->dyn.pos = pos; t.h_in->dyn.kv_max = m.kv_max; t.h_in->dyn.frame = 0; t.h_in->dyn.done = 0;
+    if (cudaMemcpyAsync(&t.d_in->dyn, &t.h_in->dyn, sizeof(VbDyn), cudaMemcpyHostToDevice, m.st) != cudaSuccess) return -1;
+    if (enqueue_decoder(t)) return -1;
+    cudaGraph_t graph = nullptr;
+    cudaGraphExec_t exec = nullptr;
+    if (cudaStreamBeginCapture(m.st, cudaStreamCaptureModeRelaxed) != cudaSuccess) return -1;
+    const int rc = enqueue_decoder(t);
+    if (cudaStreamEndCapture(m.st, &graph) != cudaSuccess || rc || !graph) return -1;
+    const cudaError_t ie = cudaGraphInstantiate(&exec, graph, 0);
+    cudaGraphDestroy(graph);
+    if (ie != cudaSuccess) return -1;
+    for (int i = 0; i < 3; i++) cudaGraphLaunch(exec, m.st);
+    cudaEventRecord(t.e0, m.st);
+    for (int i = 0; i < iters; i++) cudaGraphLaunch(exec, m.st);
+    cudaEventRecord(t.e1, m.st);
+    const bool ok = cudaStreamSynchronize(m.st) == cudaSuccess && (!ms_out || cudaEventElapsedTime(ms_out, t.e0, t.e1) == cudaSuccess);
+    cudaGraphExecDestroy(exec);
+    return ok ? 0 : -1;
 }
 
 /* The streaming decoder step (26 layers, both heads, argmax: one launch) `iters` times back to

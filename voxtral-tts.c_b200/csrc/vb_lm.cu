@@ -18,6 +18,7 @@
 
 #include <math.h>
 #include <stdio.h>
+#include <stdlib.h>
 #include <string.h>
 
 #include <algorithm>
@@ -518,8 +519,12 @@ int vb200_lm::init(const Source &src, const vb200_lm_options_t *opt) {
     block = std::min({block, max_tokens, kTcMaxRows / 2});
     if (check_sizes(cfg)) return -1;
     runs = cfg.runs();
-    int dev = 0, major = 0;
-    LM_CUDA(cudaGetDevice(&dev));
+    int count = 0, major = 0;
+    LM_CUDA(cudaGetDeviceCount(&count));
+    const char *env = getenv("VB200_DEVICE");
+    int dev = env ? atoi(env) : 0;
+    if (dev < 0 || dev >= count) dev = 0;
+    LM_CUDA(cudaSetDevice(dev));
     LM_CUDA(cudaDeviceGetAttribute(&major, cudaDevAttrComputeCapabilityMajor, dev));
     LM_CUDA(cudaDeviceGetAttribute(&n_sm, cudaDevAttrMultiProcessorCount, dev));
     if (major != 10) return fail("an sm_100 GPU is required");

@@ -133,7 +133,8 @@ __global__ void lm_fill_random_kernel(uint16_t *dst, size_t n, uint32_t seed, fl
     dst[i] = __bfloat16_as_ushort(__float2bfloat16_rn(mean + scale * 1.7320508f * s));
 }
 
-/* 64 x 64 tile, 16 columns of K per step, 4 x 4 results per thread. */
+/* 64 x 64 tile, 16 columns of K per step, 4 x 4 results per thread. The sum over K is taken in two
+ * levels, so that its rounding error grows with the step length and the number of steps, not with K. */
 constexpr int kFgT = 64, kFgK = 16;
 __global__ void __launch_bounds__(256)
 lm_gemm_f32_kernel(float *y, int ld_out, const float *x, int ldx, const uint16_t *W, int ldw, int M, int N, int K, int swiglu) {
@@ -142,7 +143,7 @@ lm_gemm_f32_kernel(float *y, int ld_out, const float *x, int ldx, const uint16_t
     pdl_wait();
     const int n0 = blockIdx.x * kFgT, m0 = blockIdx.y * kFgT;
     const int tid = threadIdx.x, tm = (tid >> 4) * 4, tn = (tid & 15) * 4;
-    float acc[4][4] = {};
+    float sum[4][4] = {};
     for (int k0 = 0; k0 < K; k0 += kFgK) {
         for (int i = tid; i < kFgT * kFgK; i += 256) {
             const int r = i / kFgK, k = i % kFgK;
@@ -151,6 +152,7 @@ lm_gemm_f32_kernel(float *y, int ld_out, const float *x, int ldx, const uint16_t
             ws[k][r] = kin && n0 + r < N ? __uint_as_float((uint32_t)W[(size_t)(n0 + r) * ldw + k0 + k] << 16) : 0.0f;
         }
         __syncthreads();
+        float acc[4][4] = {};
 #pragma unroll
         for (int k = 0; k < kFgK; k++) {
             const float4 a = *(const float4 *)&xs[k][tm], b = *(const float4 *)&ws[k][tn];
@@ -160,6 +162,10 @@ lm_gemm_f32_kernel(float *y, int ld_out, const float *x, int ldx, const uint16_t
 #pragma unroll
                 for (int j = 0; j < 4; j++) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
         }
+#pragma unroll
+        for (int i = 0; i < 4; i++)
+#pragma unroll
+            for (int j = 0; j < 4; j++) sum[i][j] += acc[i][j];
         __syncthreads();
     }
     for (int i = 0; i < 4; i++) {
@@ -168,11 +174,11 @@ lm_gemm_f32_kernel(float *y, int ld_out, const float *x, int ldx, const uint16_t
         if (swiglu) {
             for (int j = 0; j < 4; j += 2) {
                 const int n = n0 + tn + j;
-                if (n + 1 < N) y[(size_t)m * ld_out + n / 2] = acc[i][j] / (1.0f + expf(-acc[i][j])) * acc[i][j + 1];
+                if (n + 1 < N) y[(size_t)m * ld_out + n / 2] = sum[i][j] / (1.0f + expf(-sum[i][j])) * sum[i][j + 1];
             }
         } else {
             for (int j = 0; j < 4; j++)
-                if (n0 + tn + j < N) y[(size_t)m * ld_out + n0 + tn + j] = acc[i][j];
+                if (n0 + tn + j < N) y[(size_t)m * ld_out + n0 + tn + j] = sum[i][j];
         }
     }
 }

@@ -147,6 +147,7 @@ int single_begin(const float *first_embed, int start_pos, const float *noise_all
 int single_run(int n);
 int single_end(int *codes_out, int *frames_done, int *hit_end, float *device_ms);
 int gemm_sweep(int which, int iters, float *ms_out, double *bytes_per_sweep, int *launches_per_sweep);
+int decoder_step_time(int pos, int iters, float *ms_out);
 int stream_step_time(int pos, int iters, float *ms_out, double *bytes_per_launch);
 int stream_wait_expiry(int limit_us);
 bool single_on_stream();

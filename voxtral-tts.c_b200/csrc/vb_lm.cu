@@ -600,9 +600,13 @@ int vb200_lm::mixer(const Layer &l, const LmMixer &m, const RunState &s, int M) 
         a.k = {slabs + s.a, slab}; a.v = {slabs + s.b, slab};
         a.qkv = in; a.q = q; a.scratch = scratch; a.tickets = tickets;
         a.out = sink(l.mix.acts, M);
-        LM_DO(lm_attn_prepare(a, M, st));
-        if (!f32() && M > 8 && lm_attn_mma_ok(a)) LM_DO(lm_attn_mma(a, M, st));
-        else LM_DO(lm_attn_generic(a, M, st));
+        if (M == 1 && lm_attn_step_ok(a)) {
+            LM_DO(lm_attn_step(a, st));
+        } else {
+            LM_DO(lm_attn_prepare(a, M, st));
+            if (!f32() && M > 8 && lm_attn_mma_ok(a)) LM_DO(lm_attn_mma(a, M, st));
+            else LM_DO(lm_attn_generic(a, M, st));
+        }
     } else {
         LmDelta d = {};
         d.dyn = dyn();
@@ -612,9 +616,13 @@ int vb200_lm::mixer(const Layer &l, const LmMixer &m, const RunState &s, int M) 
         d.s = {slabs + s.a, slab}; d.tail = {slabs + s.b, slab};
         d.in = in; d.q = q; d.k = k; d.v = v; d.beta = beta; d.ldecay = ldecay; d.o = o;
         d.out = sink(l.mix.acts, M);
-        LM_DO(lm_delta_inputs(d, M, st));
-        LM_DO(lm_delta_scan(d, M, st));
-        LM_DO(lm_delta_gate(d, M, st));
+        if (M == 1 && lm_delta_step_ok(d)) {
+            LM_DO(lm_delta_step(d, st));
+        } else {
+            LM_DO(lm_delta_inputs(d, M, st));
+            LM_DO(lm_delta_scan(d, M, st));
+            LM_DO(lm_delta_gate(d, M, st));
+        }
     }
     return 0;
 }

@@ -5,7 +5,9 @@
  *
  *   lm_attn_prepare  one row per CTA: sums the projection's split-K partials, norms and rotates q
  *                    and k, appends k and v to the cache
- *   lm_attn_generic  fp32 pipes: decode (keys split over CTAs, last arrival merges) and the 32-bit mode
+ *   lm_attn_generic  fp32 pipes: any sizes, short portions and the 32-bit mode (keys split over CTAs,
+ *                    last arrival merges)
+ *   lm_attn_step     one token, preparation included
  *   lm_attn_mma      prompts: mma.sync on hi + lo BF16 halves of q, k, v and the weights
  *
  * Keys are visited in two stretches, the kept first tokens and the window; a stretch that is out
@@ -244,6 +246,241 @@ __global__ void __launch_bounds__(kGaThreads) lm_attn_generic_kernel(const LmAtt
     }
 }
 
+/* ------------------------------------------------------------------ one token */
+constexpr int kSaThreads = 512, kSaWarps = 16;
+
+/* grid = (key splits, KV heads). Every CTA sums the squares of the whole q and k projection itself
+ * (a few L2 reads instead of another launch), norms and rotates its own heads, and attends over its
+ * share of the visible keys: a warp serves one head of the group on one of 16 / (heads of the group)
+ * subsets of the keys, KP keys in flight, a lane four dimensions per step. The last split owns the
+ * new token and appends it. ND, NV: 128-wide steps of the key and value sizes. */
+template <int ND, int NV, int KP>
+__global__ void __launch_bounds__(kSaThreads) lm_attn_step_kernel(const LmAttn a, int lanes_h) {
+    extern __shared__ __align__(16) float sa[];
+    __shared__ float red[2][kSaWarps], sub_m[kSaWarps], sub_l[kSaWarps], wgt[kLmAttnSplits * kSaWarps];
+    __shared__ int last_flag;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int dim = a.dim, vdim = a.vdim, group = a.heads / a.kv_heads, half = a.rot / 2;
+    const int nq = a.heads * dim, nk = a.kv_heads * dim, nv = a.kv_heads * vdim;
+    float *raw = sa;                                       /* [group * dim] own q, then [dim] own k */
+    float *qs = raw + (group + 1) * dim;                   /* [group][dim] */
+    float *os = qs + group * dim;                          /* [16 warps][vdim] */
+    float *cs = os + kSaWarps * vdim;                      /* [rot] */
+    pdl_launch_dependents();
+    pdl_wait();
+    const int sp = blockIdx.x, g = blockIdx.y;
+    const int pos = a.dyn->pos;
+    /* visible keys in order: the kept ones, then the window */
+    const int n_keep = a.window > 0 ? (a.keep < pos + 1 ? a.keep : pos + 1) : 0;
+    const int w0 = a.window > 0 ? (pos - a.window + 1 > n_keep ? pos - a.window + 1 : n_keep) : 0;
+    const int n_keys = n_keep + (pos + 1 - w0);
+    int S = (n_keys + 31) / 32;
+    if (S > (int)gridDim.x) S = gridDim.x;
+    if (sp >= S) return;
+    const int x0 = (int)((long long)n_keys * sp / S), x1 = (int)((long long)n_keys * (sp + 1) / S);
+    const bool writer = sp == S - 1;
+
+    float sq = 0.0f, sk = 0.0f;
+    const int own0 = g * group * dim, own1 = own0 + group * dim, k0 = nq + g * dim, k1 = k0 + dim;
+    for (int c = tid * 4; c < nq + nk; c += kSaThreads * 4) {
+        const float4 v = lm_sum4(a.qkv, 0, c);
+        const float ss = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        if (c < nq) sq += ss; else sk += ss;
+        if (c >= own0 && c < own1) *reinterpret_cast<float4 *>(raw + c - own0) = v;
+        else if (c >= k0 && c < k1) *reinterpret_cast<float4 *>(raw + group * dim + c - k0) = v;
+    }
+    float *Kc = lm_state(a.k, a.dyn) + g * dim, *Vc = lm_state(a.v, a.dyn) + g * vdim;
+    const size_t new_row = (size_t)lm_ring_row(a.ring, pos);
+    if (writer)
+        for (int c = tid; c < vdim; c += kSaThreads) Vc[new_row * nv + c] = lm_sum_batch(a.qkv, 0, nq + nk + g * vdim + c);
+    for (int i = tid; i < half; i += kSaThreads) {
+        const float p = (float)pos, f = a.freq[i];
+        const float hi = p * f, lo = fmaf(p, f, -hi) + p * a.freq[half + i];
+        float s, c;
+        sincosf(hi, &s, &c);
+        cs[i] = (c - s * lo) * a.mag;
+        cs[half + i] = (s + c * lo) * a.mag;
+    }
+    sq = vb_warp_sum(sq);
+    sk = vb_warp_sum(sk);
+    if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+    __syncthreads();
+    sq = sk = 0.0f;
+#pragma unroll
+    for (int w = 0; w < kSaWarps; w++) { sq += red[0][w]; sk += red[1][w]; }
+    const float rq = 1.0f / sqrtf(sq / (float)nq + a.eps), rk = 1.0f / sqrtf(sk / (float)nk + a.eps);
+    const int total = (writer ? group + 1 : group) * dim;
+    for (int i = tid; i < total; i += kSaThreads) {
+        const bool isq = i < group * dim;
+        const int d = i % dim;
+        const float *gain = isq ? a.q_gain + own0 + i : a.k_gain + g * dim + d;
+        const float r = isq ? rq : rk;
+        float v = raw[i] * r * __ldg(gain);
+        if (d < a.rot) {
+            const int j = d < half ? d : d - half, other = d < half ? half : -half;
+            const float u = raw[i + other] * r * __ldg(gain + other);
+            v = d < half ? v * cs[j] - u * cs[half + j] : v * cs[j] + u * cs[half + j];
+        }
+        if (isq) qs[i] = v;
+        else Kc[new_row * nk + d] = v;
+    }
+    __syncthreads();          /* the appended row is visible to this CTA */
+
+    const int hh = warp % lanes_h, sub = warp / lanes_h, subs = kSaWarps / lanes_h;
+    float mx = -INFINITY, den = 0.0f, o[NV][4];
+#pragma unroll
+    for (int i = 0; i < NV; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
+    if (hh < group) {
+        float4 q[ND];
+#pragma unroll
+        for (int i = 0; i < ND; i++) {
+            const int d = i * 128 + lane * 4;
+            q[i] = d < dim ? *reinterpret_cast<const float4 *>(qs + hh * dim + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+        for (int xb = x0 + sub; xb < x1; xb += KP * subs) {
+            float4 kk[KP][ND], vv[KP][NV];
+#pragma unroll
+            for (int u = 0; u < KP; u++) {
+                const int x = xb + u * subs;
+                const bool in = x < x1;
+                const size_t row = in ? (size_t)lm_ring_row(a.ring, x < n_keep ? x : w0 + x - n_keep) : 0;
+#pragma unroll
+                for (int i = 0; i < ND; i++) {
+                    const int d = i * 128 + lane * 4;
+                    kk[u][i] = in && d < dim ? vb_ldcg4(Kc + row * nk + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+                }
+#pragma unroll
+                for (int i = 0; i < NV; i++) {
+                    const int d = i * 128 + lane * 4;
+                    vv[u][i] = in && d < vdim ? vb_ldcg4(Vc + row * nv + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+                }
+            }
+            float s[KP];
+#pragma unroll
+            for (int u = 0; u < KP; u++) {
+                s[u] = 0.0f;
+#pragma unroll
+                for (int i = 0; i < ND; i++)
+                    s[u] += q[i].x * kk[u][i].x + q[i].y * kk[u][i].y + q[i].z * kk[u][i].z + q[i].w * kk[u][i].w;
+            }
+#pragma unroll
+            for (int off = 16; off > 0; off >>= 1)
+#pragma unroll
+                for (int u = 0; u < KP; u++) s[u] += __shfl_xor_sync(0xffffffffu, s[u], off);
+            float top = mx;
+#pragma unroll
+            for (int u = 0; u < KP; u++) {
+                s[u] *= a.scale;
+                if (a.softcap > 0.0f) s[u] = a.softcap * tanhf(s[u] / a.softcap);
+                if (xb + u * subs >= x1) s[u] = -INFINITY;
+                top = fmaxf(top, s[u]);
+            }
+            const float c = expf(mx - top);               /* the first key of a pass is always there: top is finite */
+            mx = top;
+            den *= c;
+#pragma unroll
+            for (int i = 0; i < NV; i++) { o[i][0] *= c; o[i][1] *= c; o[i][2] *= c; o[i][3] *= c; }
+#pragma unroll
+            for (int u = 0; u < KP; u++) {
+                const float w = expf(s[u] - top);
+                den += w;
+#pragma unroll
+                for (int i = 0; i < NV; i++) {
+                    o[i][0] = fmaf(w, vv[u][i].x, o[i][0]);
+                    o[i][1] = fmaf(w, vv[u][i].y, o[i][1]);
+                    o[i][2] = fmaf(w, vv[u][i].z, o[i][2]);
+                    o[i][3] = fmaf(w, vv[u][i].w, o[i][3]);
+                }
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        const int d = i * 128 + lane * 4;
+        if (d < vdim) *reinterpret_cast<float4 *>(os + warp * vdim + d) = make_float4(o[i][0], o[i][1], o[i][2], o[i][3]);
+    }
+    if (lane == 0) { sub_m[warp] = mx; sub_l[warp] = den; }
+    __syncthreads();
+    /* merge the key subsets of every head, in order */
+    const int stride = vdim + 2;
+    float *po = a.scratch + (size_t)g * gridDim.x * group * stride;            /* [split][head][vdim + 2] */
+    for (int i = tid; i < group * vdim; i += kSaThreads) {
+        const int hd = i / vdim, d = i % vdim;
+        float M0 = -INFINITY, L = 0.0f, O = 0.0f;
+        for (int u = 0; u < subs; u++) M0 = fmaxf(M0, sub_m[u * lanes_h + hd]);
+        for (int u = 0; u < subs; u++) {
+            const int w = u * lanes_h + hd;
+            const float f = sub_m[w] > -INFINITY ? expf(sub_m[w] - M0) : 0.0f;
+            L = fmaf(sub_l[w], f, L);
+            O = fmaf(os[w * vdim + d], f, O);
+        }
+        if (S == 1) {
+            lm_put(a.out, 0, (g * group + hd) * vdim + d, O / L);
+        } else {
+            float *mine = po + ((size_t)sp * group + hd) * stride;
+            mine[d] = O;
+            if (d == 0) { mine[vdim] = M0; mine[vdim + 1] = L; }
+        }
+    }
+    if (S == 1) return;
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) {
+        const unsigned t = atomicAdd(&a.tickets[g], 1u);
+        last_flag = t == (unsigned)(S - 1);
+        if (last_flag) a.tickets[g] = 0u;
+    }
+    __syncthreads();
+    if (!last_flag) return;
+    __threadfence();
+    /* weights of the slices per head, then the slices in order */
+    if (tid < group) {
+        float m[kLmAttnSplits], M0 = -INFINITY, L = 0.0f;
+#pragma unroll
+        for (int u = 0; u < kLmAttnSplits; u++) m[u] = u < S ? __ldcg(po + ((size_t)u * group + tid) * stride + vdim) : -INFINITY;
+#pragma unroll
+        for (int u = 0; u < kLmAttnSplits; u++) M0 = fmaxf(M0, m[u]);
+#pragma unroll
+        for (int u = 0; u < kLmAttnSplits; u++)
+            if (u < S) {
+                const float f = expf(m[u] - M0);
+                L = fmaf(__ldcg(po + ((size_t)u * group + tid) * stride + vdim + 1), f, L);
+                wgt[u * kSaWarps + tid] = f;
+            }
+        sub_l[tid] = L;
+    }
+    __syncthreads();
+    for (int i = tid; i < group * vdim; i += kSaThreads) {
+        const int hd = i / vdim, d = i % vdim;
+        float t[kLmAttnSplits], O = 0.0f;
+#pragma unroll
+        for (int u = 0; u < kLmAttnSplits; u++) t[u] = u < S ? __ldcg(po + ((size_t)u * group + hd) * stride + d) : 0.0f;
+#pragma unroll
+        for (int u = 0; u < kLmAttnSplits; u++)
+            if (u < S) O = fmaf(t[u], wgt[u * kSaWarps + hd], O);
+        lm_put(a.out, 0, (g * group + hd) * vdim + d, O / sub_l[hd]);
+    }
+}
+
+inline size_t step_smem(const LmAttn &a) {
+    const int group = a.heads / a.kv_heads;
+    return sizeof(float) * ((size_t)(2 * group + 1) * a.dim + (size_t)kSaWarps * a.vdim + a.rot + 4);
+}
+
+template <int ND, int NV, int KP>
+int launch_attn_step(const LmAttn &a, int splits, int lanes_h, cudaStream_t st) {
+    const size_t smem = step_smem(a);
+    static size_t set = 48 * 1024;
+    if (smem > set) {
+        if (cudaFuncSetAttribute(lm_attn_step_kernel<ND, NV, KP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+            cudaGetLastError();
+            return -1;
+        }
+        set = smem;
+    }
+    return ok(launch_pdl(lm_attn_step_kernel<ND, NV, KP>, dim3(splits, a.kv_heads), dim3(kSaThreads), smem, st, a, lanes_h));
+}
+
 /* ------------------------------------------------------------------ prompts on the warp-level tensor cores */
 VB_DEVINL void hilo(float v, uint32_t &hi, uint32_t &lo) {
     const __nv_bfloat16 h = __float2bfloat16_rn(v);
@@ -473,6 +710,7 @@ int launch_mma(const LmAttn &a, int M, cudaStream_t st) {
 }
 
 constexpr int kSplitBudget = 296;        /* two CTAs per SM */
+constexpr int kStepCtas = 148;           /* one-token kernel: one CTA per SM */
 
 } // namespace
 
@@ -522,6 +760,21 @@ int lm_attn_mma(const LmAttn &a, int M, cudaStream_t st) {
     const bool k4 = a.dim <= 64, v4 = a.vdim <= 64;
     if (k4) return v4 ? launch_mma<4, 4>(a, M, st) : launch_mma<4, 8>(a, M, st);
     return v4 ? launch_mma<8, 4>(a, M, st) : launch_mma<8, 8>(a, M, st);
+}
+
+bool lm_attn_step_ok(const LmAttn &a) {
+    return a.heads / a.kv_heads <= kSaWarps && a.kv_heads <= kSplitBudget && a.dim % 4 == 0 && a.vdim % 4 == 0 && a.dim <= 256 &&
+           a.vdim <= 256;
+}
+
+int lm_attn_step(const LmAttn &a, cudaStream_t st) {
+    const int group = a.heads / a.kv_heads;
+    int lanes_h = 1;
+    while (lanes_h < group) lanes_h *= 2;
+    int splits = kStepCtas / a.kv_heads;
+    splits = splits < 1 ? 1 : splits > kLmAttnSplits ? kLmAttnSplits : splits;
+    if (a.dim <= 128 && a.vdim <= 128) return launch_attn_step<1, 1, 8>(a, splits, lanes_h, st);
+    return launch_attn_step<2, 2, 4>(a, splits, lanes_h, st);
 }
 
 } // namespace vb

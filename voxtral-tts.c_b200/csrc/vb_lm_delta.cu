@@ -9,12 +9,15 @@
  *   lm_delta_scan    the recurrence token by token; columns of S are independent, so a CTA owns 32
  *                    of a head's value columns, four lanes per column
  *   lm_delta_gate    head norm and gate of a row; saves the raw convolution inputs of the last rows
+ *   lm_delta_step    one token in one launch: a cluster of CTAs per head, 32 value columns each
  *
  * The convolution's memory is a ring of `taps` rows indexed by position, the state S a matrix per
  * head; both read as zero at the start of a sequence, so a slot needs no clearing.
  */
 #include "vb_lm_kernels.cuh"
 #include "vb_tc.cuh"
+
+#include <cooperative_groups.h>
 
 namespace vb {
 
@@ -180,6 +183,128 @@ __global__ void __launch_bounds__(kGtThreads) lm_delta_gate_kernel(const LmDelta
     }
 }
 
+/* ------------------------------------------------------------------ one token */
+constexpr int kStThreads = 256, kStWarps = 8, kStCols = 32;
+
+/* grid = (value column slices, heads), the slices of a head form a cluster. Warp w holds rows
+ * w, w + 8, ... of S, a lane one column. The memory row of the convolution that is written
+ * (position p, row p % taps) is none of those that other CTAs read (p - 1 ... p - taps + 1). */
+template <int NR>
+__global__ void __launch_bounds__(kStThreads) lm_delta_step_kernel(const LmDelta a) {
+    __shared__ float qs[8 * NR], ks[8 * NR], vs[kStCols], red[2][kStWarps], part[2][kStWarps][kStCols], scal[2], ssq;
+    namespace cg = cooperative_groups;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int h = blockIdx.y, group = a.heads / a.kv_heads, kv = h / group, H = a.heads;
+    const int col0 = blockIdx.x * kStCols, c = col0 + lane;
+    const bool live = c < a.vdim;
+    const int pos = a.dyn->pos, nqk = a.kv_heads * a.dim, ch = 2 * nqk + H * a.vdim;
+    float *S = lm_state(a.s, a.dyn) + (size_t)h * a.dim * a.vdim;
+    float *tail = lm_state(a.tail, a.dyn);
+
+    /* the state is requested first: it is the long way */
+    float s[NR];
+#pragma unroll
+    for (int i = 0; i < NR; i++) {
+        const int r = warp + 8 * i;
+        s[i] = (pos > 0 && live && r < a.dim) ? __ldcg(S + (size_t)r * a.vdim + c) : 0.0f;
+    }
+    float gate = 0.0f;
+    if (warp == 0 && live) gate = lm_sum_batch(a.in, 0, ch + h * a.vdim + c);
+    if (warp == 1 && lane < 2) {
+        const float x = lm_sum_batch(a.in, 0, ch + H * a.vdim + lane * H + h);
+        scal[lane] = lane == 0 ? 1.0f / (1.0f + expf(-x)) : expf(-__ldg(a.decay + h) * softplus(x + __ldg(a.dt_bias + h)));
+    }
+    /* convolution of this head's q and k and of the slice's v */
+    const int ncols = a.vdim - col0 < kStCols ? a.vdim - col0 : kStCols;
+    float sq = 0.0f, sk = 0.0f;
+    for (int i = tid; i < 2 * a.dim + ncols; i += kStThreads) {
+        const int kind = i < a.dim ? 0 : i < 2 * a.dim ? 1 : 2;
+        const int chan = kind == 0 ? kv * a.dim + i : kind == 1 ? nqk + kv * a.dim + i - a.dim : 2 * nqk + h * a.vdim + col0 + i - 2 * a.dim;
+        const float raw = lm_sum_batch(a.in, 0, chan);
+        const float *w = a.conv + (size_t)chan * a.taps;
+        float v = 0.0f;
+        for (int j = 0; j < a.taps - 1; j++) {
+            const int p = pos - (a.taps - 1) + j;
+            if (p >= 0) v = fmaf(__ldg(w + j), __ldcg(tail + (size_t)(p % a.taps) * ch + chan), v);
+        }
+        v = silu(fmaf(__ldg(w + a.taps - 1), raw, v));
+        if (kind == 2 || (blockIdx.x == 0 && h % group == 0)) tail[(size_t)(pos % a.taps) * ch + chan] = raw;
+        if (kind == 0) { qs[i] = v; sq += v * v; }
+        else if (kind == 1) { ks[i - a.dim] = v; sk += v * v; }
+        else vs[i - 2 * a.dim] = v;
+    }
+    for (int i = a.dim + tid; i < 8 * NR; i += kStThreads) qs[i] = ks[i] = 0.0f;
+    sq = vb_warp_sum(sq);
+    sk = vb_warp_sum(sk);
+    if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+    __syncthreads();
+    sq = sk = 0.0f;
+#pragma unroll
+    for (int w = 0; w < kStWarps; w++) { sq += red[0][w]; sk += red[1][w]; }
+    const float fq = 1.0f / sqrtf(sq + 1e-6f) / sqrtf((float)a.dim), fk = 1.0f / sqrtf(sk + 1e-6f);
+    const float beta = scal[0], g = scal[1];
+    float e = 0.0f;
+#pragma unroll
+    for (int i = 0; i < NR; i++) {
+        s[i] *= g;
+        e = fmaf(s[i], ks[warp + 8 * i] * fk, e);
+    }
+    part[0][warp][lane] = e;
+    __syncthreads();
+    e = 0.0f;
+#pragma unroll
+    for (int w = 0; w < kStWarps; w++) e += part[0][w][lane];
+    const float u = live ? beta * (vs[lane] - e) : 0.0f;
+    float o = 0.0f;
+#pragma unroll
+    for (int i = 0; i < NR; i++) {
+        s[i] = fmaf(ks[warp + 8 * i] * fk, u, s[i]);
+        o = fmaf(s[i], qs[warp + 8 * i] * fq, o);
+    }
+    part[1][warp][lane] = o;
+#pragma unroll
+    for (int i = 0; i < NR; i++) {
+        const int r = warp + 8 * i;
+        if (live && r < a.dim) S[(size_t)r * a.vdim + c] = s[i];
+    }
+    __syncthreads();
+    if (warp == 0) {
+        o = 0.0f;
+#pragma unroll
+        for (int w = 0; w < kStWarps; w++) o += part[1][w][lane];
+        const float t = vb_warp_sum(live ? o * o : 0.0f);
+        if (lane == 0) ssq = t;
+    }
+    /* the head's norm spans the cluster's slices */
+    cg::cluster_group cluster = cg::this_cluster();
+    cluster.sync();
+    if (warp == 0) {
+        float t = 0.0f;
+        for (unsigned r = 0; r < cluster.num_blocks(); r++) t += *cluster.map_shared_rank(&ssq, r);
+        const float rn = 1.0f / sqrtf(t / (float)a.vdim + a.eps);
+        if (live) lm_put(a.out, 0, h * a.vdim + c, o * rn * __ldg(a.norm + c) * silu(gate));
+    }
+    cluster.sync();                                   /* nobody leaves while its sum may still be read */
+}
+
+template <int NR>
+int launch_step(const LmDelta &a, cudaStream_t st) {
+    cudaLaunchConfig_t cfg = {};
+    const unsigned slices = (unsigned)(a.vdim + kStCols - 1) / kStCols;
+    cfg.gridDim = dim3(slices, a.heads); cfg.blockDim = dim3(kStThreads); cfg.stream = st;
+    cudaLaunchAttribute at[2];
+    at[0].id = cudaLaunchAttributeClusterDimension;
+    at[0].val.clusterDim.x = slices; at[0].val.clusterDim.y = 1; at[0].val.clusterDim.z = 1;
+    at[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = at;
+    static const bool no_pdl = getenv("VB200_NO_PDL") != nullptr;
+    cfg.numAttrs = no_pdl ? 1 : 2;
+    return ok(cudaLaunchKernelEx(&cfg, lm_delta_step_kernel<NR>, a));
+}
+
 } // namespace
 
 int lm_delta_channels(int heads, int kv_heads, int dim, int vdim) { return 2 * kv_heads * dim + heads * vdim; }
@@ -212,6 +337,15 @@ int lm_delta_scan(const LmDelta &a, int M, cudaStream_t st) {
 
 int lm_delta_gate(const LmDelta &a, int M, cudaStream_t st) {
     return ok(launch_pdl(lm_delta_gate_kernel, dim3(M), dim3(kGtThreads), 0, st, a, M));
+}
+
+bool lm_delta_step_ok(const LmDelta &a) { return a.dim <= 256 && a.vdim <= 8 * kStCols; }
+
+int lm_delta_step(const LmDelta &a, cudaStream_t st) {
+    if (a.dim <= 32) return launch_step<4>(a, st);
+    if (a.dim <= 64) return launch_step<8>(a, st);
+    if (a.dim <= 128) return launch_step<16>(a, st);
+    return launch_step<32>(a, st);
 }
 
 } // namespace vb

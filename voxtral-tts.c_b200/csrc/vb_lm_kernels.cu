@@ -10,100 +10,127 @@ namespace vb {
 
 namespace {
 
-constexpr int kResThreads = 512;
-
 /* Sum over the CTA; `red` holds one float per warp and is a different array for successive calls. */
 VB_DEVINL float cta_sum(float v, float *red) {
     v = vb_warp_sum(v);
-    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    const int lane = threadIdx.x & 31, warps = (int)blockDim.x >> 5;
+    if (lane == 0) red[threadIdx.x >> 5] = v;
     __syncthreads();
-    float t = 0.0f;
-#pragma unroll
-    for (int w = 0; w < kResThreads / 32; w++) t += red[w];
-    return t;
+    return vb_warp_sum(lane < warps ? red[lane] : 0.0f);
 }
 
 /* One row of the residual stream per CTA, held in registers: the sublayer's output (split-K
  * partials) is normalised, added to the stream, and the new row is normalised again for the next
- * sublayer. Variances are means of squared deviations. */
-template <int NV>
-__global__ void __launch_bounds__(kResThreads) lm_residual_kernel(const LmResidual a) {
-    __shared__ float red[4][kResThreads / 32];
+ * sublayer. Variances are means of squared deviations. A thread owns NV groups of VEC columns. */
+template <int VEC, int NV>
+__global__ void __launch_bounds__(1024) lm_residual_kernel(const LmResidual a) {
+    __shared__ float red[4][32];
+    constexpr int N = VEC * NV;
     pdl_launch_dependents();
-    pdl_wait();
-    const int m = blockIdx.x, src = a.row_of ? a.row_of[m] : m;
-    const int tid = threadIdx.x, W = a.width;
+    const int m = blockIdx.x, tid = threadIdx.x, W = a.width;
     const float inv_w = 1.0f / (float)W;
-    float x[NV];
+    auto col = [&](int i) { return (tid + i * (int)blockDim.x) * VEC; };
+    /* the gains depend on nothing that runs before */
+    float gp[N], gn[N];
+#pragma unroll
+    for (int i = 0; i < NV; i++)
+#pragma unroll
+        for (int j = 0; j < VEC; j++) {
+            const int c = col(i) + j;
+            gp[i * VEC + j] = a.post_gain && c < W ? __ldg(a.post_gain + c) : 0.0f;
+            gn[i * VEC + j] = a.next == LM_NEXT_NORM && c < W ? __ldg(a.next_gain + c) : 0.0f;
+        }
+    pdl_wait();
+    const int src = a.row_of ? a.row_of[m] : m;
+    float x[N];
     const bool need0 = a.first || a.next == LM_NEXT_CONCAT;
     const uint16_t *e0 = need0 ? a.embed + (size_t)a.tokens[src] * W : nullptr;
     if (a.first) {
 #pragma unroll
-        for (int i = 0; i < NV; i++) {
-            const int c = tid + i * kResThreads;
-            x[i] = c < W ? __uint_as_float((uint32_t)e0[c] << 16) : 0.0f;
-        }
+        for (int i = 0; i < NV; i++)
+#pragma unroll
+            for (int j = 0; j < VEC; j++) x[i * VEC + j] = col(i) < W ? __uint_as_float((uint32_t)e0[col(i) + j] << 16) : 0.0f;
     } else {
-        float r[NV];
+        float r[N];
         const bool add = a.post_gain != nullptr;
 #pragma unroll
         for (int i = 0; i < NV; i++) {
-            const int c = tid + i * kResThreads;
-            x[i] = c < W ? lm_sum(a.part, src, c) : 0.0f;
-            r[i] = (add && c < W) ? a.x[(size_t)src * W + c] : 0.0f;
+            const int c = col(i);
+            const bool in = c < W;
+            if constexpr (VEC == 4) {
+                const float4 rv = in && add ? __ldcg(reinterpret_cast<const float4 *>(a.x + (size_t)src * W + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
+                const float4 xv = in ? lm_sum4(a.part, src, c) : make_float4(0.f, 0.f, 0.f, 0.f);
+                x[i * 4] = xv.x; x[i * 4 + 1] = xv.y; x[i * 4 + 2] = xv.z; x[i * 4 + 3] = xv.w;
+                r[i * 4] = rv.x; r[i * 4 + 1] = rv.y; r[i * 4 + 2] = rv.z; r[i * 4 + 3] = rv.w;
+            } else {
+                r[i] = in && add ? a.x[(size_t)src * W + c] : 0.0f;
+                x[i] = in ? lm_sum_batch(a.part, src, c) : 0.0f;
+            }
         }
         if (add) {
             float s = 0.0f;
 #pragma unroll
-            for (int i = 0; i < NV; i++) s += x[i];
+            for (int i = 0; i < N; i++) s += x[i];
             const float mean = cta_sum(s, red[0]) * inv_w;
             s = 0.0f;
 #pragma unroll
-            for (int i = 0; i < NV; i++) {
-                const int c = tid + i * kResThreads;
-                x[i] = c < W ? x[i] - mean : 0.0f;
+            for (int i = 0; i < N; i++) {
+                x[i] = col(i / VEC) < W ? x[i] - mean : 0.0f;
                 s += x[i] * x[i];
             }
             const float rstd = 1.0f / sqrtf(cta_sum(s, red[1]) * inv_w + a.eps);
 #pragma unroll
-            for (int i = 0; i < NV; i++) {
-                const int c = tid + i * kResThreads;
-                if (c < W) x[i] = r[i] + x[i] * rstd * __ldg(a.post_gain + c);
-            }
+            for (int i = 0; i < N; i++) x[i] = r[i] + x[i] * rstd * gp[i];      /* zero beyond the row */
         }
     }
 #pragma unroll
     for (int i = 0; i < NV; i++) {
-        const int c = tid + i * kResThreads;
+        const int c = col(i);
         if (c >= W) continue;
-        if (!a.row_of) a.x[(size_t)m * W + c] = x[i];
-        if (a.tap) a.tap[(size_t)m * W + c] = x[i];
+#pragma unroll
+        for (int t = 0; t < 2; t++) {
+            float *dst = t ? a.tap : a.row_of ? nullptr : a.x;
+            if (!dst) continue;
+            dst += (size_t)m * W + c;
+            if constexpr (VEC == 4) *reinterpret_cast<float4 *>(dst) = make_float4(x[i * 4], x[i * 4 + 1], x[i * 4 + 2], x[i * 4 + 3]);
+            else *dst = x[i];
+        }
     }
+    auto put = [&](int c, const float *v) {
+        if constexpr (VEC == 4) {
+            const float q[4] = {v[0], v[1], v[2], v[3]};
+            lm_put4(a.sink, m, c, q);
+        } else {
+            lm_put(a.sink, m, c, *v);
+        }
+    };
     if (a.next == LM_NEXT_NORM) {
         float s = 0.0f;
 #pragma unroll
-        for (int i = 0; i < NV; i++) s += x[i];
+        for (int i = 0; i < N; i++) s += x[i];
         const float mean = cta_sum(s, red[2]) * inv_w;
         s = 0.0f;
 #pragma unroll
-        for (int i = 0; i < NV; i++) {
-            const int c = tid + i * kResThreads;
-            x[i] = c < W ? x[i] - mean : 0.0f;
+        for (int i = 0; i < N; i++) {
+            x[i] = col(i / VEC) < W ? x[i] - mean : 0.0f;
             s += x[i] * x[i];
         }
         const float rstd = 1.0f / sqrtf(cta_sum(s, red[3]) * inv_w + a.eps);
 #pragma unroll
-        for (int i = 0; i < NV; i++) {
-            const int c = tid + i * kResThreads;
-            if (c < W) lm_put(a.sink, m, c, x[i] * rstd * __ldg(a.next_gain + c));
-        }
+        for (int i = 0; i < N; i++) x[i] = x[i] * rstd * gn[i];
+#pragma unroll
+        for (int i = 0; i < NV; i++)
+            if (col(i) < W) put(col(i), x + i * VEC);
     } else if (a.next == LM_NEXT_CONCAT) {
 #pragma unroll
         for (int i = 0; i < NV; i++) {
-            const int c = tid + i * kResThreads;
+            const int c = col(i);
             if (c >= W) continue;
-            lm_put(a.sink, m, c, x[i]);
-            lm_put(a.sink, m, W + c, __uint_as_float((uint32_t)e0[c] << 16));
+            float e[VEC];
+#pragma unroll
+            for (int j = 0; j < VEC; j++) e[j] = __uint_as_float((uint32_t)e0[c + j] << 16);
+            put(c, x + i * VEC);
+            put(W + c, e);
         }
     }
 }
@@ -221,14 +248,19 @@ inline int ok(cudaError_t e) { return e == cudaSuccess ? 0 : -1; }
 
 int lm_residual(const LmResidual &a, int M, cudaStream_t st) {
     if (M <= 0) return 0;
-    const int nv = (a.width + kResThreads - 1) / kResThreads;
-    const dim3 g(M), b(kResThreads);
-    if (nv <= 1) return ok(launch_pdl(lm_residual_kernel<1>, g, b, 0, st, a));
-    if (nv <= 2) return ok(launch_pdl(lm_residual_kernel<2>, g, b, 0, st, a));
-    if (nv <= 4) return ok(launch_pdl(lm_residual_kernel<4>, g, b, 0, st, a));
-    if (nv <= 8) return ok(launch_pdl(lm_residual_kernel<8>, g, b, 0, st, a));
-    if (nv <= 16) return ok(launch_pdl(lm_residual_kernel<16>, g, b, 0, st, a));
-    if (nv <= 32) return ok(launch_pdl(lm_residual_kernel<32>, g, b, 0, st, a));
+    const bool v4 = (a.width & 3) == 0;
+    const int groups = v4 ? a.width / 4 : a.width;
+    const int threads = groups >= 1024 ? 1024 : (groups + 31) / 32 * 32, nv = (groups + threads - 1) / threads;
+    const dim3 g(M), b(threads);
+    if (v4) {
+        if (nv <= 1) return ok(launch_pdl(lm_residual_kernel<4, 1>, g, b, 0, st, a));
+        if (nv <= 2) return ok(launch_pdl(lm_residual_kernel<4, 2>, g, b, 0, st, a));
+        if (nv <= 4) return ok(launch_pdl(lm_residual_kernel<4, 4>, g, b, 0, st, a));
+    } else {
+        if (nv <= 1) return ok(launch_pdl(lm_residual_kernel<1, 1>, g, b, 0, st, a));
+        if (nv <= 4) return ok(launch_pdl(lm_residual_kernel<1, 4>, g, b, 0, st, a));
+        if (nv <= 16) return ok(launch_pdl(lm_residual_kernel<1, 16>, g, b, 0, st, a));
+    }
     return -1;
 }
 

@@ -24,6 +24,8 @@ struct LmDyn {
     int pad;
 };
 
+constexpr int kLmMaxParts = 8;   /* split-K factor limit of the GEMM */
+
 /* Split-K partials of a GEMM: n buffers [M][ld], stride floats apart; their sum is the result. */
 struct LmPart {
     const float *p;
@@ -36,6 +38,29 @@ VB_DEVINL float lm_sum(const LmPart &g, int m, int c) {
     float v = __ldcg(q);
     for (int i = 1; i < g.n; i++) v += __ldcg(q + (size_t)i * g.stride);
     return v;
+}
+
+/* The same with every partial requested before the first is used. */
+VB_DEVINL float lm_sum_batch(const LmPart &g, int m, int c) {
+    const float *q = g.p + (size_t)m * g.ld + c;
+    float t[kLmMaxParts], v = 0.0f;
+#pragma unroll
+    for (int i = 0; i < kLmMaxParts; i++) t[i] = i < g.n ? __ldcg(q + (size_t)i * g.stride) : 0.0f;
+#pragma unroll
+    for (int i = 0; i < kLmMaxParts; i++) v += t[i];
+    return v;
+}
+/* Four columns from c on (c and ld multiples of 4). */
+VB_DEVINL float4 lm_sum4(const LmPart &g, int m, int c) {
+    const float *q = g.p + (size_t)m * g.ld + c;
+    float4 t[kLmMaxParts];
+#pragma unroll
+    for (int i = 0; i < kLmMaxParts; i++)
+        t[i] = i < g.n ? __ldcg(reinterpret_cast<const float4 *>(q + (size_t)i * g.stride)) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 1; i < kLmMaxParts; i++)
+        if (i < g.n) { t[0].x += t[i].x; t[0].y += t[i].y; t[0].z += t[i].z; t[0].w += t[i].w; }
+    return t[0];
 }
 
 /* Activation rows of the next GEMM. */
@@ -56,6 +81,23 @@ VB_DEVINL void lm_put(const LmSink &s, int m, int c, float v) {
         o[0] = t0;
         if (s.n_terms > 1) o[term] = t1;
         if (s.n_terms > 2) o[2 * term] = t2;
+    }
+}
+
+/* Four columns from c on (a multiple of 4; rows are padded to multiples of 64). */
+VB_DEVINL void lm_put4(const LmSink &s, int m, int c, const float (&v)[4]) {
+    if (s.rows) {
+        *reinterpret_cast<float4 *>(s.rows + (size_t)m * s.ld + c) = make_float4(v[0], v[1], v[2], v[3]);
+    } else {
+        uint16_t t[3][4];
+#pragma unroll
+        for (int i = 0; i < 4; i++) vb_split3(v[i], t[0][i], t[1][i], t[2][i]);
+        uint16_t *o = s.terms + (size_t)m * s.ld + c;
+        const size_t term = (size_t)s.rows_pad * s.ld;
+#pragma unroll
+        for (int j = 0; j < 3; j++)
+            if (j < s.n_terms)
+                *reinterpret_cast<uint2 *>(o + j * term) = make_uint2(t[j][0] | ((uint32_t)t[j][1] << 16), t[j][2] | ((uint32_t)t[j][3] << 16));
     }
 }
 
@@ -134,6 +176,8 @@ size_t lm_attn_scratch_floats(int heads, int kv_heads, int vdim);
 int lm_attn_ticket_count(int heads, int kv_heads);
 int lm_attn_prepare(const LmAttn &a, int M, cudaStream_t st);              /* norm, rotation, cache append */
 int lm_attn_generic(const LmAttn &a, int M, cudaStream_t st);              /* fp32 pipes, any size */
+bool lm_attn_step_ok(const LmAttn &a);
+int lm_attn_step(const LmAttn &a, cudaStream_t st);                        /* one token: norm, rotation, append, attention */
 bool lm_attn_mma_ok(const LmAttn &a);
 int lm_attn_mma(const LmAttn &a, int M, cudaStream_t st);                  /* warp-level tensor cores, prompts */
 
@@ -159,6 +203,8 @@ int lm_delta_channels(int heads, int kv_heads, int dim, int vdim);
 int lm_delta_inputs(const LmDelta &a, int M, cudaStream_t st);             /* convolution, unit norms, step sizes, decays */
 int lm_delta_scan(const LmDelta &a, int M, cudaStream_t st);               /* token by token, fp32 pipes */
 int lm_delta_gate(const LmDelta &a, int M, cudaStream_t st);               /* head norm, gate; saves the convolution's tail */
+bool lm_delta_step_ok(const LmDelta &a);
+int lm_delta_step(const LmDelta &a, cudaStream_t st);                      /* one token: all of the above in one launch */
 bool lm_delta_supported(int dim, int vdim);
 
 } // namespace vb

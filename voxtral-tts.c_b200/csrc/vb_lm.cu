@@ -132,7 +132,7 @@ struct vb200_lm {
 
     /* activations */
     float *x = nullptr, *part_in = nullptr, *part_out = nullptr, *part_head = nullptr, *logits = nullptr;
-    float *q = nullptr, *k = nullptr, *v = nullptr, *o = nullptr, *beta = nullptr, *ldecay = nullptr;
+    float *q = nullptr, *k = nullptr, *v = nullptr, *o = nullptr, *beta = nullptr, *decays = nullptr;
     float *scratch = nullptr, *tap = nullptr;
     unsigned *tickets = nullptr;
     int *status = nullptr, *log = nullptr, *zero = nullptr;
@@ -485,7 +485,7 @@ int vb200_lm::make_buffers() {
     const size_t B = block;
     if (alloc(&x, B * W) || alloc(&part_in, in) || alloc(&part_out, out) || alloc(&part_head, part_floats(head, kHeadRows)) ||
         alloc(&logits, (size_t)kHeadRows * head.N) || alloc(&q, B * qn) || alloc(&k, B * kn) || alloc(&v, B * vn) || alloc(&o, B * on) ||
-        alloc(&beta, B * hn) || alloc(&ldecay, B * hn) || alloc(&scratch, scr) || alloc(&tickets, (size_t)tick, true) ||
+        alloc(&beta, B * hn) || alloc(&decays, B * hn) || alloc(&scratch, scr) || alloc(&tickets, (size_t)tick, true) ||
         alloc(&status, 4, true) || alloc(&log, kLogCap, true) || alloc(&zero, 4, true) || alloc(&d_in, 4 + 2 * B, true))
         return -1;
     for (int i = 0; i < 2; i++) {
@@ -598,13 +598,14 @@ int vb200_lm::mixer(const Layer &l, const LmMixer &m, const RunState &s, int M) 
         a.q_gain = l.mix.q_gain; a.k_gain = l.mix.k_gain; a.eps = (float)cfg.eps;
         a.ring = s.ring;
         a.k = {slabs + s.a, slab}; a.v = {slabs + s.b, slab};
+        a.split = !f32() && lm_attn_mma_ok(m.dim, m.vdim);
         a.qkv = in; a.q = q; a.scratch = scratch; a.tickets = tickets;
         a.out = sink(l.mix.acts, M);
         if (M == 1 && lm_attn_step_ok(a)) {
             LM_DO(lm_attn_step(a, st));
         } else {
             LM_DO(lm_attn_prepare(a, M, st));
-            if (!f32() && M > 8 && lm_attn_mma_ok(a)) LM_DO(lm_attn_mma(a, M, st));
+            if (a.split && M > 8) LM_DO(lm_attn_mma(a, M, st));
             else LM_DO(lm_attn_generic(a, M, st));
         }
     } else {
@@ -614,7 +615,7 @@ int vb200_lm::mixer(const Layer &l, const LmMixer &m, const RunState &s, int M) 
         d.eps = (float)cfg.eps;
         d.conv = l.mix.conv; d.decay = l.mix.decay; d.dt_bias = l.mix.dt_bias; d.norm = l.mix.norm;
         d.s = {slabs + s.a, slab}; d.tail = {slabs + s.b, slab};
-        d.in = in; d.q = q; d.k = k; d.v = v; d.beta = beta; d.ldecay = ldecay; d.o = o;
+        d.in = in; d.q = q; d.k = k; d.v = v; d.beta = beta; d.decays = decays; d.o = o;
         d.out = sink(l.mix.acts, M);
         if (M == 1 && lm_delta_step_ok(d)) {
             LM_DO(lm_delta_step(d, st));

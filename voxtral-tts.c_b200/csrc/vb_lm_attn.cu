@@ -8,7 +8,8 @@
  *   lm_attn_generic  fp32 pipes: any sizes, short portions and the 32-bit mode (keys split over CTAs,
  *                    last arrival merges)
  *   lm_attn_step     one token, preparation included
- *   lm_attn_mma      prompts: mma.sync on hi + lo BF16 halves of q, k, v and the weights
+ *   lm_attn_mma      prompts: mma.sync on hi + lo BF16 halves of q, k, v and the weights; the cache keeps
+ *                    k and v as such halves
  *
  * Keys are visited in two stretches, the kept first tokens and the window; a stretch that is out
  * of reach of all of a CTA's rows is never loaded.
@@ -21,6 +22,38 @@ namespace vb {
 namespace {
 
 inline int ok(cudaError_t e) { return e == cudaSuccess ? 0 : -1; }
+
+/* ------------------------------------------------------------------ cache elements */
+VB_DEVINL void hilo(float v, uint32_t &hi, uint32_t &lo) {
+    const __nv_bfloat16 h = __float2bfloat16_rn(v);
+    hi = __bfloat16_as_ushort(h);
+    lo = __bfloat16_as_ushort(__float2bfloat16_rn(v - __bfloat162float(h)));
+}
+/* `head`: a head's part of a cache row, `size` elements in either form. */
+VB_DEVINL void kv_put(float *head, int size, int d, float v, int split) {
+    if (split) {
+        uint32_t hi, lo;
+        hilo(v, hi, lo);
+        uint16_t *h = reinterpret_cast<uint16_t *>(head);
+        h[d] = (uint16_t)hi;
+        h[size + d] = (uint16_t)lo;
+    } else {
+        head[d] = v;
+    }
+}
+VB_DEVINL float kv_get(const float *head, int size, int d, int split) {
+    if (!split) return __ldcg(head + d);
+    const unsigned short *h = reinterpret_cast<const unsigned short *>(head);
+    return __uint_as_float((uint32_t)__ldcg(h + d) << 16) + __uint_as_float((uint32_t)__ldcg(h + size + d) << 16);
+}
+template <bool SPLIT>
+VB_DEVINL float4 kv_get4(const float *head, int size, int d) {
+    if constexpr (!SPLIT) return vb_ldcg4(head + d);
+    const uint16_t *h = reinterpret_cast<const uint16_t *>(head);
+    const uint2 hi = __ldcg(reinterpret_cast<const uint2 *>(h + d)), lo = __ldcg(reinterpret_cast<const uint2 *>(h + size + d));
+    return make_float4(vb_bf16_lo(hi.x) + vb_bf16_lo(lo.x), vb_bf16_hi(hi.x) + vb_bf16_hi(lo.x), vb_bf16_lo(hi.y) + vb_bf16_lo(lo.y),
+                       vb_bf16_hi(hi.y) + vb_bf16_hi(lo.y));
+}
 
 /* ------------------------------------------------------------------ q, k, v of a row */
 constexpr int kPrepThreads = 512;
@@ -53,7 +86,7 @@ __global__ void __launch_bounds__(kPrepThreads) lm_attn_prepare_kernel(const LmA
         if (c < nq) sq += v * v; else sk += v * v;
     }
     float *Vr = lm_state(a.v, a.dyn) + row * nv;
-    for (int c = tid; c < nv; c += kPrepThreads) Vr[c] = lm_sum(a.qkv, m, nq + nk + c);
+    for (int c = tid; c < nv; c += kPrepThreads) kv_put(Vr + c / a.vdim * a.vdim, a.vdim, c % a.vdim, lm_sum(a.qkv, m, nq + nk + c), a.split);
     sq = vb_warp_sum(sq);
     sk = vb_warp_sum(sk);
     if ((tid & 31) == 0) { red[0][tid >> 5] = sq; red[1][tid >> 5] = sk; }
@@ -74,7 +107,8 @@ __global__ void __launch_bounds__(kPrepThreads) lm_attn_prepare_kernel(const LmA
             const float u = buf[c + other] * r * __ldg(gain + j + other);
             v = d < half ? v * cs[i] - u * cs[half + i] : v * cs[i] + u * cs[half + i];
         }
-        (isq ? Q : Kr)[j] = v;
+        if (isq) Q[j] = v;
+        else kv_put(Kr + j - d, a.dim, d, v, a.split);
     }
 }
 
@@ -151,11 +185,11 @@ __global__ void __launch_bounds__(kGaThreads) lm_attn_generic_kernel(const LmAtt
         __syncthreads();
         for (int i = tid; i < n * dim; i += kGaThreads) {
             const int j = i / dim, d = i % dim;
-            K[j * (dim + 1) + d] = __ldcg(Kc + (size_t)lm_ring_row(a.ring, j0 + j) * ldk + g * dim + d);
+            K[j * (dim + 1) + d] = kv_get(Kc + (size_t)lm_ring_row(a.ring, j0 + j) * ldk + g * dim, dim, d, a.split);
         }
         for (int i = tid; i < n * vdim; i += kGaThreads) {
             const int j = i / vdim, d = i % vdim;
-            V[i] = __ldcg(Vc + (size_t)lm_ring_row(a.ring, j0 + j) * ldv + g * vdim + d);
+            V[i] = kv_get(Vc + (size_t)lm_ring_row(a.ring, j0 + j) * ldv + g * vdim, vdim, d, a.split);
         }
         __syncthreads();
         for (int p = warp; p < np; p += kGaThreads / 32) {
@@ -254,7 +288,7 @@ constexpr int kSaThreads = 512, kSaWarps = 16;
  * share of the visible keys: a warp serves one head of the group on one of 16 / (heads of the group)
  * subsets of the keys, KP keys in flight, a lane four dimensions per step. The last split owns the
  * new token and appends it. ND, NV: 128-wide steps of the key and value sizes. */
-template <int ND, int NV, int KP>
+template <int ND, int NV, int KP, bool SPLIT>
 __global__ void __launch_bounds__(kSaThreads) lm_attn_step_kernel(const LmAttn a, int lanes_h) {
     extern __shared__ __align__(16) float sa[];
     __shared__ float red[2][kSaWarps], sub_m[kSaWarps], sub_l[kSaWarps], wgt[kLmAttnSplits * kSaWarps];
@@ -292,7 +326,7 @@ __global__ void __launch_bounds__(kSaThreads) lm_attn_step_kernel(const LmAttn a
     float *Kc = lm_state(a.k, a.dyn) + g * dim, *Vc = lm_state(a.v, a.dyn) + g * vdim;
     const size_t new_row = (size_t)lm_ring_row(a.ring, pos);
     if (writer)
-        for (int c = tid; c < vdim; c += kSaThreads) Vc[new_row * nv + c] = lm_sum_batch(a.qkv, 0, nq + nk + g * vdim + c);
+        for (int c = tid; c < vdim; c += kSaThreads) kv_put(Vc + new_row * nv, vdim, c, lm_sum_batch(a.qkv, 0, nq + nk + g * vdim + c), SPLIT);
     for (int i = tid; i < half; i += kSaThreads) {
         const float p = (float)pos, f = a.freq[i];
         const float hi = p * f, lo = fmaf(p, f, -hi) + p * a.freq[half + i];
@@ -322,7 +356,7 @@ __global__ void __launch_bounds__(kSaThreads) lm_attn_step_kernel(const LmAttn a
             v = d < half ? v * cs[j] - u * cs[half + j] : v * cs[j] + u * cs[half + j];
         }
         if (isq) qs[i] = v;
-        else Kc[new_row * nk + d] = v;
+        else kv_put(Kc + new_row * nk, dim, d, v, SPLIT);
     }
     __syncthreads();          /* the appended row is visible to this CTA */
 
@@ -347,12 +381,12 @@ __global__ void __launch_bounds__(kSaThreads) lm_attn_step_kernel(const LmAttn a
 #pragma unroll
                 for (int i = 0; i < ND; i++) {
                     const int d = i * 128 + lane * 4;
-                    kk[u][i] = in && d < dim ? vb_ldcg4(Kc + row * nk + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+                    kk[u][i] = in && d < dim ? kv_get4<SPLIT>(Kc + row * nk, dim, d) : make_float4(0.f, 0.f, 0.f, 0.f);
                 }
 #pragma unroll
                 for (int i = 0; i < NV; i++) {
                     const int d = i * 128 + lane * 4;
-                    vv[u][i] = in && d < vdim ? vb_ldcg4(Vc + row * nv + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+                    vv[u][i] = in && d < vdim ? kv_get4<SPLIT>(Vc + row * nv, vdim, d) : make_float4(0.f, 0.f, 0.f, 0.f);
                 }
             }
             float s[KP];
@@ -467,26 +501,21 @@ inline size_t step_smem(const LmAttn &a) {
     return sizeof(float) * ((size_t)(2 * group + 1) * a.dim + (size_t)kSaWarps * a.vdim + a.rot + 4);
 }
 
-template <int ND, int NV, int KP>
+template <int ND, int NV, int KP, bool SPLIT>
 int launch_attn_step(const LmAttn &a, int splits, int lanes_h, cudaStream_t st) {
     const size_t smem = step_smem(a);
     static size_t set = 48 * 1024;
     if (smem > set) {
-        if (cudaFuncSetAttribute(lm_attn_step_kernel<ND, NV, KP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+        if (cudaFuncSetAttribute(lm_attn_step_kernel<ND, NV, KP, SPLIT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
             cudaGetLastError();
             return -1;
         }
         set = smem;
     }
-    return ok(launch_pdl(lm_attn_step_kernel<ND, NV, KP>, dim3(splits, a.kv_heads), dim3(kSaThreads), smem, st, a, lanes_h));
+    return ok(launch_pdl(lm_attn_step_kernel<ND, NV, KP, SPLIT>, dim3(splits, a.kv_heads), dim3(kSaThreads), smem, st, a, lanes_h));
 }
 
 /* ------------------------------------------------------------------ prompts on the warp-level tensor cores */
-VB_DEVINL void hilo(float v, uint32_t &hi, uint32_t &lo) {
-    const __nv_bfloat16 h = __float2bfloat16_rn(v);
-    hi = __bfloat16_as_ushort(h);
-    lo = __bfloat16_as_ushort(__float2bfloat16_rn(v - __bfloat162float(h)));
-}
 VB_DEVINL void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
@@ -509,33 +538,22 @@ VB_DEVINL uint32_t tile_off(int key, int chunk) {
 
 constexpr int kMaThreads = 256, kMaWarps = 8, kMaKeys = 32;
 
-/* Stages 32 keys of one KV head: fp32 rows of the cache -> hi and lo BF16 tiles, zero beyond the
- * keys and beyond the head's size. */
+/* Requests 32 keys of one KV head: the high and low halves of the cache rows, 16 bytes per copy,
+ * straight into the swizzled tiles. What lies beyond the head's size in a tile is not touched. */
 template <int STEPS>
-VB_DEVINL void stage_tile(unsigned char *hi_t, unsigned char *lo_t, const float *cache, int ld, int col0, int size, int j0, int n,
-                          const LmRing &ring) {
-    constexpr int kQuads = STEPS * 4;                   /* groups of four values per row */
-    for (int i = threadIdx.x; i < kMaKeys * kQuads; i += kMaThreads) {
-        const int key = i / kQuads, f = i % kQuads;
-        float e[4] = {0.f, 0.f, 0.f, 0.f};
-        if (key < n && 4 * f < size) {
-            const float *src = cache + (size_t)lm_ring_row(ring, j0 + key) * ld + col0 + 4 * f;
-            if ((size & 3) == 0) {
-                const float4 v = __ldcg(reinterpret_cast<const float4 *>(src));
-                e[0] = v.x; e[1] = v.y; e[2] = v.z; e[3] = v.w;
-            } else {
-#pragma unroll
-                for (int u = 0; u < 4; u++)
-                    if (4 * f + u < size) e[u] = __ldcg(src + u);
-            }
-        }
-        uint32_t h[4], l[4];
-#pragma unroll
-        for (int u = 0; u < 4; u++) hilo(e[u], h[u], l[u]);
-        const uint32_t off = tile_off<STEPS>(key, f >> 1) + (uint32_t)(f & 1) * 8u;
-        *reinterpret_cast<uint2 *>(hi_t + off) = make_uint2(h[0] | (h[1] << 16), h[2] | (h[3] << 16));
-        *reinterpret_cast<uint2 *>(lo_t + off) = make_uint2(l[0] | (l[1] << 16), l[2] | (l[3] << 16));
+VB_DEVINL void request_tile(unsigned char *hi_t, const float *cache, int ld, int col0, int size, int j0, int n, const LmRing &ring) {
+    const int per = size / 8;                           /* chunks of a plane */
+    for (int i = threadIdx.x; i < n * 2 * per; i += kMaThreads) {
+        const int key = i / (2 * per), f = i % (2 * per), plane = f >= per ? 1 : 0, chunk = f - plane * per;
+        const uint16_t *src = reinterpret_cast<const uint16_t *>(cache + (size_t)lm_ring_row(ring, j0 + key) * ld + col0) + f * 8;
+        unsigned char *dst = hi_t + plane * (kMaKeys * STEPS * 32) + tile_off<STEPS>(key, chunk);
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(vb_smem_u32(dst)), "l"(src) : "memory");
     }
+}
+
+/* cap * tanh(x / cap), the hyperbolic tangent through one exponential (absolute error about 1e-7 of cap) */
+VB_DEVINL float soft_cap(float x, float cap, float two_over_cap) {
+    return cap - 2.0f * cap * __fdividef(1.0f, 1.0f + __expf(x * two_over_cap));
 }
 
 /* A CTA serves one KV head; each of its eight warps owns 16 query rows of one query head of the
@@ -546,9 +564,12 @@ VB_DEVINL void stage_tile(unsigned char *hi_t, unsigned char *lo_t, const float 
 template <int DK, int DV>
 __global__ void __launch_bounds__(kMaThreads) lm_attn_mma_kernel(const LmAttn a, int M) {
     extern __shared__ __align__(128) unsigned char ma_tiles[];
-    unsigned char *Kh = ma_tiles, *Kl = Kh + kMaKeys * DK * 32, *Vh = Kl + kMaKeys * DK * 32, *Vl = Vh + kMaKeys * DV * 32;
+    /* two buffers of K high, K low, V high, V low */
+    constexpr int kTileK = kMaKeys * DK * 32, kTileV = kMaKeys * DV * 32, kBuf = 2 * (kTileK + kTileV);
     pdl_launch_dependents();
+    for (int i = threadIdx.x; i < 2 * kBuf / 16; i += kMaThreads) reinterpret_cast<uint4 *>(ma_tiles)[i] = make_uint4(0u, 0u, 0u, 0u);
     pdl_wait();
+    __syncthreads();
     const int group = a.heads / a.kv_heads, g = blockIdx.y;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3;
     const int n_tiles_q = (M + 15) / 16 * group;
@@ -588,17 +609,26 @@ __global__ void __launch_bounds__(kMaThreads) lm_attn_mma_kernel(const LmAttn a,
 #pragma unroll
     for (int i = 0; i < 2 * DV; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
     float mA = -INFINITY, mB = -INFINITY, lA = 0.0f, lB = 0.0f;
-    const uint32_t sKh = vb_smem_u32(Kh), sKl = vb_smem_u32(Kl), sVh = vb_smem_u32(Vh), sVl = vb_smem_u32(Vl);
+    const uint32_t smem0 = vb_smem_u32(ma_tiles);
     const int mat = lane >> 3, mr = lane & 7;
-    const float inv_cap = a.softcap > 0.0f ? 1.0f / a.softcap : 0.0f;
+    const float two_over_cap = a.softcap > 0.0f ? 2.0f / a.softcap : 0.0f;
+    auto request = [&](int t) {
+        int j0, n;
+        key_tile<kMaKeys>(kt, t, &j0, &n);
+        unsigned char *b = ma_tiles + (t & 1) * kBuf;
+        request_tile<DK>(b, Kc, ldk, g * a.dim, a.dim, j0, n, a.ring);
+        request_tile<DV>(b + 2 * kTileK, Vc, ldv, g * a.vdim, a.vdim, j0, n, a.ring);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    if (kt.n_tiles > 0) request(0);
 
     for (int t = 0; t < kt.n_tiles; t++) {
         int j0, n;
         key_tile<kMaKeys>(kt, t, &j0, &n);
-        __syncthreads();
-        stage_tile<DK>(Kh, Kl, Kc, ldk, g * a.dim, a.dim, j0, n, a.ring);
-        stage_tile<DV>(Vh, Vl, Vc, ldv, g * a.vdim, a.vdim, j0, n, a.ring);
-        __syncthreads();
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();                               /* this buffer is complete, the other one is free */
+        if (t + 1 < kt.n_tiles) request(t + 1);
+        const uint32_t sKh = smem0 + (uint32_t)((t & 1) * kBuf), sKl = sKh + kTileK, sVh = sKl + kTileK, sVl = sVh + kTileV;
         /* nothing of this tile for this warp's rows: later than all of them, or behind every window and not kept */
         if (!active || j0 > w_imax || (a.window > 0 && w_imin - (j0 + n - 1) >= a.window && j0 >= a.keep)) continue;
 
@@ -628,7 +658,7 @@ __global__ void __launch_bounds__(kMaThreads) lm_attn_mma_kernel(const LmAttn a,
             for (int c = 0; c < 4; c++) {
                 const int key = nt * 8 + 2 * tq + (c & 1);
                 float v = s[nt][c] * a.scale;
-                if (a.softcap > 0.0f) v = a.softcap * tanhf(v * inv_cap);
+                if (a.softcap > 0.0f) v = soft_cap(v, a.softcap, two_over_cap);
                 if (key >= n || !key_seen(c < 2 ? iA : iB, j0 + key, a.window, a.keep)) v = -INFINITY;
                 s[nt][c] = v;
                 if (c < 2) tA = fmaxf(tA, v); else tB = fmaxf(tB, v);
@@ -696,7 +726,7 @@ __global__ void __launch_bounds__(kMaThreads) lm_attn_mma_kernel(const LmAttn a,
 
 template <int DK, int DV>
 int launch_mma(const LmAttn &a, int M, cudaStream_t st) {
-    constexpr size_t smem = (size_t)kMaKeys * 64 * (DK + DV);
+    constexpr size_t smem = (size_t)2 * kMaKeys * 64 * (DK + DV);
     static bool attr = false;
     if (!attr) {
         if (cudaFuncSetAttribute(lm_attn_mma_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
@@ -754,7 +784,7 @@ int lm_attn_generic(const LmAttn &a, int M, cudaStream_t st) {
     return ok(launch_pdl(lm_attn_generic_kernel, dim3(tiles, a.kv_heads, splits), dim3(kGaThreads), smem, st, a, M));
 }
 
-bool lm_attn_mma_ok(const LmAttn &a) { return a.dim <= 128 && a.vdim <= 128; }
+bool lm_attn_mma_ok(int dim, int vdim) { return dim <= 128 && vdim <= 128 && dim % 8 == 0 && vdim % 8 == 0; }
 
 int lm_attn_mma(const LmAttn &a, int M, cudaStream_t st) {
     const bool k4 = a.dim <= 64, v4 = a.vdim <= 64;
@@ -773,8 +803,9 @@ int lm_attn_step(const LmAttn &a, cudaStream_t st) {
     while (lanes_h < group) lanes_h *= 2;
     int splits = kStepCtas / a.kv_heads;
     splits = splits < 1 ? 1 : splits > kLmAttnSplits ? kLmAttnSplits : splits;
-    if (a.dim <= 128 && a.vdim <= 128) return launch_attn_step<1, 1, 8>(a, splits, lanes_h, st);
-    return launch_attn_step<2, 2, 4>(a, splits, lanes_h, st);
+    if (a.split) return launch_attn_step<1, 1, 8, true>(a, splits, lanes_h, st);      /* sizes up to 128 */
+    if (a.dim <= 128 && a.vdim <= 128) return launch_attn_step<1, 1, 8, false>(a, splits, lanes_h, st);
+    return launch_attn_step<2, 2, 4, false>(a, splits, lanes_h, st);
 }
 
 } // namespace vb

@@ -5,9 +5,9 @@
  *   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q        (per head, fp32)
  *   out = rmsnorm(o) * silu(gate)
  *
- *   lm_delta_inputs  convolution, unit norms, step sizes beta, log decays: 16 rows per CTA
- *   lm_delta_scan    the recurrence token by token; columns of S are independent, so a CTA owns 32
- *                    of a head's value columns, four lanes per column
+ *   lm_delta_inputs  convolution, unit norms, step sizes beta, decays: 16 rows per CTA
+ *   lm_delta_scan    the recurrence token by token, in fp32; columns of S are independent, so a CTA owns
+ *                    32 of a head's value columns, S in registers, a few lanes per column
  *   lm_delta_gate    head norm and gate of a row; saves the raw convolution inputs of the last rows
  *   lm_delta_step    one token in one launch: a cluster of CTAs per head, 32 value columns each
  *
@@ -46,7 +46,7 @@ __global__ void __launch_bounds__(kInThreads) lm_delta_inputs_kernel(const LmDel
             const int r = r0 + i / H, h = i % H;
             const int cb = ch + H * a.vdim;           /* columns: q, k, v, gate, b, a */
             a.beta[(size_t)r * H + h] = 1.0f / (1.0f + expf(-lm_sum(a.in, r, cb + h)));
-            a.ldecay[(size_t)r * H + h] = -__ldg(a.decay + h) * softplus(lm_sum(a.in, r, cb + H + h) + __ldg(a.dt_bias + h));
+            a.decays[(size_t)r * H + h] = expf(-__ldg(a.decay + h) * softplus(lm_sum(a.in, r, cb + H + h) + __ldg(a.dt_bias + h)));
         }
         return;
     }
@@ -90,73 +90,189 @@ __global__ void __launch_bounds__(kInThreads) lm_delta_inputs_kernel(const LmDel
 }
 
 /* ------------------------------------------------------------------ the recurrence, token by token */
-constexpr int kScThreads = 128, kScCols = 32, kScTok = 16;
+constexpr int kScCols = 32, kScTok = 16;
 
-/* grid = (value column tiles, heads). Lane rg of a column's four lanes holds rows 4 i + rg of S. */
-template <int NR>
-__global__ void __launch_bounds__(kScThreads) lm_delta_scan_kernel(const LmDelta a, int M) {
-    __shared__ float ks[kScTok][4 * NR], qs[kScTok][4 * NR], vs[kScTok][kScCols], bs[kScTok], gs[kScTok];
+/* two fp32 lanes per instruction */
+VB_DEVINL uint64_t f2_pack(float lo, float hi) {
+    uint64_t r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+VB_DEVINL float f2_sum(uint64_t v) {
+    float lo, hi;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+    return lo + hi;
+}
+VB_DEVINL uint64_t f2_fma(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+VB_DEVINL uint64_t f2_mul(uint64_t a, uint64_t b) {
+    uint64_t r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+VB_DEVINL void cp_async4(void *smem, const void *gmem) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(vb_smem_u32(smem)), "l"(gmem) : "memory");
+}
+VB_DEVINL void cp_async16(void *smem, const void *gmem) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(vb_smem_u32(smem)), "l"(gmem) : "memory");
+}
+
+/* One buffer of the scan's inputs: kScTok tokens of k, q (padded to DP rows), the CTA's columns of v, step
+ * sizes and decays. */
+template <int DP>
+struct ScanBuf {
+    float k[kScTok][DP], q[kScTok][DP], v[kScTok][kScCols], beta[kScTok], g[kScTok];
+};
+
+/* grid = (value column tiles, heads), LPC lanes per column, each with NR rows of S: groups of four
+ * rows, lane rg takes groups rg, rg + LPC, ... Per token the read-out of the token before and the
+ * prediction S^T k are taken from the same S, so that one pass and one round of shuffles serves
+ * both; the decay is applied to the prediction and, with the update, to S. The inputs of the next
+ * kScTok tokens are copied while the current ones are worked on. */
+template <int LPC, int NR>
+__global__ void __launch_bounds__(kScCols * LPC) lm_delta_scan_kernel(const LmDelta a, int M) {
+    constexpr int DP = LPC * NR, kThreads = kScCols * LPC, NG = NR / 4;
+    extern __shared__ __align__(16) unsigned char scan_smem[];
+    ScanBuf<DP> *buf = reinterpret_cast<ScanBuf<DP> *>(scan_smem);
     pdl_launch_dependents();
-    pdl_wait();
     const int tid = threadIdx.x, h = blockIdx.y, kv = h / (a.heads / a.kv_heads);
-    const int rg = tid & 3, cl = tid >> 2, c = blockIdx.x * kScCols + cl;
+    const int rg = tid % LPC, cl = tid / LPC, c0 = blockIdx.x * kScCols, c = c0 + cl;
     const bool live = c < a.vdim;
     const int nqk = a.kv_heads * a.dim, nv = a.heads * a.vdim;
-    float *S = lm_state(a.s, a.dyn) + (size_t)h * a.dim * a.vdim;
-    float s[NR];
-    const bool fresh = a.dyn->pos == 0;
-#pragma unroll
-    for (int i = 0; i < NR; i++) {
-        const int r = 4 * i + rg;
-        s[i] = (!fresh && live && r < a.dim) ? S[(size_t)r * a.vdim + c] : 0.0f;
-    }
-    for (int t0 = 0; t0 < M; t0 += kScTok) {
+    /* rows and columns beyond the sizes stay zero in both buffers */
+    for (int i = tid; i < (int)(2 * sizeof(ScanBuf<DP>) / 4); i += kThreads) reinterpret_cast<float *>(scan_smem)[i] = 0.0f;
+    pdl_wait();
+    __syncthreads();
+    auto request = [&](int t0, int b) {
         const int nt = M - t0 < kScTok ? M - t0 : kScTok;
-        __syncthreads();
-        for (int i = tid; i < nt * 4 * NR; i += kScThreads) {
-            const int t = i / (4 * NR), d = i % (4 * NR);
-            const size_t at = (size_t)(t0 + t) * nqk + kv * a.dim + d;
-            ks[t][d] = d < a.dim ? a.k[at] : 0.0f;
-            qs[t][d] = d < a.dim ? a.q[at] : 0.0f;
+        if ((a.dim & 3) == 0) {
+            const int per = a.dim / 4;
+            for (int i = tid; i < nt * per; i += kThreads) {
+                const int t = i / per, d = i % per * 4;
+                const size_t at = (size_t)(t0 + t) * nqk + kv * a.dim + d;
+                cp_async16(&buf[b].k[t][d], a.k + at);
+                cp_async16(&buf[b].q[t][d], a.q + at);
+            }
+        } else {
+            for (int i = tid; i < nt * a.dim; i += kThreads) {
+                const int t = i / a.dim, d = i % a.dim;
+                const size_t at = (size_t)(t0 + t) * nqk + kv * a.dim + d;
+                cp_async4(&buf[b].k[t][d], a.k + at);
+                cp_async4(&buf[b].q[t][d], a.q + at);
+            }
         }
-        for (int i = tid; i < nt * kScCols; i += kScThreads) {
-            const int t = i / kScCols, cc = blockIdx.x * kScCols + i % kScCols;
-            vs[t][i % kScCols] = cc < a.vdim ? a.v[(size_t)(t0 + t) * nv + h * a.vdim + cc] : 0.0f;
+        for (int i = tid; i < nt * kScCols; i += kThreads) {
+            const int t = i / kScCols, cc = i % kScCols;
+            if (c0 + cc < a.vdim) cp_async4(&buf[b].v[t][cc], a.v + (size_t)(t0 + t) * nv + h * a.vdim + c0 + cc);
         }
         if (tid < nt) {
-            bs[tid] = a.beta[(size_t)(t0 + tid) * a.heads + h];
-            gs[tid] = expf(a.ldecay[(size_t)(t0 + tid) * a.heads + h]);
+            cp_async4(&buf[b].beta[tid], a.beta + (size_t)(t0 + tid) * a.heads + h);
+            cp_async4(&buf[b].g[tid], a.decays + (size_t)(t0 + tid) * a.heads + h);
         }
-        __syncthreads();
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    request(0, 0);
+
+    float *S = lm_state(a.s, a.dyn) + (size_t)h * a.dim * a.vdim;
+    uint64_t s[NR / 2];
+    const bool fresh = a.dyn->pos == 0;
+#pragma unroll
+    for (int i = 0; i < NG; i++) {
+        float x[4];
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const int r = (i * LPC + rg) * 4 + j;
+            x[j] = (!fresh && live && r < a.dim) ? S[(size_t)r * a.vdim + c] : 0.0f;
+        }
+        s[2 * i] = f2_pack(x[0], x[1]);
+        s[2 * i + 1] = f2_pack(x[2], x[3]);
+    }
+    float *out = a.o + h * a.vdim + c;
+    uint64_t qp[NR / 2];                                  /* query of the token before */
+#pragma unroll
+    for (int i = 0; i < NR / 2; i++) qp[i] = 0;
+    auto dot_reduce = [&](float v) {
+#pragma unroll
+        for (int o = 1; o < LPC; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+        return v;
+    };
+    for (int t0 = 0, b = 0; t0 < M; t0 += kScTok, b ^= 1) {
+        const int nt = M - t0 < kScTok ? M - t0 : kScTok;
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();                                  /* this buffer is complete, the other one is free */
+        if (t0 + kScTok < M) request(t0 + kScTok, b ^ 1);
+#pragma unroll 1
         for (int t = 0; t < nt; t++) {
-            const float g = gs[t];
-            float e0 = 0.0f, e1 = 0.0f;
+            const float g = buf[b].g[t], beta = buf[b].beta[t], v = buf[b].v[t][cl];
+            uint64_t k[NR / 2];
 #pragma unroll
-            for (int i = 0; i < NR; i++) {
-                s[i] *= g;
-                if (i & 1) e1 = fmaf(s[i], ks[t][4 * i + rg], e1); else e0 = fmaf(s[i], ks[t][4 * i + rg], e0);
+            for (int i = 0; i < NG; i++) {
+                const ulonglong2 x = *reinterpret_cast<const ulonglong2 *>(&buf[b].k[t][(i * LPC + rg) * 4]);
+                k[2 * i] = x.x;
+                k[2 * i + 1] = x.y;
             }
-            float e = e0 + e1;
-            e += __shfl_xor_sync(0xffffffffu, e, 1);
-            e += __shfl_xor_sync(0xffffffffu, e, 2);
-            const float u = bs[t] * (vs[t][cl] - e);
-            float o0 = 0.0f, o1 = 0.0f;
+            uint64_t e0 = 0, e1 = 0, o0 = 0, o1 = 0;
 #pragma unroll
-            for (int i = 0; i < NR; i++) {
-                s[i] = fmaf(ks[t][4 * i + rg], u, s[i]);
-                if (i & 1) o1 = fmaf(s[i], qs[t][4 * i + rg], o1); else o0 = fmaf(s[i], qs[t][4 * i + rg], o0);
+            for (int i = 0; i < NR / 2; i += 2) {
+                e0 = f2_fma(s[i], k[i], e0);
+                e1 = f2_fma(s[i + 1], k[i + 1], e1);
+                o0 = f2_fma(s[i], qp[i], o0);
+                o1 = f2_fma(s[i + 1], qp[i + 1], o1);
             }
-            float o = o0 + o1;
-            o += __shfl_xor_sync(0xffffffffu, o, 1);
-            o += __shfl_xor_sync(0xffffffffu, o, 2);
-            if (rg == 0 && live) a.o[(size_t)(t0 + t) * nv + h * a.vdim + c] = o;
+            float e = f2_sum(e0) + f2_sum(e1), o = f2_sum(o0) + f2_sum(o1);
+#pragma unroll
+            for (int x = 1; x < LPC; x <<= 1) {
+                e += __shfl_xor_sync(0xffffffffu, e, x);
+                o += __shfl_xor_sync(0xffffffffu, o, x);
+            }
+            if (rg == 0 && live && t0 + t > 0) out[(size_t)(t0 + t - 1) * nv] = o;
+            const float u = beta * (v - g * e);
+            const uint64_t g2 = f2_pack(g, g), u2 = f2_pack(u, u);
+#pragma unroll
+            for (int i = 0; i < NR / 2; i++) s[i] = f2_fma(s[i], g2, f2_mul(k[i], u2));
+#pragma unroll
+            for (int i = 0; i < NG; i++) {
+                const ulonglong2 x = *reinterpret_cast<const ulonglong2 *>(&buf[b].q[t][(i * LPC + rg) * 4]);
+                qp[2 * i] = x.x;
+                qp[2 * i + 1] = x.y;
+            }
         }
     }
+    uint64_t o0 = 0, o1 = 0;
 #pragma unroll
-    for (int i = 0; i < NR; i++) {
-        const int r = 4 * i + rg;
-        if (live && r < a.dim) S[(size_t)r * a.vdim + c] = s[i];
+    for (int i = 0; i < NR / 2; i += 2) {
+        o0 = f2_fma(s[i], qp[i], o0);
+        o1 = f2_fma(s[i + 1], qp[i + 1], o1);
     }
+    const float o = dot_reduce(f2_sum(o0) + f2_sum(o1));
+    if (rg == 0 && live) out[(size_t)(M - 1) * nv] = o;
+#pragma unroll
+    for (int i = 0; i < NR / 2; i++) {
+        float x[2];
+        asm("mov.b64 {%0, %1}, %2;" : "=f"(x[0]), "=f"(x[1]) : "l"(s[i]));
+#pragma unroll
+        for (int j = 0; j < 2; j++) {
+            const int r = ((i / 2) * LPC + rg) * 4 + (i & 1) * 2 + j;
+            if (live && r < a.dim) S[(size_t)r * a.vdim + c] = x[j];
+        }
+    }
+}
+
+template <int LPC, int NR>
+int launch_scan(const LmDelta &a, int M, cudaStream_t st) {
+    constexpr size_t smem = 2 * sizeof(ScanBuf<LPC * NR>);
+    static bool attr = false;
+    if (!attr) {
+        if (cudaFuncSetAttribute(lm_delta_scan_kernel<LPC, NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+            cudaGetLastError();
+            return -1;
+        }
+        attr = true;
+    }
+    return ok(launch_pdl(lm_delta_scan_kernel<LPC, NR>, dim3((a.vdim + kScCols - 1) / kScCols, a.heads), dim3(kScCols * LPC), smem, st, a, M));
 }
 
 /* ------------------------------------------------------------------ head norm, gate, convolution memory */
@@ -327,11 +443,10 @@ int lm_delta_inputs(const LmDelta &a, int M, cudaStream_t st) {
 }
 
 int lm_delta_scan(const LmDelta &a, int M, cudaStream_t st) {
-    const dim3 g((a.vdim + kScCols - 1) / kScCols, a.heads), b(kScThreads);
-    if (a.dim <= 32) return ok(launch_pdl(lm_delta_scan_kernel<8>, g, b, 0, st, a, M));
-    if (a.dim <= 64) return ok(launch_pdl(lm_delta_scan_kernel<16>, g, b, 0, st, a, M));
-    if (a.dim <= 128) return ok(launch_pdl(lm_delta_scan_kernel<32>, g, b, 0, st, a, M));
-    if (a.dim <= 256) return ok(launch_pdl(lm_delta_scan_kernel<64>, g, b, 0, st, a, M));
+    if (a.dim <= 32) return launch_scan<4, 8>(a, M, st);
+    if (a.dim <= 64) return launch_scan<4, 16>(a, M, st);
+    if (a.dim <= 128) return launch_scan<4, 32>(a, M, st);
+    if (a.dim <= 256) return launch_scan<8, 32>(a, M, st);
     return -1;
 }
 

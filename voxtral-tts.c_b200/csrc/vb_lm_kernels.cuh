@@ -164,6 +164,8 @@ struct LmAttn {
     float eps;
     LmRing ring;
     LmState k, v;                /* [ring rows][kv_heads * dim], [..][kv_heads * vdim] */
+    int split;                   /* 1: a head's part of a cache row is [size] BF16 high halves, then [size] low halves
+                                    (hi + lo carry 16 mantissa bits), ready for the tensor cores; 0: fp32 */
     LmPart qkv;
     float *q;                    /* [M][heads * dim] normed and rotated */
     float *scratch;              /* key-split partials */
@@ -178,7 +180,7 @@ int lm_attn_prepare(const LmAttn &a, int M, cudaStream_t st);              /* no
 int lm_attn_generic(const LmAttn &a, int M, cudaStream_t st);              /* fp32 pipes, any size */
 bool lm_attn_step_ok(const LmAttn &a);
 int lm_attn_step(const LmAttn &a, cudaStream_t st);                        /* one token: norm, rotation, append, attention */
-bool lm_attn_mma_ok(const LmAttn &a);
+bool lm_attn_mma_ok(int dim, int vdim);                                    /* sizes it runs at; needs split caches */
 int lm_attn_mma(const LmAttn &a, int M, cudaStream_t st);                  /* warp-level tensor cores, prompts */
 
 /* ---- gated delta rule (vb_lm_delta.cu) ---- */
@@ -194,9 +196,8 @@ struct LmDelta {
     LmState tail;                /* [taps][channels] raw convolution inputs, position p in row p % taps */
     LmPart in;                   /* columns q, k, v, gate, b, a */
     float *q, *k, *v;            /* [M][kv_heads * dim], same, [M][heads * vdim] */
-    float *beta, *ldecay;        /* [M][heads]; log of the decay */
+    float *beta, *decays;        /* [M][heads] */
     float *o;                    /* [M][heads * vdim] */
-    float *chunk;                /* per-chunk matrices of the chunked form */
     LmSink out;
 };
 int lm_delta_channels(int heads, int kv_heads, int dim, int vdim);

@@ -41,6 +41,17 @@ VB_DEVINL void kv_put(float *head, int size, int d, float v, int split) {
         head[d] = v;
     }
 }
+VB_DEVINL void kv_put4(float *head, int size, int d, float4 v, int split) {
+    if (split) {
+        uint32_t h[4], l[4];
+        hilo(v.x, h[0], l[0]); hilo(v.y, h[1], l[1]); hilo(v.z, h[2], l[2]); hilo(v.w, h[3], l[3]);
+        uint16_t *p = reinterpret_cast<uint16_t *>(head);
+        *reinterpret_cast<uint2 *>(p + d) = make_uint2(h[0] | (h[1] << 16), h[2] | (h[3] << 16));
+        *reinterpret_cast<uint2 *>(p + size + d) = make_uint2(l[0] | (l[1] << 16), l[2] | (l[3] << 16));
+    } else {
+        *reinterpret_cast<float4 *>(head + d) = v;
+    }
+}
 VB_DEVINL float kv_get(const float *head, int size, int d, int split) {
     if (!split) return __ldcg(head + d);
     const unsigned short *h = reinterpret_cast<const unsigned short *>(head);
@@ -59,7 +70,7 @@ VB_DEVINL float4 kv_get4(const float *head, int size, int d) {
 constexpr int kPrepThreads = 512;
 
 __global__ void __launch_bounds__(kPrepThreads) lm_attn_prepare_kernel(const LmAttn a) {
-    extern __shared__ float prep_smem[];
+    extern __shared__ __align__(16) float prep_smem[];
     __shared__ float red[2][kPrepThreads / 32];
     const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim;
     float *buf = prep_smem;                       /* [nq + nk] */
@@ -80,13 +91,28 @@ __global__ void __launch_bounds__(kPrepThreads) lm_attn_prepare_kernel(const LmA
         cs[half + i] = (s + c * lo) * a.mag;
     }
     float sq = 0.0f, sk = 0.0f;
-    for (int c = tid; c < nq + nk; c += kPrepThreads) {
-        const float v = lm_sum(a.qkv, m, c);
-        buf[c] = v;
-        if (c < nq) sq += v * v; else sk += v * v;
-    }
     float *Vr = lm_state(a.v, a.dyn) + row * nv;
-    for (int c = tid; c < nv; c += kPrepThreads) kv_put(Vr + c / a.vdim * a.vdim, a.vdim, c % a.vdim, lm_sum(a.qkv, m, nq + nk + c), a.split);
+    if (((nq | nk | a.vdim) & 3) == 0) {
+        for (int c = tid * 4; c < nq + nk + nv; c += kPrepThreads * 4) {
+            const float4 v = lm_sum4(a.qkv, m, c);
+            if (c < nq + nk) {
+                const float ss = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+                *reinterpret_cast<float4 *>(buf + c) = v;
+                if (c < nq) sq += ss; else sk += ss;
+            } else {
+                const int j = c - nq - nk, d = j % a.vdim;
+                kv_put4(Vr + j - d, a.vdim, d, v, a.split);
+            }
+        }
+    } else {
+        for (int c = tid; c < nq + nk; c += kPrepThreads) {
+            const float v = lm_sum_batch(a.qkv, m, c);
+            buf[c] = v;
+            if (c < nq) sq += v * v; else sk += v * v;
+        }
+        for (int c = tid; c < nv; c += kPrepThreads)
+            kv_put(Vr + c / a.vdim * a.vdim, a.vdim, c % a.vdim, lm_sum_batch(a.qkv, m, nq + nk + c), a.split);
+    }
     sq = vb_warp_sum(sq);
     sk = vb_warp_sum(sk);
     if ((tid & 31) == 0) { red[0][tid >> 5] = sq; red[1][tid >> 5] = sk; }
@@ -96,7 +122,7 @@ __global__ void __launch_bounds__(kPrepThreads) lm_attn_prepare_kernel(const LmA
     for (int w = 0; w < kPrepThreads / 32; w++) { sq += red[0][w]; sk += red[1][w]; }
     const float rq = 1.0f / sqrtf(sq / (float)nq + a.eps), rk = 1.0f / sqrtf(sk / (float)nk + a.eps);
     float *Kr = lm_state(a.k, a.dyn) + row * nk, *Q = a.q + (size_t)m * nq;
-    for (int c = tid; c < nq + nk; c += kPrepThreads) {
+    auto value = [&](int c) {                     /* column c normed and rotated */
         const bool isq = c < nq;
         const int j = isq ? c : c - nq, d = j % a.dim;
         const float *gain = isq ? a.q_gain : a.k_gain;
@@ -107,8 +133,21 @@ __global__ void __launch_bounds__(kPrepThreads) lm_attn_prepare_kernel(const LmA
             const float u = buf[c + other] * r * __ldg(gain + j + other);
             v = d < half ? v * cs[i] - u * cs[half + i] : v * cs[i] + u * cs[half + i];
         }
-        if (isq) Q[j] = v;
-        else kv_put(Kr + j - d, a.dim, d, v, a.split);
+        return v;
+    };
+    if (((nq | nk | a.dim) & 3) == 0) {
+        for (int c = tid * 4; c < nq + nk; c += kPrepThreads * 4) {
+            const float4 v = make_float4(value(c), value(c + 1), value(c + 2), value(c + 3));
+            const int j = c < nq ? c : c - nq, d = j % a.dim;
+            if (c < nq) *reinterpret_cast<float4 *>(Q + j) = v;
+            else kv_put4(Kr + j - d, a.dim, d, v, a.split);
+        }
+    } else {
+        for (int c = tid; c < nq + nk; c += kPrepThreads) {
+            const int j = c < nq ? c : c - nq, d = j % a.dim;
+            if (c < nq) Q[j] = value(c);
+            else kv_put(Kr + j - d, a.dim, d, value(c), a.split);
+        }
     }
 }
 
@@ -371,22 +410,26 @@ __global__ void __launch_bounds__(kSaThreads) lm_attn_step_kernel(const LmAttn a
             const int d = i * 128 + lane * 4;
             q[i] = d < dim ? *reinterpret_cast<const float4 *>(qs + hh * dim + d) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
+        const int first = w0 > a.ring.keep ? (w0 - a.ring.keep) % a.ring.ring : 0;      /* ring place of the window's first key */
         for (int xb = x0 + sub; xb < x1; xb += KP * subs) {
+            /* every load of the pass is requested unconditionally (beyond the range: the last key again), so that
+             * they are all in flight together */
             float4 kk[KP][ND], vv[KP][NV];
 #pragma unroll
             for (int u = 0; u < KP; u++) {
-                const int x = xb + u * subs;
-                const bool in = x < x1;
-                const size_t row = in ? (size_t)lm_ring_row(a.ring, x < n_keep ? x : w0 + x - n_keep) : 0;
+                int x = xb + u * subs;
+                x = x < x1 ? x : x1 - 1;
+                int r = first + x - n_keep;
+                r = x < n_keep ? x : a.ring.keep + (r < a.ring.ring ? r : r - a.ring.ring);
 #pragma unroll
                 for (int i = 0; i < ND; i++) {
                     const int d = i * 128 + lane * 4;
-                    kk[u][i] = in && d < dim ? kv_get4<SPLIT>(Kc + row * nk, dim, d) : make_float4(0.f, 0.f, 0.f, 0.f);
+                    kk[u][i] = kv_get4<SPLIT>(Kc + (size_t)r * nk, dim, d < dim ? d : 0);
                 }
 #pragma unroll
                 for (int i = 0; i < NV; i++) {
                     const int d = i * 128 + lane * 4;
-                    vv[u][i] = in && d < vdim ? kv_get4<SPLIT>(Vc + row * nv, vdim, d) : make_float4(0.f, 0.f, 0.f, 0.f);
+                    vv[u][i] = kv_get4<SPLIT>(Vc + (size_t)r * nv, vdim, d < vdim ? d : 0);
                 }
             }
             float s[KP];

@@ -7,7 +7,7 @@
  *
  *   lm_delta_inputs  convolution, unit norms, step sizes beta, decays: 16 rows per CTA
  *   lm_delta_scan    the recurrence token by token, in fp32; columns of S are independent, so a CTA owns
- *                    32 of a head's value columns, S in registers, a few lanes per column
+ *                    16 of a head's value columns, S in registers, eight lanes per column
  *   lm_delta_gate    head norm and gate of a row; saves the raw convolution inputs of the last rows
  *   lm_delta_step    one token in one launch: a cluster of CTAs per head, 32 value columns each
  *
@@ -34,7 +34,7 @@ constexpr int kInThreads = 128, kInRows = 16;
 /* grid = (row tiles, 2 * kv_heads + heads + 1): one head of q, k or v per CTA; the last column of
  * CTAs works out step sizes and decays. */
 __global__ void __launch_bounds__(kInThreads) lm_delta_inputs_kernel(const LmDelta a, int M) {
-    extern __shared__ float in_smem[];
+    extern __shared__ __align__(16) float in_smem[];
     pdl_launch_dependents();
     pdl_wait();
     const int r0 = blockIdx.x * kInRows, rows = M - r0 < kInRows ? M - r0 : kInRows;
@@ -58,22 +58,45 @@ __global__ void __launch_bounds__(kInThreads) lm_delta_inputs_kernel(const LmDel
     float *raw = in_smem, *out = raw + (kInRows + past) * size;      /* [past + rows][size], [rows][size] */
     const int pos0 = a.dyn->pos;
     const float *tail = lm_state(a.tail, a.dyn);
-    for (int i = tid; i < (past + rows) * size; i += kInThreads) {
-        const int r = r0 - past + i / size, c = c0 + i % size;       /* row of this launch, may be an earlier token */
-        float v = 0.0f;
-        if (r >= 0) v = lm_sum(a.in, r, c);
-        else if (pos0 + r >= 0) v = tail[(size_t)((pos0 + r) % a.taps) * ch + c];
-        raw[i] = v;
+    auto past_row = [&](int r, int c) {          /* an earlier token's input, zero before the sequence's start */
+        return pos0 + r >= 0 ? tail[(size_t)((pos0 + r) % a.taps) * ch + c] : 0.0f;
+    };
+    if (((c0 | size) & 3) == 0) {
+        const int per = size / 4;
+        for (int i = tid; i < (past + rows) * per; i += kInThreads) {
+            const int r = r0 - past + i / per, d = i % per * 4, c = c0 + d;
+            *reinterpret_cast<float4 *>(raw + (i / per) * size + d) =
+                r >= 0 ? lm_sum4(a.in, r, c) : make_float4(past_row(r, c), past_row(r, c + 1), past_row(r, c + 2), past_row(r, c + 3));
+        }
+    } else {
+        for (int i = tid; i < (past + rows) * size; i += kInThreads) {
+            const int r = r0 - past + i / size, c = c0 + i % size;
+            raw[i] = r >= 0 ? lm_sum_batch(a.in, r, c) : past_row(r, c);
+        }
     }
     __syncthreads();
-    for (int i = tid; i < rows * size; i += kInThreads) {
-        const int r = i / size, d = i % size;
+    /* a thread keeps to its channels, so that their taps stay in registers */
+    constexpr int kRegTaps = 4;
+    for (int d = tid; d < size; d += kInThreads) {
         const float *w = a.conv + (size_t)(c0 + d) * a.taps;
-        float v = 0.0f;
-        for (int j = 0; j < a.taps; j++) v = fmaf(__ldg(w + j), raw[(r + j) * size + d], v);
-        v = silu(v);
-        if (kind == 2) a.v[(size_t)(r0 + r) * H * a.vdim + head * a.vdim + d] = v;
-        else out[i] = v;
+        float wr[kRegTaps];
+        if (a.taps <= kRegTaps) {
+#pragma unroll
+            for (int j = 0; j < kRegTaps; j++) wr[j] = j < a.taps ? __ldg(w + j) : 0.0f;
+        }
+        for (int r = 0; r < rows; r++) {
+            float v = 0.0f;
+            if (a.taps <= kRegTaps) {
+#pragma unroll
+                for (int j = 0; j < kRegTaps; j++)
+                    if (j < a.taps) v = fmaf(wr[j], raw[(r + j) * size + d], v);
+            } else {
+                for (int j = 0; j < a.taps; j++) v = fmaf(__ldg(w + j), raw[(r + j) * size + d], v);
+            }
+            v = silu(v);
+            if (kind == 2) a.v[(size_t)(r0 + r) * H * a.vdim + head * a.vdim + d] = v;
+            else out[r * size + d] = v;
+        }
     }
     if (kind == 2) return;
     __syncthreads();
@@ -90,7 +113,7 @@ __global__ void __launch_bounds__(kInThreads) lm_delta_inputs_kernel(const LmDel
 }
 
 /* ------------------------------------------------------------------ the recurrence, token by token */
-constexpr int kScCols = 32, kScTok = 16;
+constexpr int kScCols = 16, kScTok = 16;
 
 /* two fp32 lanes per instruction */
 VB_DEVINL uint64_t f2_pack(float lo, float hi) {
@@ -130,8 +153,10 @@ struct ScanBuf {
 /* grid = (value column tiles, heads), LPC lanes per column, each with NR rows of S: groups of four
  * rows, lane rg takes groups rg, rg + LPC, ... Per token the read-out of the token before and the
  * prediction S^T k are taken from the same S, so that one pass and one round of shuffles serves
- * both; the decay is applied to the prediction and, with the update, to S. The inputs of the next
- * kScTok tokens are copied while the current ones are worked on. */
+ * both. The registers hold S / scale, `scale` being the product of the decays since it was last
+ * folded in, so that a token's update is one multiply-add per element; it is folded in before it
+ * gets small enough to matter for the range. The inputs of the next kScTok tokens are copied while the
+ * current ones are worked on. */
 template <int LPC, int NR>
 __global__ void __launch_bounds__(kScCols * LPC) lm_delta_scan_kernel(const LmDelta a, int M) {
     constexpr int DP = LPC * NR, kThreads = kScCols * LPC, NG = NR / 4;
@@ -194,26 +219,34 @@ __global__ void __launch_bounds__(kScCols * LPC) lm_delta_scan_kernel(const LmDe
     uint64_t qp[NR / 2];                                  /* query of the token before */
 #pragma unroll
     for (int i = 0; i < NR / 2; i++) qp[i] = 0;
-    auto dot_reduce = [&](float v) {
+    float scale = 1.0f;
+    auto fold = [&]() {
+        const uint64_t f2 = f2_pack(scale, scale);
 #pragma unroll
-        for (int o = 1; o < LPC; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-        return v;
+        for (int i = 0; i < NR / 2; i++) s[i] = f2_mul(s[i], f2);
+        scale = 1.0f;
+    };
+    auto load = [&](uint64_t (&x)[NR / 2], const float *row) {
+#pragma unroll
+        for (int i = 0; i < NG; i++) {
+            const ulonglong2 y = *reinterpret_cast<const ulonglong2 *>(row + (i * LPC + rg) * 4);
+            x[2 * i] = y.x;
+            x[2 * i + 1] = y.y;
+        }
     };
     for (int t0 = 0, b = 0; t0 < M; t0 += kScTok, b ^= 1) {
         const int nt = M - t0 < kScTok ? M - t0 : kScTok;
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();                                  /* this buffer is complete, the other one is free */
         if (t0 + kScTok < M) request(t0 + kScTok, b ^ 1);
-#pragma unroll 1
+        uint64_t k[NR / 2], kn[NR / 2];
+        load(k, buf[b].k[0]);
+        float g = buf[b].g[0], beta = buf[b].beta[0], v = buf[b].v[0][cl];
+#pragma unroll 2
         for (int t = 0; t < nt; t++) {
-            const float g = buf[b].g[t], beta = buf[b].beta[t], v = buf[b].v[t][cl];
-            uint64_t k[NR / 2];
-#pragma unroll
-            for (int i = 0; i < NG; i++) {
-                const ulonglong2 x = *reinterpret_cast<const ulonglong2 *>(&buf[b].k[t][(i * LPC + rg) * 4]);
-                k[2 * i] = x.x;
-                k[2 * i + 1] = x.y;
-            }
+            const int tn = t + 1 < nt ? t + 1 : t;        /* the next token's inputs are on their way during this one */
+            load(kn, buf[b].k[tn]);
+            const float gn = buf[b].g[tn], betan = buf[b].beta[tn], vn = buf[b].v[tn][cl];
             uint64_t e0 = 0, e1 = 0, o0 = 0, o1 = 0;
 #pragma unroll
             for (int i = 0; i < NR / 2; i += 2) {
@@ -223,31 +256,44 @@ __global__ void __launch_bounds__(kScCols * LPC) lm_delta_scan_kernel(const LmDe
                 o1 = f2_fma(s[i + 1], qp[i + 1], o1);
             }
             float e = f2_sum(e0) + f2_sum(e1), o = f2_sum(o0) + f2_sum(o1);
+            load(qp, buf[b].q[t]);
 #pragma unroll
             for (int x = 1; x < LPC; x <<= 1) {
                 e += __shfl_xor_sync(0xffffffffu, e, x);
                 o += __shfl_xor_sync(0xffffffffu, o, x);
             }
-            if (rg == 0 && live && t0 + t > 0) out[(size_t)(t0 + t - 1) * nv] = o;
-            const float u = beta * (v - g * e);
-            const uint64_t g2 = f2_pack(g, g), u2 = f2_pack(u, u);
+            if (rg == 0 && live && t0 + t > 0) out[(size_t)(t0 + t - 1) * nv] = o * scale;
+            scale *= g;
+            const float inv = 1.0f / scale;               /* off the chain that goes through S */
+            if (scale < 0x1p-40f) {
+                /* (also a decay of zero, whose inverse is not used) */
+                const float before = scale;
+                fold();
+                const float u = beta * (v - before * e);
+                const uint64_t u2 = f2_pack(u, u);
 #pragma unroll
-            for (int i = 0; i < NR / 2; i++) s[i] = f2_fma(s[i], g2, f2_mul(k[i], u2));
+                for (int i = 0; i < NR / 2; i++) s[i] = f2_fma(k[i], u2, s[i]);
+            } else {
+                const float u = beta * (v - scale * e) * inv;
+                const uint64_t u2 = f2_pack(u, u);
 #pragma unroll
-            for (int i = 0; i < NG; i++) {
-                const ulonglong2 x = *reinterpret_cast<const ulonglong2 *>(&buf[b].q[t][(i * LPC + rg) * 4]);
-                qp[2 * i] = x.x;
-                qp[2 * i + 1] = x.y;
+                for (int i = 0; i < NR / 2; i++) s[i] = f2_fma(k[i], u2, s[i]);
             }
+#pragma unroll
+            for (int i = 0; i < NR / 2; i++) k[i] = kn[i];
+            g = gn; beta = betan; v = vn;
         }
     }
+    fold();
     uint64_t o0 = 0, o1 = 0;
 #pragma unroll
     for (int i = 0; i < NR / 2; i += 2) {
         o0 = f2_fma(s[i], qp[i], o0);
         o1 = f2_fma(s[i + 1], qp[i + 1], o1);
     }
-    const float o = dot_reduce(f2_sum(o0) + f2_sum(o1));
+    float o = f2_sum(o0) + f2_sum(o1);
+#pragma unroll
+    for (int x = 1; x < LPC; x <<= 1) o += __shfl_xor_sync(0xffffffffu, o, x);
     if (rg == 0 && live) out[(size_t)(M - 1) * nv] = o;
 #pragma unroll
     for (int i = 0; i < NR / 2; i++) {
@@ -300,14 +346,14 @@ __global__ void __launch_bounds__(kGtThreads) lm_delta_gate_kernel(const LmDelta
 }
 
 /* ------------------------------------------------------------------ one token */
-constexpr int kStThreads = 256, kStWarps = 8, kStCols = 32;
+constexpr int kStThreads = 512, kStWarps = 16, kStCols = 32, kStTaps = 4;
 
 /* grid = (value column slices, heads), the slices of a head form a cluster. Warp w holds rows
- * w, w + 8, ... of S, a lane one column. The memory row of the convolution that is written
+ * w, w + 16, ... of S, a lane one column. The memory row of the convolution that is written
  * (position p, row p % taps) is none of those that other CTAs read (p - 1 ... p - taps + 1). */
 template <int NR>
 __global__ void __launch_bounds__(kStThreads) lm_delta_step_kernel(const LmDelta a) {
-    __shared__ float qs[8 * NR], ks[8 * NR], vs[kStCols], red[2][kStWarps], part[2][kStWarps][kStCols], scal[2], ssq;
+    __shared__ float qs[kStWarps * NR], ks[kStWarps * NR], vs[kStCols], red[2][kStWarps], part[2][kStWarps][kStCols], scal[2], ssq;
     namespace cg = cooperative_groups;
     pdl_launch_dependents();
     pdl_wait();
@@ -323,7 +369,7 @@ __global__ void __launch_bounds__(kStThreads) lm_delta_step_kernel(const LmDelta
     float s[NR];
 #pragma unroll
     for (int i = 0; i < NR; i++) {
-        const int r = warp + 8 * i;
+        const int r = warp + kStWarps * i;
         s[i] = (pos > 0 && live && r < a.dim) ? __ldcg(S + (size_t)r * a.vdim + c) : 0.0f;
     }
     float gate = 0.0f;
@@ -341,9 +387,17 @@ __global__ void __launch_bounds__(kStThreads) lm_delta_step_kernel(const LmDelta
         const float raw = lm_sum_batch(a.in, 0, chan);
         const float *w = a.conv + (size_t)chan * a.taps;
         float v = 0.0f;
-        for (int j = 0; j < a.taps - 1; j++) {
-            const int p = pos - (a.taps - 1) + j;
-            if (p >= 0) v = fmaf(__ldg(w + j), __ldcg(tail + (size_t)(p % a.taps) * ch + chan), v);
+        for (int j0 = 0; j0 < a.taps - 1; j0 += kStTaps) {
+            float x[kStTaps], wj[kStTaps];              /* requested together, unconditionally */
+#pragma unroll
+            for (int u = 0; u < kStTaps; u++) {
+                const int j = j0 + u < a.taps - 1 ? j0 + u : j0, p = pos - (a.taps - 1) + j;
+                x[u] = __ldcg(tail + (size_t)((p + a.taps) % a.taps) * ch + chan);
+                wj[u] = __ldg(w + j);
+            }
+#pragma unroll
+            for (int u = 0; u < kStTaps; u++)
+                if (j0 + u < a.taps - 1 && pos - (a.taps - 1) + j0 + u >= 0) v = fmaf(wj[u], x[u], v);
         }
         v = silu(fmaf(__ldg(w + a.taps - 1), raw, v));
         if (kind == 2 || (blockIdx.x == 0 && h % group == 0)) tail[(size_t)(pos % a.taps) * ch + chan] = raw;
@@ -351,7 +405,7 @@ __global__ void __launch_bounds__(kStThreads) lm_delta_step_kernel(const LmDelta
         else if (kind == 1) { ks[i - a.dim] = v; sk += v * v; }
         else vs[i - 2 * a.dim] = v;
     }
-    for (int i = a.dim + tid; i < 8 * NR; i += kStThreads) qs[i] = ks[i] = 0.0f;
+    for (int i = a.dim + tid; i < kStWarps * NR; i += kStThreads) qs[i] = ks[i] = 0.0f;
     sq = vb_warp_sum(sq);
     sk = vb_warp_sum(sk);
     if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
@@ -365,7 +419,7 @@ __global__ void __launch_bounds__(kStThreads) lm_delta_step_kernel(const LmDelta
 #pragma unroll
     for (int i = 0; i < NR; i++) {
         s[i] *= g;
-        e = fmaf(s[i], ks[warp + 8 * i] * fk, e);
+        e = fmaf(s[i], ks[warp + kStWarps * i] * fk, e);
     }
     part[0][warp][lane] = e;
     __syncthreads();
@@ -376,13 +430,13 @@ __global__ void __launch_bounds__(kStThreads) lm_delta_step_kernel(const LmDelta
     float o = 0.0f;
 #pragma unroll
     for (int i = 0; i < NR; i++) {
-        s[i] = fmaf(ks[warp + 8 * i] * fk, u, s[i]);
-        o = fmaf(s[i], qs[warp + 8 * i] * fq, o);
+        s[i] = fmaf(ks[warp + kStWarps * i] * fk, u, s[i]);
+        o = fmaf(s[i], qs[warp + kStWarps * i] * fq, o);
     }
     part[1][warp][lane] = o;
 #pragma unroll
     for (int i = 0; i < NR; i++) {
-        const int r = warp + 8 * i;
+        const int r = warp + kStWarps * i;
         if (live && r < a.dim) S[(size_t)r * a.vdim + c] = s[i];
     }
     __syncthreads();
@@ -443,9 +497,9 @@ int lm_delta_inputs(const LmDelta &a, int M, cudaStream_t st) {
 }
 
 int lm_delta_scan(const LmDelta &a, int M, cudaStream_t st) {
-    if (a.dim <= 32) return launch_scan<4, 8>(a, M, st);
-    if (a.dim <= 64) return launch_scan<4, 16>(a, M, st);
-    if (a.dim <= 128) return launch_scan<4, 32>(a, M, st);
+    if (a.dim <= 32) return launch_scan<8, 4>(a, M, st);
+    if (a.dim <= 64) return launch_scan<8, 8>(a, M, st);
+    if (a.dim <= 128) return launch_scan<8, 16>(a, M, st);
     if (a.dim <= 256) return launch_scan<8, 32>(a, M, st);
     return -1;
 }
@@ -457,10 +511,9 @@ int lm_delta_gate(const LmDelta &a, int M, cudaStream_t st) {
 bool lm_delta_step_ok(const LmDelta &a) { return a.dim <= 256 && a.vdim <= 8 * kStCols; }
 
 int lm_delta_step(const LmDelta &a, cudaStream_t st) {
-    if (a.dim <= 32) return launch_step<4>(a, st);
-    if (a.dim <= 64) return launch_step<8>(a, st);
-    if (a.dim <= 128) return launch_step<16>(a, st);
-    return launch_step<32>(a, st);
+    if (a.dim <= 64) return launch_step<4>(a, st);
+    if (a.dim <= 128) return launch_step<8>(a, st);
+    return launch_step<16>(a, st);
 }
 
 } // namespace vb

@@ -440,36 +440,35 @@ __global__ void __launch_bounds__(kSaThreads) lm_attn_step_kernel(const LmAttn a
                 for (int i = 0; i < ND; i++)
                     s[u] += q[i].x * kk[u][i].x + q[i].y * kk[u][i].y + q[i].z * kk[u][i].z + q[i].w * kk[u][i].w;
             }
+            /* a lane ends up with the score of one of the pass's keys (32 / KP lanes share one) */
+            constexpr int kShare = 32 / KP;
+            vb_warp_multi_sum<KP>(s, lane);
+            float sc = s[0] * a.scale;
+            if (a.softcap > 0.0f) sc = a.softcap * tanhf(sc / a.softcap);
+            if (xb + (lane / kShare) * subs >= x1) sc = -INFINITY;
+            float top = sc;
 #pragma unroll
-            for (int off = 16; off > 0; off >>= 1)
-#pragma unroll
-                for (int u = 0; u < KP; u++) s[u] += __shfl_xor_sync(0xffffffffu, s[u], off);
-            float top = mx;
-#pragma unroll
-            for (int u = 0; u < KP; u++) {
-                s[u] *= a.scale;
-                if (a.softcap > 0.0f) s[u] = a.softcap * tanhf(s[u] / a.softcap);
-                if (xb + u * subs >= x1) s[u] = -INFINITY;
-                top = fmaxf(top, s[u]);
-            }
-            const float c = expf(mx - top);               /* the first key of a pass is always there: top is finite */
+            for (int off = kShare; off < 32; off <<= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, off));
+            top = fmaxf(top, mx);                         /* the first key of a pass is always there: finite */
+            const float c = expf(mx - top), w = expf(sc - top);
             mx = top;
-            den *= c;
+            den = den * c + w;                            /* this lane's key only; added up at the end */
 #pragma unroll
             for (int i = 0; i < NV; i++) { o[i][0] *= c; o[i][1] *= c; o[i][2] *= c; o[i][3] *= c; }
 #pragma unroll
             for (int u = 0; u < KP; u++) {
-                const float w = expf(s[u] - top);
-                den += w;
+                const float wu = __shfl_sync(0xffffffffu, w, u * kShare);
 #pragma unroll
                 for (int i = 0; i < NV; i++) {
-                    o[i][0] = fmaf(w, vv[u][i].x, o[i][0]);
-                    o[i][1] = fmaf(w, vv[u][i].y, o[i][1]);
-                    o[i][2] = fmaf(w, vv[u][i].z, o[i][2]);
-                    o[i][3] = fmaf(w, vv[u][i].w, o[i][3]);
+                    o[i][0] = fmaf(wu, vv[u][i].x, o[i][0]);
+                    o[i][1] = fmaf(wu, vv[u][i].y, o[i][1]);
+                    o[i][2] = fmaf(wu, vv[u][i].z, o[i][2]);
+                    o[i][3] = fmaf(wu, vv[u][i].w, o[i][3]);
                 }
             }
         }
+#pragma unroll
+        for (int off = 32 / KP; off < 32; off <<= 1) den += __shfl_xor_sync(0xffffffffu, den, off);
     }
 #pragma unroll
     for (int i = 0; i < NV; i++) {

@@ -131,6 +131,11 @@ VB_DEVINL uint64_t f2_fma(uint64_t a, uint64_t b, uint64_t c) {
     asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
     return r;
 }
+VB_DEVINL uint64_t f2_add(uint64_t a, uint64_t b) {
+    uint64_t r;
+    asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
 VB_DEVINL uint64_t f2_mul(uint64_t a, uint64_t b) {
     uint64_t r;
     asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
@@ -153,10 +158,8 @@ struct ScanBuf {
 /* grid = (value column tiles, heads), LPC lanes per column, each with NR rows of S: groups of four
  * rows, lane rg takes groups rg, rg + LPC, ... Per token the read-out of the token before and the
  * prediction S^T k are taken from the same S, so that one pass and one round of shuffles serves
- * both. The registers hold S / scale, `scale` being the product of the decays since it was last
- * folded in, so that a token's update is one multiply-add per element; it is folded in before it
- * gets small enough to matter for the range. The inputs of the next kScTok tokens are copied while the
- * current ones are worked on. */
+ * both; the decay is applied to the prediction and, while the sums travel, to S. The inputs of the
+ * next kScTok tokens are copied while the current ones are worked on. */
 template <int LPC, int NR>
 __global__ void __launch_bounds__(kScCols * LPC) lm_delta_scan_kernel(const LmDelta a, int M) {
     constexpr int DP = LPC * NR, kThreads = kScCols * LPC, NG = NR / 4;
@@ -219,13 +222,6 @@ __global__ void __launch_bounds__(kScCols * LPC) lm_delta_scan_kernel(const LmDe
     uint64_t qp[NR / 2];                                  /* query of the token before */
 #pragma unroll
     for (int i = 0; i < NR / 2; i++) qp[i] = 0;
-    float scale = 1.0f;
-    auto fold = [&]() {
-        const uint64_t f2 = f2_pack(scale, scale);
-#pragma unroll
-        for (int i = 0; i < NR / 2; i++) s[i] = f2_mul(s[i], f2);
-        scale = 1.0f;
-    };
     auto load = [&](uint64_t (&x)[NR / 2], const float *row) {
 #pragma unroll
         for (int i = 0; i < NG; i++) {
@@ -239,14 +235,12 @@ __global__ void __launch_bounds__(kScCols * LPC) lm_delta_scan_kernel(const LmDe
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();                                  /* this buffer is complete, the other one is free */
         if (t0 + kScTok < M) request(t0 + kScTok, b ^ 1);
-        uint64_t k[NR / 2], kn[NR / 2];
-        load(k, buf[b].k[0]);
-        float g = buf[b].g[0], beta = buf[b].beta[0], v = buf[b].v[0][cl];
+        const ScanBuf<DP> &in = buf[b];
+        uint64_t k[NR / 2];
+        load(k, in.k[0]);
+        float g = in.g[0], beta = in.beta[0], v = in.v[0][cl];
 #pragma unroll 2
         for (int t = 0; t < nt; t++) {
-            const int tn = t + 1 < nt ? t + 1 : t;        /* the next token's inputs are on their way during this one */
-            load(kn, buf[b].k[tn]);
-            const float gn = buf[b].g[tn], betan = buf[b].beta[tn], vn = buf[b].v[tn][cl];
             uint64_t e0 = 0, e1 = 0, o0 = 0, o1 = 0;
 #pragma unroll
             for (int i = 0; i < NR / 2; i += 2) {
@@ -255,36 +249,33 @@ __global__ void __launch_bounds__(kScCols * LPC) lm_delta_scan_kernel(const LmDe
                 o0 = f2_fma(s[i], qp[i], o0);
                 o1 = f2_fma(s[i + 1], qp[i + 1], o1);
             }
-            float e = f2_sum(e0) + f2_sum(e1), o = f2_sum(o0) + f2_sum(o1);
-            load(qp, buf[b].q[t]);
+            float e = f2_sum(f2_add(e0, e1)), o = f2_sum(f2_add(o0, o1));
+            /* independent of the reductions: the decayed S, the next token's inputs (the last one's again at the
+             * end), this token's query */
+            const int tn = t + 1 < nt ? t + 1 : t;
+            const uint64_t g2 = f2_pack(g, g);
+            const float bv = beta * v, bg = -beta * g;
+            uint64_t kn[NR / 2];
+            load(kn, in.k[tn]);
+            g = in.g[tn]; beta = in.beta[tn]; v = in.v[tn][cl];
+            load(qp, in.q[t]);
+#pragma unroll
+            for (int i = 0; i < NR / 2; i++) s[i] = f2_mul(s[i], g2);
 #pragma unroll
             for (int x = 1; x < LPC; x <<= 1) {
                 e += __shfl_xor_sync(0xffffffffu, e, x);
                 o += __shfl_xor_sync(0xffffffffu, o, x);
             }
-            if (rg == 0 && live && t0 + t > 0) out[(size_t)(t0 + t - 1) * nv] = o * scale;
-            scale *= g;
-            const float inv = 1.0f / scale;               /* off the chain that goes through S */
-            if (scale < 0x1p-40f) {
-                /* (also a decay of zero, whose inverse is not used) */
-                const float before = scale;
-                fold();
-                const float u = beta * (v - before * e);
-                const uint64_t u2 = f2_pack(u, u);
+            const float u = fmaf(bg, e, bv);              /* beta (v - g S^T k) */
+            const uint64_t u2 = f2_pack(u, u);
 #pragma unroll
-                for (int i = 0; i < NR / 2; i++) s[i] = f2_fma(k[i], u2, s[i]);
-            } else {
-                const float u = beta * (v - scale * e) * inv;
-                const uint64_t u2 = f2_pack(u, u);
-#pragma unroll
-                for (int i = 0; i < NR / 2; i++) s[i] = f2_fma(k[i], u2, s[i]);
+            for (int i = 0; i < NR / 2; i++) {
+                s[i] = f2_fma(k[i], u2, s[i]);
+                k[i] = kn[i];
             }
-#pragma unroll
-            for (int i = 0; i < NR / 2; i++) k[i] = kn[i];
-            g = gn; beta = betan; v = vn;
+            if (rg == 0 && live && t0 + t > 0) out[(size_t)(t0 + t - 1) * nv] = o;
         }
     }
-    fold();
     uint64_t o0 = 0, o1 = 0;
 #pragma unroll
     for (int i = 0; i < NR / 2; i += 2) {

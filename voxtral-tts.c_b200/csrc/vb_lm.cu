@@ -132,7 +132,7 @@ struct vb200_lm {
 
     /* activations */
     float *x = nullptr, *part_in = nullptr, *part_out = nullptr, *part_head = nullptr, *logits = nullptr;
-    float *q = nullptr, *k = nullptr, *v = nullptr, *o = nullptr, *beta = nullptr, *decays = nullptr;
+    float *q = nullptr, *k = nullptr, *v = nullptr, *o = nullptr, *beta = nullptr, *decays = nullptr, *gram = nullptr;
     float *scratch = nullptr, *tap = nullptr;
     unsigned *tickets = nullptr;
     int *status = nullptr, *log = nullptr, *zero = nullptr;
@@ -464,7 +464,7 @@ size_t vb200_lm::part_floats(const Linear &l, int max_rows) const {
 
 int vb200_lm::make_buffers() {
     const int W = cfg.width;
-    size_t in = 0, out = part_floats(loop_in, block), qn = 0, kn = 0, vn = 0, hn = 0, on = 0, scr = 0;
+    size_t in = 0, out = part_floats(loop_in, block), qn = 0, kn = 0, vn = 0, hn = 0, on = 0, gn = 0, scr = 0;
     int tick = 1;
     for (size_t i = 0; i < layers.size(); i++) {
         const LmMixer &m = cfg.layers[i].mixer;
@@ -476,6 +476,7 @@ int vb200_lm::make_buffers() {
             vn = std::max(vn, (size_t)m.heads * m.vdim);
             on = std::max(on, (size_t)m.heads * m.vdim);
             hn = std::max(hn, (size_t)m.heads);
+            gn = std::max(gn, (size_t)m.kv_heads);
         } else {
             qn = std::max(qn, (size_t)m.heads * m.dim);
             scr = std::max(scr, lm_attn_scratch_floats(m.heads, m.kv_heads, m.vdim));
@@ -485,7 +486,8 @@ int vb200_lm::make_buffers() {
     const size_t B = block;
     if (alloc(&x, B * W) || alloc(&part_in, in) || alloc(&part_out, out) || alloc(&part_head, part_floats(head, kHeadRows)) ||
         alloc(&logits, (size_t)kHeadRows * head.N) || alloc(&q, B * qn) || alloc(&k, B * kn) || alloc(&v, B * vn) || alloc(&o, B * on) ||
-        alloc(&beta, B * hn) || alloc(&decays, B * hn) || alloc(&scratch, scr) || alloc(&tickets, (size_t)tick, true) ||
+        alloc(&beta, B * hn) || alloc(&decays, B * hn) ||
+        alloc(&gram, (B + kLmDeltaRows) / kLmDeltaGroup * gn * 2 * kLmDeltaGroup * kLmDeltaGroup) || alloc(&scratch, scr) || alloc(&tickets, (size_t)tick, true) ||
         alloc(&status, 4, true) || alloc(&log, kLogCap, true) || alloc(&zero, 4, true) || alloc(&d_in, 4 + 2 * B, true))
         return -1;
     for (int i = 0; i < 2; i++) {
@@ -615,7 +617,7 @@ int vb200_lm::mixer(const Layer &l, const LmMixer &m, const RunState &s, int M) 
         d.eps = (float)cfg.eps;
         d.conv = l.mix.conv; d.decay = l.mix.decay; d.dt_bias = l.mix.dt_bias; d.norm = l.mix.norm;
         d.s = {slabs + s.a, slab}; d.tail = {slabs + s.b, slab};
-        d.in = in; d.q = q; d.k = k; d.v = v; d.beta = beta; d.decays = decays; d.o = o;
+        d.in = in; d.q = q; d.k = k; d.v = v; d.beta = beta; d.decays = decays; d.gram = gram; d.o = o; d.status = status;
         d.out = sink(l.mix.acts, M);
         if (M == 1 && lm_delta_step_ok(d)) {
             LM_DO(lm_delta_step(d, st));

@@ -5,9 +5,10 @@
  *   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q        (per head, fp32)
  *   out = rmsnorm(o) * silu(gate)
  *
- *   lm_delta_inputs  convolution, unit norms, step sizes beta, decays: 16 rows per CTA
- *   lm_delta_scan    the recurrence token by token, in fp32; columns of S are independent, so a CTA owns
- *                    16 of a head's value columns, S in registers, eight lanes per column
+ *   lm_delta_inputs  convolution, unit norms, step sizes beta, decays: 16 rows per CTA; inner products
+ *                    of the scan's groups
+ *   lm_delta_scan    the recurrence in fp32, four tokens at a time; columns of S are independent, so a CTA
+ *                    owns 16 of a head's value columns, S in registers, eight or more lanes per column
  *   lm_delta_gate    head norm and gate of a row; saves the raw convolution inputs of the last rows
  *   lm_delta_step    one token in one launch: a cluster of CTAs per head, 32 value columns each
  *
@@ -29,35 +30,14 @@ VB_DEVINL float silu(float z) { return z / (1.0f + expf(-z)); }
 VB_DEVINL float softplus(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 
 /* ------------------------------------------------------------------ inputs of the recurrence */
-constexpr int kInThreads = 128, kInRows = 16;
+constexpr int kScGroup = kLmDeltaGroup, kGramRow = 2 * kScGroup * kScGroup;
+constexpr int kInThreads = 128, kInRows = kLmDeltaRows;
 
-/* grid = (row tiles, 2 * kv_heads + heads + 1): one head of q, k or v per CTA; the last column of
- * CTAs works out step sizes and decays. */
-__global__ void __launch_bounds__(kInThreads) lm_delta_inputs_kernel(const LmDelta a, int M) {
-    extern __shared__ __align__(16) float in_smem[];
-    pdl_launch_dependents();
-    pdl_wait();
-    const int r0 = blockIdx.x * kInRows, rows = M - r0 < kInRows ? M - r0 : kInRows;
-    const int tid = threadIdx.x, G = a.kv_heads, H = a.heads;
-    const int nqk = G * a.dim, ch = 2 * nqk + H * a.vdim;
-    int unit = blockIdx.y;
-    if (unit == 2 * G + H) {
-        for (int i = tid; i < rows * H; i += kInThreads) {
-            const int r = r0 + i / H, h = i % H;
-            const int cb = ch + H * a.vdim;           /* columns: q, k, v, gate, b, a */
-            a.beta[(size_t)r * H + h] = 1.0f / (1.0f + expf(-lm_sum(a.in, r, cb + h)));
-            a.decays[(size_t)r * H + h] = expf(-__ldg(a.decay + h) * softplus(lm_sum(a.in, r, cb + H + h) + __ldg(a.dt_bias + h)));
-        }
-        return;
-    }
-    const int kind = unit < G ? 0 : unit < 2 * G ? 1 : 2;     /* q, k, v */
-    const int head = kind == 2 ? unit - 2 * G : unit % G;
-    const int size = kind == 2 ? a.vdim : a.dim;
-    const int c0 = kind == 2 ? 2 * nqk + head * a.vdim : kind * nqk + head * a.dim;   /* first channel */
-    const int past = a.taps - 1;
-    float *raw = in_smem, *out = raw + (kInRows + past) * size;      /* [past + rows][size], [rows][size] */
-    const int pos0 = a.dyn->pos;
-    const float *tail = lm_state(a.tail, a.dyn);
+/* Short convolution and silu of `size` channels from c0 on, rows [r0, r0 + rows): out[row][ld_out].
+ * `raw` is room for the inputs, earlier tokens included. */
+VB_DEVINL void conv_rows(const LmDelta &a, float *raw, float *out, int ld_out, int c0, int size, int r0, int rows, const float *tail,
+                         int ch, int pos0) {
+    const int tid = threadIdx.x, past = a.taps - 1;
     auto past_row = [&](int r, int c) {          /* an earlier token's input, zero before the sequence's start */
         return pos0 + r >= 0 ? tail[(size_t)((pos0 + r) % a.taps) * ch + c] : 0.0f;
     };
@@ -93,27 +73,74 @@ __global__ void __launch_bounds__(kInThreads) lm_delta_inputs_kernel(const LmDel
             } else {
                 for (int j = 0; j < a.taps; j++) v = fmaf(__ldg(w + j), raw[(r + j) * size + d], v);
             }
-            v = silu(v);
-            if (kind == 2) a.v[(size_t)(r0 + r) * H * a.vdim + head * a.vdim + d] = v;
-            else out[r * size + d] = v;
+            out[(size_t)r * ld_out + d] = silu(v);
         }
-    }
-    if (kind == 2) return;
-    __syncthreads();
-    const int warp = tid >> 5, lane = tid & 31;
-    float *dst = kind == 0 ? a.q : a.k;
-    const float post = kind == 0 ? 1.0f / sqrtf((float)a.dim) : 1.0f;
-    for (int r = warp; r < rows; r += kInThreads / 32) {
-        float s = 0.0f;
-        for (int d = lane; d < size; d += 32) s += out[r * size + d] * out[r * size + d];
-        s = vb_warp_sum(s);
-        const float f = 1.0f / sqrtf(s + 1e-6f) * post;
-        for (int d = lane; d < size; d += 32) dst[(size_t)(r0 + r) * nqk + head * a.dim + d] = out[r * size + d] * f;
     }
 }
 
-/* ------------------------------------------------------------------ the recurrence, token by token */
-constexpr int kScCols = 16, kScTok = 16;
+/* grid = (row tiles, kv_heads + heads + 1): q and k of a key head, v of a value head, or (last)
+ * step sizes and decays. The q and k CTAs also leave the inner products of the scan's groups. */
+__global__ void __launch_bounds__(kInThreads) lm_delta_inputs_kernel(const LmDelta a, int M) {
+    extern __shared__ __align__(16) float in_smem[];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int r0 = blockIdx.x * kInRows, rows = M - r0 < kInRows ? M - r0 : kInRows;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, G = a.kv_heads, H = a.heads;
+    const int nqk = G * a.dim, ch = 2 * nqk + H * a.vdim, unit = blockIdx.y;
+    if (unit == G + H) {
+        for (int i = tid; i < rows * H; i += kInThreads) {
+            const int r = r0 + i / H, h = i % H;
+            const int cb = ch + H * a.vdim;           /* columns: q, k, v, gate, b, a */
+            a.beta[(size_t)r * H + h] = 1.0f / (1.0f + expf(-lm_sum(a.in, r, cb + h)));
+            a.decays[(size_t)r * H + h] = expf(-__ldg(a.decay + h) * softplus(lm_sum(a.in, r, cb + H + h) + __ldg(a.dt_bias + h)));
+        }
+        return;
+    }
+    const int pos0 = a.dyn->pos;
+    const float *tail = lm_state(a.tail, a.dyn);
+    if (unit >= G) {
+        const int head = unit - G;
+        conv_rows(a, in_smem, a.v + (size_t)r0 * H * a.vdim + head * a.vdim, H * a.vdim, 2 * nqk + head * a.vdim, a.vdim, r0, rows, tail, ch,
+                  pos0);
+        return;
+    }
+    const int dim = a.dim;
+    float *qk = in_smem, *raw = qk + 2 * kInRows * dim;         /* [q, k][kInRows][dim], room for the raw rows */
+    for (int kind = 0; kind < 2; kind++) {
+        float *out = qk + kind * kInRows * dim, *dst = kind == 0 ? a.q : a.k;
+        conv_rows(a, raw, out, dim, kind * nqk + unit * dim, dim, r0, rows, tail, ch, pos0);
+        __syncthreads();
+        const float post = kind == 0 ? 1.0f / sqrtf((float)dim) : 1.0f;
+        for (int r = warp; r < kInRows; r += kInThreads / 32) {
+            float s = 0.0f;
+            if (r < rows)
+                for (int d = lane; d < dim; d += 32) s += out[r * dim + d] * out[r * dim + d];
+            s = vb_warp_sum(s);
+            const float f = 1.0f / sqrtf(s + 1e-6f) * post;
+            for (int d = lane; d < dim; d += 32) {
+                const float v = r < rows ? out[r * dim + d] * f : 0.0f;
+                out[r * dim + d] = v;
+                if (r < rows) dst[(size_t)(r0 + r) * nqk + unit * dim + d] = v;
+            }
+        }
+        __syncthreads();
+    }
+    /* inner products inside a group of kScGroup tokens: k_t . k_j and q_t . k_j */
+    const float *Q = qk, *K = qk + kInRows * dim;
+    for (int i = warp; i < kInRows / kScGroup * kGramRow; i += kInThreads / 32) {
+        const int j = i % kScGroup, t = i / kScGroup % kScGroup, isq = i / (kScGroup * kScGroup) % 2, grp = i / kGramRow;
+        float s = 0.0f;
+        if (j <= t) {
+            const float *x = (isq ? Q : K) + (grp * kScGroup + t) * dim, *y = K + (grp * kScGroup + j) * dim;
+            for (int d = lane; d < dim; d += 32) s = fmaf(x[d], y[d], s);
+        }
+        s = vb_warp_sum(s);
+        if (lane == 0) a.gram[((size_t)(r0 / kScGroup + grp) * G + unit) * kGramRow + isq * kScGroup * kScGroup + t * kScGroup + j] = s;
+    }
+}
+
+/* ------------------------------------------------------------------ the recurrence */
+constexpr int kScCols = 16, kScTok = 16, kScGroups = kScTok / kScGroup, kScBufs = 3;
 
 /* two fp32 lanes per instruction */
 VB_DEVINL uint64_t f2_pack(float lo, float hi) {
@@ -144,66 +171,158 @@ VB_DEVINL uint64_t f2_mul(uint64_t a, uint64_t b) {
 VB_DEVINL void cp_async4(void *smem, const void *gmem) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(vb_smem_u32(smem)), "l"(gmem) : "memory");
 }
-VB_DEVINL void cp_async16(void *smem, const void *gmem) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(vb_smem_u32(smem)), "l"(gmem) : "memory");
-}
 
-/* One buffer of the scan's inputs: kScTok tokens of k, q (padded to DP rows), the CTA's columns of v, step
- * sizes and decays. */
-template <int DP>
-struct ScanBuf {
-    float k[kScTok][DP], q[kScTok][DP], v[kScTok][kScCols], beta[kScTok], g[kScTok];
+/* Coefficients of one group of four tokens for one head. With c_t the product of the decays up to
+ * token t of the group, d_tj that of the tokens after j up to t, and S the state before the group,
+ *   u_t = beta_t v_t - beta_t c_t (S^T k_t) - sum_{j<t} beta_t d_tj (k_t . k_j) u_j
+ *   o_t = c_t (S^T q_t) + sum_{j<=t} d_tj (q_t . k_j) u_j
+ *   S  <- c_3 S + sum_j d_3j k_j u_j^T
+ * which is the recurrence, token for token, with the four predictions taken from one S. */
+struct __align__(16) ScanCoef {
+    float beta[4], e[4];        /* beta_t; -beta_t c_t */
+    float u[8];                 /* -beta_t d_tj (k_t . k_j) for (1,0) (2,0) (2,1) (3,0) (3,1) (3,2) */
+    float s[4];                 /* d_3j */
+    float o[4][4];              /* d_tj (q_t . k_j), zero for j > t */
+    float c[4];                 /* c_t */
 };
 
-/* grid = (value column tiles, heads), LPC lanes per column, each with NR rows of S: groups of four
- * rows, lane rg takes groups rg, rg + LPC, ... Per token the read-out of the token before and the
- * prediction S^T k are taken from the same S, so that one pass and one round of shuffles serves
- * both; the decay is applied to the prediction and, while the sums travel, to S. The inputs of the
- * next kScTok tokens are copied while the current ones are worked on. */
+/* One buffer of the scan's inputs: kScTok tokens of k, q (padded to DP rows), the CTA's columns of v, step
+ * sizes, decays and inner products, and the coefficients made of them. */
+template <int DP>
+struct __align__(16) ScanBuf {
+    float k[kScTok][DP], q[kScTok][DP], v[kScTok][kScCols], gram[kScGroups][kGramRow], beta[kScTok], g[kScTok];
+    ScanCoef coef[kScGroups];
+};
+
+/* grid = (value column tiles, heads). All warps but the last hold S: LPC lanes per column, each with
+ * NR rows in groups of four (lane rg takes groups rg, rg + LPC, ...). Four tokens at a time: their
+ * eight inner products with S (S^T k_t, S^T q_t) are independent and are summed over the lanes in
+ * one halving butterfly, the rest is scalars. The last warp copies the inputs of the next blocks
+ * of kScTok tokens (bulk copies where rows start on 16-byte boundaries) and works out their
+ * coefficients. */
 template <int LPC, int NR>
-__global__ void __launch_bounds__(kScCols * LPC) lm_delta_scan_kernel(const LmDelta a, int M) {
-    constexpr int DP = LPC * NR, kThreads = kScCols * LPC, NG = NR / 4;
+__global__ void __launch_bounds__(kScCols * LPC + 32) lm_delta_scan_kernel(const LmDelta a, int M) {
+    static_assert(kScGroup == 4 && LPC >= 8, "the butterfly spreads eight values over at least eight lanes");
+    constexpr int DP = LPC * NR, kCompute = kScCols * LPC, kThreads = kCompute + 32, NG = NR / 4;
     extern __shared__ __align__(16) unsigned char scan_smem[];
+    __shared__ uint64_t full[kScBufs];
+    __shared__ volatile int gave_up;
     ScanBuf<DP> *buf = reinterpret_cast<ScanBuf<DP> *>(scan_smem);
     pdl_launch_dependents();
-    const int tid = threadIdx.x, h = blockIdx.y, kv = h / (a.heads / a.kv_heads);
-    const int rg = tid % LPC, cl = tid / LPC, c0 = blockIdx.x * kScCols, c = c0 + cl;
-    const bool live = c < a.vdim;
-    const int nqk = a.kv_heads * a.dim, nv = a.heads * a.vdim;
-    /* rows and columns beyond the sizes stay zero in both buffers */
-    for (int i = tid; i < (int)(2 * sizeof(ScanBuf<DP>) / 4); i += kThreads) reinterpret_cast<float *>(scan_smem)[i] = 0.0f;
+    const int tid = threadIdx.x, lane = tid & 31, h = blockIdx.y, kv = h / (a.heads / a.kv_heads);
+    const int c0 = blockIdx.x * kScCols;
+    const int nqk = a.kv_heads * a.dim, nv = a.heads * a.vdim, n_blocks = (M + kScTok - 1) / kScTok;
+    const bool bulk = ((a.dim | a.vdim) & 3) == 0;
+    /* rows and columns beyond the sizes stay zero in every buffer */
+    for (int i = tid; i < (int)(kScBufs * sizeof(ScanBuf<DP>) / 4); i += kThreads) reinterpret_cast<float *>(scan_smem)[i] = 0.0f;
+    if (tid == 0) {
+        for (int i = 0; i < kScBufs; i++) vb_mbar_init(&full[i], 1);
+        gave_up = 0;
+        vb_mbar_init_fence();
+    }
+    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");      /* the zeros come before the copies */
     pdl_wait();
     __syncthreads();
-    auto request = [&](int t0, int b) {
-        const int nt = M - t0 < kScTok ? M - t0 : kScTok;
-        if ((a.dim & 3) == 0) {
-            const int per = a.dim / 4;
-            for (int i = tid; i < nt * per; i += kThreads) {
-                const int t = i / per, d = i % per * 4;
-                const size_t at = (size_t)(t0 + t) * nqk + kv * a.dim + d;
-                cp_async16(&buf[b].k[t][d], a.k + at);
-                cp_async16(&buf[b].q[t][d], a.q + at);
-            }
-        } else {
-            for (int i = tid; i < nt * a.dim; i += kThreads) {
-                const int t = i / a.dim, d = i % a.dim;
-                const size_t at = (size_t)(t0 + t) * nqk + kv * a.dim + d;
-                cp_async4(&buf[b].k[t][d], a.k + at);
-                cp_async4(&buf[b].q[t][d], a.q + at);
-            }
-        }
-        for (int i = tid; i < nt * kScCols; i += kThreads) {
-            const int t = i / kScCols, cc = i % kScCols;
-            if (c0 + cc < a.vdim) cp_async4(&buf[b].v[t][cc], a.v + (size_t)(t0 + t) * nv + h * a.vdim + c0 + cc);
-        }
-        if (tid < nt) {
-            cp_async4(&buf[b].beta[tid], a.beta + (size_t)(t0 + tid) * a.heads + h);
-            cp_async4(&buf[b].g[tid], a.decays + (size_t)(t0 + tid) * a.heads + h);
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    };
-    request(0, 0);
 
+    if (tid >= kCompute) {
+        /* ---- inputs and coefficients ---- */
+        const int cols = a.vdim - c0 < kScCols ? a.vdim - c0 : kScCols;
+        auto request = [&](int blk) {
+            if (blk < n_blocks && !gave_up) {
+                const int b = blk % kScBufs;
+                ScanBuf<DP> &d = buf[b];
+                const int t0 = blk * kScTok, nt = M - t0 < kScTok ? M - t0 : kScTok, groups = (nt + kScGroup - 1) / kScGroup;
+                const float *gram = a.gram + ((size_t)(t0 / kScGroup) * a.kv_heads + kv) * kGramRow;
+                if (lane < nt) {
+                    cp_async4(&d.beta[lane], a.beta + (size_t)(t0 + lane) * a.heads + h);
+                    cp_async4(&d.g[lane], a.decays + (size_t)(t0 + lane) * a.heads + h);
+                }
+                if (bulk) {
+                    if (lane == 0) vb_mbar_arrive_expect_tx(&full[b], (uint32_t)(4 * (nt * (2 * a.dim + cols) + groups * kGramRow)));
+                    __syncwarp();
+                    const int t = lane & 15;
+                    const size_t at = (size_t)(t0 + t) * nqk + kv * a.dim;
+                    if (t < nt) vb_bulk_g2s(lane < 16 ? d.k[t] : d.q[t], (lane < 16 ? a.k : a.q) + at, (uint32_t)a.dim * 4u, &full[b]);
+                    if (lane < nt) vb_bulk_g2s(d.v[lane], a.v + (size_t)(t0 + lane) * nv + h * a.vdim + c0, (uint32_t)cols * 4u, &full[b]);
+                    if (lane < groups) vb_bulk_g2s(d.gram[lane], gram + (size_t)lane * a.kv_heads * kGramRow, kGramRow * 4u, &full[b]);
+                } else {
+                    for (int t = 0; t < nt; t++) {
+                        const size_t at = (size_t)(t0 + t) * nqk + kv * a.dim;
+                        for (int i = lane; i < a.dim; i += 32) { cp_async4(&d.k[t][i], a.k + at + i); cp_async4(&d.q[t][i], a.q + at + i); }
+                        if (lane < cols) cp_async4(&d.v[t][lane], a.v + (size_t)(t0 + t) * nv + h * a.vdim + c0 + lane);
+                    }
+                    for (int i = lane; i < groups * kGramRow; i += 32)
+                        cp_async4(&d.gram[i / kGramRow][i % kGramRow], gram + (size_t)(i / kGramRow) * a.kv_heads * kGramRow + i % kGramRow);
+                }
+            }
+            asm volatile("cp.async.commit_group;" ::: "memory");
+        };
+        auto arrived = [&](int blk) {                     /* everything requested for block blk has landed */
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+            if (bulk && blk < n_blocks && !vb_mbar_wait(&full[blk % kScBufs], (uint32_t)(blk / kScBufs) & 1u, &gave_up)) {
+                atomicCAS(a.status, 0, 51);
+                gave_up = 1;
+            }
+            __syncwarp();
+        };
+        auto coefficients = [&](int blk) {                /* one lane per group; tokens beyond the end change nothing */
+            if (blk >= n_blocks || lane >= kScGroups) return;
+            ScanBuf<DP> &d = buf[blk % kScBufs];
+            const int nt = M - blk * kScTok, tg = lane * kScGroup;
+            ScanCoef &x = d.coef[lane];
+            float g[4], b[4], c = 1.0f;
+#pragma unroll
+            for (int t = 0; t < 4; t++) {
+                g[t] = tg + t < nt ? d.g[tg + t] : 1.0f;
+                b[t] = tg + t < nt ? d.beta[tg + t] : 0.0f;
+            }
+            int n = 0;
+#pragma unroll
+            for (int t = 0; t < 4; t++) {
+                c *= g[t];
+                x.beta[t] = b[t];
+                x.e[t] = -b[t] * c;
+                x.c[t] = c;
+                float dt[4] = {0.0f, 0.0f, 0.0f, 0.0f}, p = 1.0f;
+#pragma unroll
+                for (int j = 3; j >= 0; j--) {
+                    if (j > t) { x.o[t][j] = 0.0f; continue; }
+                    dt[j] = p;
+                    x.o[t][j] = tg + t < nt ? p * d.gram[lane][kScGroup * kScGroup + t * 4 + j] : 0.0f;
+                    if (t == 3) x.s[j] = p;
+                    p *= g[j];
+                }
+#pragma unroll
+                for (int j = 0; j < t; j++) x.u[n++] = tg + t < nt ? -b[t] * dt[j] * d.gram[lane][t * 4 + j] : 0.0f;
+            }
+        };
+        auto clear_tail = [&](int blk) {                  /* tokens beyond the end: no stale k, q, v in a used group */
+            if (blk != n_blocks - 1) return;
+            ScanBuf<DP> &d = buf[blk % kScBufs];
+            const int nt = M - blk * kScTok, ne = (nt + kScGroup - 1) / kScGroup * kScGroup;
+            for (int t = nt; t < ne; t++) {
+                for (int i = lane; i < DP; i += 32) d.k[t][i] = d.q[t][i] = 0.0f;
+                if (lane < kScCols) d.v[t][lane] = 0.0f;
+            }
+        };
+        request(0);
+        request(1);
+        arrived(0);
+        coefficients(0);
+        clear_tail(0);
+        __syncthreads();                                  /* block 0 is ready */
+        for (int blk = 0; blk < n_blocks; blk++) {
+            request(blk + 2);
+            arrived(blk + 1);
+            coefficients(blk + 1);
+            clear_tail(blk + 1);
+            __syncthreads();                              /* block blk is done with, blk + 1 is ready */
+        }
+        return;
+    }
+
+    const int rg = tid % LPC, cl = tid / LPC, c = c0 + cl;
+    const bool live = c < a.vdim;
     float *S = lm_state(a.s, a.dyn) + (size_t)h * a.dim * a.vdim;
     uint64_t s[NR / 2];
     const bool fresh = a.dyn->pos == 0;
@@ -218,10 +337,6 @@ __global__ void __launch_bounds__(kScCols * LPC) lm_delta_scan_kernel(const LmDe
         s[2 * i] = f2_pack(x[0], x[1]);
         s[2 * i + 1] = f2_pack(x[2], x[3]);
     }
-    float *out = a.o + h * a.vdim + c;
-    uint64_t qp[NR / 2];                                  /* query of the token before */
-#pragma unroll
-    for (int i = 0; i < NR / 2; i++) qp[i] = 0;
     auto load = [&](uint64_t (&x)[NR / 2], const float *row) {
 #pragma unroll
         for (int i = 0; i < NG; i++) {
@@ -230,62 +345,75 @@ __global__ void __launch_bounds__(kScCols * LPC) lm_delta_scan_kernel(const LmDe
             x[2 * i + 1] = y.y;
         }
     };
-    for (int t0 = 0, b = 0; t0 < M; t0 += kScTok, b ^= 1) {
-        const int nt = M - t0 < kScTok ? M - t0 : kScTok;
-        asm volatile("cp.async.wait_group 0;" ::: "memory");
-        __syncthreads();                                  /* this buffer is complete, the other one is free */
-        if (t0 + kScTok < M) request(t0 + kScTok, b ^ 1);
-        const ScanBuf<DP> &in = buf[b];
-        uint64_t k[NR / 2];
-        load(k, in.k[0]);
-        float g = in.g[0], beta = in.beta[0], v = in.v[0][cl];
-#pragma unroll 2
-        for (int t = 0; t < nt; t++) {
-            uint64_t e0 = 0, e1 = 0, o0 = 0, o1 = 0;
+    auto dot = [&](const uint64_t (&x)[NR / 2]) {
+        uint64_t e0 = 0, e1 = 0;
 #pragma unroll
-            for (int i = 0; i < NR / 2; i += 2) {
-                e0 = f2_fma(s[i], k[i], e0);
-                e1 = f2_fma(s[i + 1], k[i + 1], e1);
-                o0 = f2_fma(s[i], qp[i], o0);
-                o1 = f2_fma(s[i + 1], qp[i + 1], o1);
-            }
-            float e = f2_sum(f2_add(e0, e1)), o = f2_sum(f2_add(o0, o1));
-            /* independent of the reductions: the decayed S, the next token's inputs (the last one's again at the
-             * end), this token's query */
-            const int tn = t + 1 < nt ? t + 1 : t;
-            const uint64_t g2 = f2_pack(g, g);
-            const float bv = beta * v, bg = -beta * g;
-            uint64_t kn[NR / 2];
-            load(kn, in.k[tn]);
-            g = in.g[tn]; beta = in.beta[tn]; v = in.v[tn][cl];
-            load(qp, in.q[t]);
-#pragma unroll
-            for (int i = 0; i < NR / 2; i++) s[i] = f2_mul(s[i], g2);
-#pragma unroll
-            for (int x = 1; x < LPC; x <<= 1) {
-                e += __shfl_xor_sync(0xffffffffu, e, x);
-                o += __shfl_xor_sync(0xffffffffu, o, x);
-            }
-            const float u = fmaf(bg, e, bv);              /* beta (v - g S^T k) */
-            const uint64_t u2 = f2_pack(u, u);
-#pragma unroll
-            for (int i = 0; i < NR / 2; i++) {
-                s[i] = f2_fma(k[i], u2, s[i]);
-                k[i] = kn[i];
-            }
-            if (rg == 0 && live && t0 + t > 0) out[(size_t)(t0 + t - 1) * nv] = o;
+        for (int i = 0; i < NR / 2; i += 2) {
+            e0 = f2_fma(s[i], x[i], e0);
+            e1 = f2_fma(s[i + 1], x[i + 1], e1);
         }
-    }
-    uint64_t o0 = 0, o1 = 0;
+        return f2_sum(f2_add(e0, e1));
+    };
+    /* after the butterfly lane rg holds value rg / (LPC / 8): 0 .. 3 are S^T k_t, 4 .. 7 are S^T q_t */
+    constexpr int kShare = LPC / 8;
+    const int mine = rg / kShare, lane0 = lane & ~(LPC - 1), ot = mine & 3;
+    const bool writes = live && mine >= 4 && rg % kShare == 0;
+    float *out = a.o + h * a.vdim + c;
+    __syncthreads();                                      /* block 0 is ready */
+    for (int blk = 0; blk < n_blocks; blk++) {
+        const ScanBuf<DP> &in = buf[blk % kScBufs];
+        const int t0 = blk * kScTok, nt = M - t0 < kScTok ? M - t0 : kScTok;
+        /* already complete: taken here too, so that this thread sees what the copies wrote */
+        if (bulk && !vb_mbar_wait(&full[blk % kScBufs], (uint32_t)(blk / kScBufs) & 1u, &gave_up)) gave_up = 1;
+        __syncwarp();
+#pragma unroll 1
+        for (int tg = 0; tg < nt; tg += kScGroup) {
+            const ScanCoef &x = in.coef[tg / kScGroup];
+            uint64_t k[4][NR / 2];
+            float y[8];
 #pragma unroll
-    for (int i = 0; i < NR / 2; i += 2) {
-        o0 = f2_fma(s[i], qp[i], o0);
-        o1 = f2_fma(s[i + 1], qp[i + 1], o1);
-    }
-    float o = f2_sum(o0) + f2_sum(o1);
+            for (int t = 0; t < 4; t++) {
+                uint64_t qt[NR / 2];
+                load(k[t], in.k[tg + t]);
+                load(qt, in.q[tg + t]);
+                y[t] = dot(k[t]);
+                y[4 + t] = dot(qt);
+            }
+            const float4 beta = *reinterpret_cast<const float4 *>(x.beta), ec = *reinterpret_cast<const float4 *>(x.e),
+                         u0 = *reinterpret_cast<const float4 *>(x.u), u1 = *reinterpret_cast<const float4 *>(x.u + 4),
+                         sc = *reinterpret_cast<const float4 *>(x.s), oc = *reinterpret_cast<const float4 *>(x.o[ot]);
+            const float oe = x.c[ot], c3 = x.c[3];
+            const float v0 = beta.x * in.v[tg][cl], v1 = beta.y * in.v[tg + 1][cl], v2 = beta.z * in.v[tg + 2][cl], v3 = beta.w * in.v[tg + 3][cl];
+            /* eight sums over the LPC lanes */
 #pragma unroll
-    for (int x = 1; x < LPC; x <<= 1) o += __shfl_xor_sync(0xffffffffu, o, x);
-    if (rg == 0 && live) out[(size_t)(M - 1) * nv] = o;
+            for (int n = 4, off = LPC / 2; n >= 1; n >>= 1, off >>= 1) {
+                const bool up = (rg & off) != 0;
+#pragma unroll
+                for (int i = 0; i < n; i++) {
+                    const float send = up ? y[i] : y[i + n], keep = up ? y[i + n] : y[i];
+                    y[i] = keep + __shfl_xor_sync(0xffffffffu, send, off);
+                }
+            }
+#pragma unroll
+            for (int off = kShare / 2; off >= 1; off >>= 1) y[0] += __shfl_xor_sync(0xffffffffu, y[0], off);
+            const float e0 = __shfl_sync(0xffffffffu, y[0], lane0), e1 = __shfl_sync(0xffffffffu, y[0], lane0 + kShare),
+                        e2 = __shfl_sync(0xffffffffu, y[0], lane0 + 2 * kShare), e3 = __shfl_sync(0xffffffffu, y[0], lane0 + 3 * kShare);
+            const uint64_t cc = f2_pack(c3, c3);
+#pragma unroll
+            for (int i = 0; i < NR / 2; i++) s[i] = f2_mul(s[i], cc);
+            const float w0 = fmaf(ec.x, e0, v0);
+            const float w1 = fmaf(u0.x, w0, fmaf(ec.y, e1, v1));
+            const float w2 = fmaf(u0.z, w1, fmaf(u0.y, w0, fmaf(ec.z, e2, v2)));
+            const float w3 = fmaf(u1.y, w2, fmaf(u1.x, w1, fmaf(u0.w, w0, fmaf(ec.w, e3, v3))));
+            const uint64_t d0 = f2_pack(sc.x * w0, sc.x * w0), d1 = f2_pack(sc.y * w1, sc.y * w1), d2 = f2_pack(sc.z * w2, sc.z * w2),
+                           d3 = f2_pack(sc.w * w3, sc.w * w3);
+#pragma unroll
+            for (int i = 0; i < NR / 2; i++) s[i] = f2_fma(k[3][i], d3, f2_fma(k[2][i], d2, f2_fma(k[1][i], d1, f2_fma(k[0][i], d0, s[i]))));
+            const float o = fmaf(oc.w, w3, fmaf(oc.z, w2, fmaf(oc.y, w1, fmaf(oc.x, w0, oe * y[0]))));
+            if (writes && tg + ot < nt) out[(size_t)(t0 + tg + ot) * nv] = o;
+        }
+        __syncthreads();                                  /* block blk is done with, blk + 1 is ready */
+    }
 #pragma unroll
     for (int i = 0; i < NR / 2; i++) {
         float x[2];
@@ -300,7 +428,8 @@ __global__ void __launch_bounds__(kScCols * LPC) lm_delta_scan_kernel(const LmDe
 
 template <int LPC, int NR>
 int launch_scan(const LmDelta &a, int M, cudaStream_t st) {
-    constexpr size_t smem = 2 * sizeof(ScanBuf<LPC * NR>);
+    constexpr size_t smem = kScBufs * sizeof(ScanBuf<LPC * NR>);
+    static_assert(smem <= 220 * 1024, "over what a CTA may use");
     static bool attr = false;
     if (!attr) {
         if (cudaFuncSetAttribute(lm_delta_scan_kernel<LPC, NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
@@ -309,7 +438,10 @@ int launch_scan(const LmDelta &a, int M, cudaStream_t st) {
         }
         attr = true;
     }
-    return ok(launch_pdl(lm_delta_scan_kernel<LPC, NR>, dim3((a.vdim + kScCols - 1) / kScCols, a.heads), dim3(kScCols * LPC), smem, st, a, M));
+    /* A plain launch: started early, under the tail of the kernel before it, the CTAs would crowd onto the first
+     * SMs that have room, and this kernel's time is that of its most crowded SM. */
+    lm_delta_scan_kernel<LPC, NR><<<dim3((a.vdim + kScCols - 1) / kScCols, a.heads), kScCols * LPC + 32, smem, st>>>(a, M);
+    return ok(cudaGetLastError());
 }
 
 /* ------------------------------------------------------------------ head norm, gate, convolution memory */
@@ -472,8 +604,8 @@ int lm_delta_channels(int heads, int kv_heads, int dim, int vdim) { return 2 * k
 bool lm_delta_supported(int dim, int vdim) { return dim >= 1 && dim <= 256 && vdim >= 1; }
 
 int lm_delta_inputs(const LmDelta &a, int M, cudaStream_t st) {
-    const int size = a.dim > a.vdim ? a.dim : a.vdim;
-    const size_t smem = sizeof(float) * (size_t)(2 * kInRows + a.taps - 1) * size;
+    const size_t raw = kInRows + a.taps - 1, qk = (raw + 2 * kInRows) * a.dim, v = raw * a.vdim;
+    const size_t smem = sizeof(float) * (qk > v ? qk : v);
     if (smem > 200 * 1024) return -1;
     static size_t set = 48 * 1024;
     if (smem > set) {
@@ -483,7 +615,7 @@ int lm_delta_inputs(const LmDelta &a, int M, cudaStream_t st) {
         }
         set = smem;
     }
-    return ok(launch_pdl(lm_delta_inputs_kernel, dim3((M + kInRows - 1) / kInRows, 2 * a.kv_heads + a.heads + 1), dim3(kInThreads), smem,
+    return ok(launch_pdl(lm_delta_inputs_kernel, dim3((M + kInRows - 1) / kInRows, a.kv_heads + a.heads + 1), dim3(kInThreads), smem,
                          st, a, M));
 }
 
@@ -491,7 +623,7 @@ int lm_delta_scan(const LmDelta &a, int M, cudaStream_t st) {
     if (a.dim <= 32) return launch_scan<8, 4>(a, M, st);
     if (a.dim <= 64) return launch_scan<8, 8>(a, M, st);
     if (a.dim <= 128) return launch_scan<8, 16>(a, M, st);
-    if (a.dim <= 256) return launch_scan<8, 32>(a, M, st);
+    if (a.dim <= 256) return launch_scan<16, 16>(a, M, st);
     return -1;
 }
 

@@ -197,12 +197,16 @@ struct LmDelta {
     LmPart in;                   /* columns q, k, v, gate, b, a */
     float *q, *k, *v;            /* [M][kv_heads * dim], same, [M][heads * vdim] */
     float *beta, *decays;        /* [M][heads] */
+    float *gram;                 /* [groups][kv_heads][k_t.k_j, q_t.k_j][t][j]: inner products inside groups of tokens */
+    int *status;                 /* set non-zero when a bounded wait runs out */
     float *o;                    /* [M][heads * vdim] */
     LmSink out;
 };
+constexpr int kLmDeltaGroup = 4;         /* tokens per group of the scan */
+constexpr int kLmDeltaRows = 16;         /* rows are prepared in multiples of this */
 int lm_delta_channels(int heads, int kv_heads, int dim, int vdim);
 int lm_delta_inputs(const LmDelta &a, int M, cudaStream_t st);             /* convolution, unit norms, step sizes, decays */
-int lm_delta_scan(const LmDelta &a, int M, cudaStream_t st);               /* token by token, fp32 pipes */
+int lm_delta_scan(const LmDelta &a, int M, cudaStream_t st);               /* the recurrence, fp32 pipes */
 int lm_delta_gate(const LmDelta &a, int M, cudaStream_t st);               /* head norm, gate; saves the convolution's tail */
 bool lm_delta_step_ok(const LmDelta &a);
 int lm_delta_step(const LmDelta &a, cudaStream_t st);                      /* one token: all of the above in one launch */

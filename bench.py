@@ -481,10 +481,6 @@ def lm_bench(args):
     speech decoder at equal size. Device time (CUDA events); the weights of a step exceed L2 many times.
     `--lm-only NAME` with `--m` prompt tokens and `--reps` new tokens runs one of them alone (profiling)."""
     pkg = load_package()
-    from importlib import util
-    spec = util.spec_from_file_location("vb200_lm_binding", os.path.join(ROOT, "voxtral-tts.c_b200", "lm.py"))
-    lm_mod = util.module_from_spec(spec)
-    spec.loader.exec_module(lm_mod)
     peak, src = measured_hbm_peak()
     rng = np.random.default_rng(0)
     configs = lm_configs()
@@ -493,7 +489,7 @@ def lm_bench(args):
         if args.lm_layers:
             c["layers"] = c["layers"][:args.lm_layers]
             c.pop("loop", None)
-        with lm_mod.LanguageModel(config=c, max_tokens=args.m + args.reps + 8) as lm:
+        with pkg.LanguageModel(config=c, max_tokens=args.m + args.reps + 8) as lm:
             for _ in range(2):
                 s = lm.open()
                 lm.generate(s, rng.integers(0, c["vocab"], args.m), max(args.reps, 1))
@@ -507,7 +503,7 @@ def lm_bench(args):
     time.sleep(1.5)
     sampler.begin()
     for name, c in configs.items():
-        with lm_mod.LanguageModel(config=c, max_tokens=8192) as lm:
+        with pkg.LanguageModel(config=c, max_tokens=8192) as lm:
             m = {"runs": lm.info.runs, "weight_bytes": lm.info.weight_bytes, "state_bytes": lm.info.state_bytes_per_seq, "prefill": []}
             embed = c["vocab"] * c["width"] * 2
             layers = lm.info.weight_bytes - 2 * embed

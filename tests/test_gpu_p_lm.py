@@ -1,6 +1,5 @@
 """Decoder language models on the GPU against the plain statement of the design (lm_plain.py), through
 the library's own step function, slots and generation loop."""
-import importlib.util
 import json
 import os
 import subprocess
@@ -20,11 +19,7 @@ DTYPES = ("float32", "bfloat16")
 
 @pytest.fixture(scope="module")
 def lm_mod(pkg):
-    from conftest import PKG_DIR
-    spec = importlib.util.spec_from_file_location("vb200_lm_binding", os.path.join(PKG_DIR, "lm.py"))
-    mod = importlib.util.module_from_spec(spec)
-    spec.loader.exec_module(mod)
-    return mod
+    return pkg
 
 
 class Case:

@@ -1,7 +1,6 @@
 """Decoder language models, host side: configuration reader and registry (no GPU needed), and the plain
 statement's own consistency."""
 import copy
-import importlib.util
 import json
 import os
 
@@ -14,11 +13,7 @@ from lm_models import as_float, attention, config, delta, tokens, weights, write
 
 @pytest.fixture(scope="module")
 def lm_mod(pkg):
-    from conftest import PKG_DIR
-    spec = importlib.util.spec_from_file_location("vb200_lm_binding", os.path.join(PKG_DIR, "lm.py"))
-    mod = importlib.util.module_from_spec(spec)
-    spec.loader.exec_module(mod)
-    return mod
+    return pkg
 
 
 GOOD = config([delta(), attention(), attention(window=0, rot=0, softcap=0, ff=0)], loop=(1, 2, 2))
@@ -109,6 +104,6 @@ def test_delta_rule_in_two_pieces():
 def test_yarn_frequencies():
     f, m = plain.rope_frequencies({"dims": 16, "base": 10000.0})
     assert m == 1.0 and np.allclose(f, 10000.0 ** (-np.arange(8) / 8))
-    y, m = plain.rope_frequencies({"dims": 16, "base": 10000.0, "scaling": {"factor": 4.0, "original": 2048, "fast": 32, "slow": 1}})
-    assert np.isclose(m, 0.1 * np.log(4.0) + 1)
-    assert np.allclose(y[0], f[0]) and np.allclose(y[-1], f[-1] / 4) and np.all(y <= f) and np.all(y >= f / 4)
+    y, m = plain.rope_frequencies({"dims": 16, "base": 10000.0, "scaling": {"factor": 5.0, "original": 1500, "fast": 40, "slow": 2}})
+    assert np.isclose(m, 0.1 * np.log(5.0) + 1)
+    assert np.allclose(y[0], f[0]) and np.allclose(y[-1], f[-1] / 5) and np.all(y <= f) and np.all(y >= f / 5 * (1 - 1e-12))

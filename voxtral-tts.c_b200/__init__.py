@@ -5,6 +5,8 @@ include/voxtral_b200_ext.h). This module only loads it with ctypes and mirrors
 the reference's call sequence (tts_cuda_init -> upload -> forward calls) in
 Python. There is no fallback: a missing library or a missing sm_100 GPU raises.
 
+The decoder language models (include/voxtral_b200_lm.h) are bound in lm.py: LanguageModel.
+
 The directory name is not a valid Python identifier; load it with
 importlib (see tests/conftest.py: load_package()).
 """
@@ -13,6 +15,8 @@ import os
 import zlib
 
 import numpy as np
+
+from .lm import LanguageModel, check_config  # noqa: F401
 
 HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(HERE, "lib", "libvoxtral_b200.so")

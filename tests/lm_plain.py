@@ -1,5 +1,5 @@
 """Plain, slow statement of the decoder language models the library serves (the Kegizen design),
-in double precision, one function per mechanism. Checker only: it shares nothing with the product.
+in double precision, one function per mechanism. For tests only: it shares nothing with the product.
 
 Weights are a dict name -> float64 array, the configuration is the dict of a model folder's
 config.json. Sequences are processed one token at a time wherever a mechanism has memory, so what

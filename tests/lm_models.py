@@ -33,8 +33,27 @@ def attention(heads=4, kv_heads=2, dim=32, vdim=48, window=17, keep=3, rot=16, b
     return {"type": "attention", "mixer": m, "mlp": {"kind": "dense", "ff": ff} if ff else None}
 
 
+def latent(heads=4, dim=24, rot_dim=8, vdim=40, kv_rank=48, q_rank=56, window=19, scale=0.3, base=3000.0, kv_from=None, ff=72, experts=0, top=2,
+           rot=None):
+    """A latent attention beside a squared-ReLU feed-forward, one or `experts` of size ff (0: none)."""
+    m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "q_rank": q_rank, "scale": scale}
+    if rot_dim:
+        m["rot"] = {"base": base, "dims": rot_dim if rot is None else rot}
+    if window:
+        m["mask"] = {"size": window}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    mlp = None
+    if ff and experts:
+        mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+    elif ff:
+        mlp = {"kind": "dense", "ff": ff}
+    return {"type": "latent_attention", "mixer": m, "mlp": mlp}
+
+
 def config(layers, width=136, vocab=203, loop=None, eps=2e-5):
-    c = {"architecture": "Kegizen", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width}
+    name = "Bupozen" if layers[0]["type"] == "latent_attention" else "Kegizen"
+    c = {"architecture": name, "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width}
     if loop:
         c["loop"] = dict(zip(("start", "stop", "times"), loop))
     return c
@@ -47,6 +66,9 @@ def shapes(cfg):
         s["loop.in"] = (W, 2 * W)
     for i, l in enumerate(cfg["layers"]):
         p, m = f"l{i}", l["mixer"]
+        if l["type"] == "latent_attention":
+            s.update(latent_shapes(l, p, W))
+            continue
         H, G, d, vd = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
         s[f"{p}.norm1"] = s[f"{p}.norm1b"] = (W,)
         if l["type"] == "delta":
@@ -70,14 +92,30 @@ def shapes(cfg):
     return s
 
 
+def latent_shapes(l, p, W):
+    m, mlp = l["mixer"], l["mlp"]
+    H, R, Q = m["heads"], m["kv_rank"], m["q_rank"]
+    s = {f"{p}.norm1": (W,), f"{p}.mix.dq": (Q, W), f"{p}.mix.dq.norm": (Q,), f"{p}.mix.uq": (H * (m["dim"] + m["rot_dim"]), Q)}
+    if m.get("kv_from") is None:
+        s[f"{p}.mix.dkv"], s[f"{p}.mix.dkv.norm"] = (R + m["rot_dim"], W), (R,)
+    s.update({f"{p}.mix.uk": (H * m["dim"], R), f"{p}.mix.uv": (H * m["vdim"], R), f"{p}.mix.g": (H, W), f"{p}.mix.o": (W, H * m["vdim"])})
+    if mlp and mlp["kind"] == "moe":
+        s[f"{p}.mlp.router"] = (mlp["router"]["experts"], W)
+        for e in range(mlp["router"]["experts"]):
+            s[f"{p}.mlp.e{e}.up"], s[f"{p}.mlp.e{e}.down"] = (mlp["expert"]["ff"], W), (W, mlp["expert"]["ff"])
+    elif mlp:
+        s[f"{p}.mlp.up"], s[f"{p}.mlp.down"] = (mlp["ff"], W), (W, mlp["ff"])
+    return s
+
+
 def weights(cfg, seed, qk_gain=1.6):
-    """BF16 values (as uint16) by name. Query and key gains are large enough that a softmax puts most
+    """BF16 values (as uint16) by name. Routers choose clearly. Query and key gains are large enough that a softmax puts most
     of its weight on a few keys, decays range from almost none to almost all, gains are not one."""
     rng = np.random.default_rng(seed)
     out = {}
     for name, shape in shapes(cfg).items():
         z = rng.standard_normal(shape)
-        if name.endswith((".q.norm", ".k.norm")):
+        if name.endswith((".q.norm", ".k.norm", ".dq.norm")):
             a = qk_gain * (1.0 + 0.2 * z)
         elif "norm" in name:
             a = 1.0 + 0.2 * z
@@ -89,10 +127,44 @@ def weights(cfg, seed, qk_gain=1.6):
             a = 0.6 * z
         elif name == "embed":
             a = z
+        elif name.endswith(".router"):
+            a = 3.0 * z / np.sqrt(shape[-1])
         else:
             a = z / np.sqrt(shape[-1]) * (2.0 if name == "head" else 1.0)
         out[name] = bf16(a)
     return out
+
+
+LIMIT = {"float32": 2e-5, "bfloat16": 4e-4}      # summation order; two-term BF16 products of prompts
+DTYPES = ("float32", "bfloat16")
+
+
+class Case:
+    """A model folder with its weights in double precision."""
+
+    def __init__(self, mod, path, cfg, seed, **kw):
+        self.mod, self.cfg = mod, cfg
+        w = weights(cfg, seed, **kw)
+        self.folder = write_folder(path, cfg, w)
+        self.w = as_float(w)
+
+    def rewrite(self):
+        write_folder(self.folder, self.cfg, {n: bf16(a) for n, a in self.w.items()})
+        self.w = as_float({n: bf16(a) for n, a in self.w.items()})
+
+    def open(self, dtype, **kw):
+        kw.setdefault("max_tokens", 2048)
+        return self.mod.LanguageModel(self.folder, dtype=dtype, **kw)
+
+
+def feed(lm, seq, toks, sizes):
+    """Logits at every place, the tokens cut into portions of the given sizes (repeated)."""
+    out, at, i = [], 0, 0
+    while at < len(toks):
+        n = min(sizes[i % len(sizes)], len(toks) - at)
+        out.append(lm.step(seq, toks[at:at + n], range(n)))
+        at, i = at + n, i + 1
+    return np.concatenate(out)
 
 
 def as_float(w):

@@ -1,5 +1,5 @@
-"""Plain, slow statement of the decoder language models the library serves (the Kegizen design),
-in double precision, one function per mechanism. For tests only: it shares nothing with the product.
+"""Plain, slow statement of the decoder language models the library serves (the Kegizen and Bupozen
+designs), in double precision, one function per mechanism. For tests only: it shares nothing with the product.
 
 Weights are a dict name -> float64 array, the configuration is the dict of a model folder's
 config.json. Sequences are processed one token at a time wherever a mechanism has memory, so what
@@ -138,6 +138,90 @@ def delta(h, w, name, mix, eps):
     return out.reshape(T, H * vd) @ w[name + ".o"].T
 
 
+def rotate_neighbours(x, positions, rot):
+    """x [T, ..., dim]: the first rot.dims dimensions, 2i paired with 2i + 1."""
+    if not rot:
+        return x
+    f, m = rope_frequencies(rot)
+    n = rot["dims"]
+    a = np.asarray(positions, dtype=np.float64).reshape((-1,) + (1,) * (x.ndim - 1)) * f
+    c, s = np.cos(a) * m, np.sin(a) * m
+    u, v = x[..., 0:n:2], x[..., 1:n:2]
+    out = x.copy()
+    out[..., 0:n:2] = u * c - v * s
+    out[..., 1:n:2] = v * c + u * s
+    return out
+
+
+def latent_memory(h, w, name, mix, eps):
+    """What a latent attention keeps of every token: the normed latent [T, kv_rank] and the rotated key part
+    [T, rot_dim] that all heads share."""
+    y = h @ w[name + ".dkv"].T
+    r = mix["kv_rank"]
+    return rms_norm(y[:, :r], w[name + ".dkv.norm"], eps), rotate_neighbours(y[:, r:], np.arange(h.shape[0]), mix.get("rot"))
+
+
+def latent_attention(h, w, name, mix, eps, memory):
+    """Attention whose keys and values are read out of a latent (c, shared key part), with a gate per head."""
+    T = h.shape[0]
+    H, d, e, vd = mix["heads"], mix["dim"], mix["rot_dim"], mix["vdim"]
+    c, shared = memory
+    q = (rms_norm(h @ w[name + ".dq"].T, w[name + ".dq.norm"], eps) @ w[name + ".uq"].T).reshape(T, H, d + e)
+    q_plain, q_rot = q[..., :d], rotate_neighbours(q[..., d:], np.arange(T), mix.get("rot"))
+    k = (c @ w[name + ".uk"].T).reshape(T, H, d)
+    v = (c @ w[name + ".uv"].T).reshape(T, H, vd)
+    gate = sigmoid(h @ w[name + ".g"].T)
+    mask = np.array([[visible(i, j, mix.get("mask")) for j in range(T)] for i in range(T)])
+    out = np.zeros((T, H, vd))
+    for hd in range(H):
+        s = (q_plain[:, hd] @ k[:, hd].T + q_rot[:, hd] @ shared.T) * mix["scale"]
+        s = np.where(mask, s, -np.inf)
+        p = np.exp(s - s.max(axis=1, keepdims=True))
+        out[:, hd] = (p / p.sum(axis=1, keepdims=True)) @ v[:, hd] * gate[:, hd, None]
+    return out.reshape(T, H * vd) @ w[name + ".o"].T
+
+
+def relu2_mlp(h, up, down):
+    return np.maximum(h @ up.T, 0.0) ** 2 @ down.T
+
+
+def route(h, router, top):
+    """Per token: the `top` experts with the largest logits, and the softmax over their logits."""
+    z = h @ router.T
+    chosen = np.argsort(-z, axis=1, kind="stable")[:, :top]
+    zc = np.take_along_axis(z, chosen, axis=1)
+    p = np.exp(zc - zc.max(axis=1, keepdims=True))
+    return chosen, p / p.sum(axis=1, keepdims=True)
+
+
+def experts_mlp(h, w, name, spec):
+    chosen, weight = route(h, w[name + ".router"], spec["router"]["top"])
+    out = np.zeros_like(h)
+    for t in range(h.shape[0]):
+        for e, p in zip(chosen[t], weight[t]):
+            out[t] += p * relu2_mlp(h[t:t + 1], w[f"{name}.e{e}.up"], w[f"{name}.e{e}.down"])[0]
+    return out
+
+
+def parallel_layer(x, w, i, cfg, memories):
+    """One norm feeds the mixer and the feed-forward; both are added to the stream. `memories`: what the
+    latent attentions before this one keep, by layer; a layer with kv_from reads another layer's."""
+    spec, eps = cfg["layers"][i], cfg["norm"]["eps"]
+    mix, mlp = spec["mixer"], spec.get("mlp")
+    h = rms_norm(x, w[f"l{i}.norm1"], eps)
+    if mix.get("kv_from") is None:
+        memories[i] = latent_memory(h, w, f"l{i}.mix", mix, eps)
+        source = i
+    else:
+        source = mix["kv_from"]
+    y = latent_attention(h, w, f"l{i}.mix", mix, eps, memories[source])
+    if mlp and mlp["kind"] == "moe":
+        y = y + experts_mlp(h, w, f"l{i}.mlp", mlp)
+    elif mlp:
+        y = y + relu2_mlp(h, w[f"l{i}.mlp.up"], w[f"l{i}.mlp.down"])
+    return x + y
+
+
 MIXERS = {"delta": delta, "attention": attention}
 
 
@@ -169,7 +253,12 @@ def layer_runs(cfg):
 def forward(w, cfg, tokens):
     """Logits [T, vocab] and the residual stream after every layer run [runs, T, width]."""
     x0 = w["embed"][np.asarray(tokens)]
-    x, taps = x0, []
+    x, taps, memories = x0, [], {}
+    if cfg["architecture"] == "Bupozen":
+        for i in range(len(cfg["layers"])):
+            x = parallel_layer(x, w, i, cfg, memories)
+            taps.append(x)
+        return rms_norm(x, w["final.norm"], cfg["norm"]["eps"]) @ w["head"].T, np.stack(taps)
     for i, starts_pass in layer_runs(cfg):
         if starts_pass:
             x = np.concatenate([x, x0], axis=1) @ w["loop.in"].T

@@ -8,40 +8,16 @@ import numpy as np
 import pytest
 
 import lm_plain as plain
-from lm_models import as_float, attention, bf16, config, delta, error, tokens, weights, write_folder
+from lm_models import DTYPES, LIMIT, Case, attention, config, delta, error, feed, tokens, weights, write_folder
 
 pytestmark = pytest.mark.gpu
 
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-LIMIT = {"float32": 2e-5, "bfloat16": 4e-4}      # summation order; two-term BF16 products of prompts
-DTYPES = ("float32", "bfloat16")
 
 
 @pytest.fixture(scope="module")
 def lm_mod(pkg):
     return pkg
-
-
-class Case:
-    def __init__(self, mod, path, cfg, seed, **kw):
-        self.mod, self.cfg = mod, cfg
-        w = weights(cfg, seed, **kw)
-        self.folder = write_folder(path, cfg, w)
-        self.w = as_float(w)
-
-    def open(self, dtype, **kw):
-        kw.setdefault("max_tokens", 2048)
-        return self.mod.LanguageModel(self.folder, dtype=dtype, **kw)
-
-
-def feed(lm, seq, toks, sizes):
-    """Logits at every place, the tokens cut into portions of the given sizes (repeated)."""
-    out, at, i = [], 0, 0
-    while at < len(toks):
-        n = min(sizes[i % len(sizes)], len(toks) - at)
-        out.append(lm.step(seq, toks[at:at + n], range(n)))
-        at, i = at + n, i + 1
-    return np.concatenate(out)
 
 
 MECHANISMS = {
@@ -245,7 +221,8 @@ def test_far_key_among_hundreds(lm_mod, tmp_path):
     w["l0.mix.k"][:, W // 2:] = 0.0
     w["l0.mix.q"][:] = np.concatenate([w["l0.mix.k"][:, W // 2:], w["l0.mix.k"][:, :W // 2]], axis=1).tolist() * 2
     w["embed"][asks, W // 2:] = w["embed"][far, :W // 2]
-    write_folder(c.folder, cfg, {n: bf16(a) for n, a in w.items()})
+    c.rewrite()
+    w = c.w
     filler = [t for t in tokens(cfg, 700, 2) if t not in (far, asks)]
     toks = filler[:30] + [far] + filler[30:620] + [asks, asks]
     want = plain.forward(w, cfg, toks)[0]
@@ -277,7 +254,7 @@ def test_long_memory_of_the_state(lm_mod, tmp_path):
     cfg = config([delta(heads=2, kv_heads=1, dim=64, vdim=64, conv=4, ff=0)], width=64)
     c = Case(lm_mod, tmp_path, cfg, seed=12)
     c.w["l0.mix.A_log"][:] = (-7.0, -4.0)
-    write_folder(c.folder, cfg, {n: bf16(a) for n, a in c.w.items()})
+    c.rewrite()
     toks = tokens(cfg, 700, 3)
     want = plain.forward(c.w, cfg, toks)[0]
     for dtype in DTYPES:

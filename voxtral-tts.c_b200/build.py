@@ -22,7 +22,8 @@ OBJDIR = os.path.join(LIBDIR, "obj")
 
 # the decoder language models (vb_lm.cu and what it uses) and the speech path; vb_tc.cu and
 # vb_upload.cu serve both
-LM_SOURCES = ["vb_tc.cu", "vb_upload.cu", "vb_lm.cu", "vb_lm_kernels.cu", "vb_lm_attn.cu", "vb_lm_delta.cu",
+LM_SOURCES = ["vb_tc.cu", "vb_upload.cu", "vb_lm.cu", "vb_lm_kernels.cu", "vb_lm_attn.cu", "vb_lm_latent.cu",
+              "vb_lm_moe.cu", "vb_lm_delta.cu",
               "vb_lm_config.cpp", "vb_json.cpp", "vb_safetensors.cpp"]
 SOURCES = LM_SOURCES + ["vb_engine.cu", "vb_simple.cu", "vb_model.cu", "vb_prefill.cu", "vb_abi.cu", "vb_noalloc.cu",
                         "vb_acoustic_tc.cu", "vb_batch.cu", "vb_stream.cu", "vb_codec.cu", "vb_synth.cpp"]

@@ -14,7 +14,7 @@
  * Keys are visited in two stretches, the kept first tokens and the window; a stretch that is out
  * of reach of all of a CTA's rows is never loaded.
  */
-#include "vb_lm_kernels.cuh"
+#include "vb_lm_attn.cuh"
 #include "vb_tc.cuh"
 
 namespace vb {
@@ -22,49 +22,6 @@ namespace vb {
 namespace {
 
 inline int ok(cudaError_t e) { return e == cudaSuccess ? 0 : -1; }
-
-/* ------------------------------------------------------------------ cache elements */
-VB_DEVINL void hilo(float v, uint32_t &hi, uint32_t &lo) {
-    const __nv_bfloat16 h = __float2bfloat16_rn(v);
-    hi = __bfloat16_as_ushort(h);
-    lo = __bfloat16_as_ushort(__float2bfloat16_rn(v - __bfloat162float(h)));
-}
-/* `head`: a head's part of a cache row, `size` elements in either form. */
-VB_DEVINL void kv_put(float *head, int size, int d, float v, int split) {
-    if (split) {
-        uint32_t hi, lo;
-        hilo(v, hi, lo);
-        uint16_t *h = reinterpret_cast<uint16_t *>(head);
-        h[d] = (uint16_t)hi;
-        h[size + d] = (uint16_t)lo;
-    } else {
-        head[d] = v;
-    }
-}
-VB_DEVINL void kv_put4(float *head, int size, int d, float4 v, int split) {
-    if (split) {
-        uint32_t h[4], l[4];
-        hilo(v.x, h[0], l[0]); hilo(v.y, h[1], l[1]); hilo(v.z, h[2], l[2]); hilo(v.w, h[3], l[3]);
-        uint16_t *p = reinterpret_cast<uint16_t *>(head);
-        *reinterpret_cast<uint2 *>(p + d) = make_uint2(h[0] | (h[1] << 16), h[2] | (h[3] << 16));
-        *reinterpret_cast<uint2 *>(p + size + d) = make_uint2(l[0] | (l[1] << 16), l[2] | (l[3] << 16));
-    } else {
-        *reinterpret_cast<float4 *>(head + d) = v;
-    }
-}
-VB_DEVINL float kv_get(const float *head, int size, int d, int split) {
-    if (!split) return __ldcg(head + d);
-    const unsigned short *h = reinterpret_cast<const unsigned short *>(head);
-    return __uint_as_float((uint32_t)__ldcg(h + d) << 16) + __uint_as_float((uint32_t)__ldcg(h + size + d) << 16);
-}
-template <bool SPLIT>
-VB_DEVINL float4 kv_get4(const float *head, int size, int d) {
-    if constexpr (!SPLIT) return vb_ldcg4(head + d);
-    const uint16_t *h = reinterpret_cast<const uint16_t *>(head);
-    const uint2 hi = __ldcg(reinterpret_cast<const uint2 *>(h + d)), lo = __ldcg(reinterpret_cast<const uint2 *>(h + size + d));
-    return make_float4(vb_bf16_lo(hi.x) + vb_bf16_lo(lo.x), vb_bf16_hi(hi.x) + vb_bf16_hi(lo.x), vb_bf16_lo(hi.y) + vb_bf16_lo(lo.y),
-                       vb_bf16_hi(hi.y) + vb_bf16_hi(lo.y));
-}
 
 /* ------------------------------------------------------------------ q, k, v of a row */
 constexpr int kPrepThreads = 512;
@@ -81,14 +38,7 @@ __global__ void __launch_bounds__(kPrepThreads) lm_attn_prepare_kernel(const LmA
     const int pos = a.dyn->pos + m;
     const size_t row = (size_t)lm_ring_row(a.ring, pos);
     for (int i = tid; i < half; i += kPrepThreads) {
-        /* the angle pos * f to twice fp32's precision: sine and cosine of its leading part, and the
-         * remainder as a first-order correction */
-        const float p = (float)pos, f = a.freq[i];
-        const float hi = p * f, lo = fmaf(p, f, -hi) + p * a.freq[half + i];
-        float s, c;
-        sincosf(hi, &s, &c);
-        cs[i] = (c - s * lo) * a.mag;
-        cs[half + i] = (s + c * lo) * a.mag;
+        lm_angle(pos, a.freq[i], a.freq[half + i], a.mag, &cs[i], &cs[half + i]);
     }
     float sq = 0.0f, sk = 0.0f;
     float *Vr = lm_state(a.v, a.dyn) + row * nv;
@@ -149,36 +99,6 @@ __global__ void __launch_bounds__(kPrepThreads) lm_attn_prepare_kernel(const LmA
             else kv_put(Kr + j - d, a.dim, d, value(c), a.split);
         }
     }
-}
-
-/* ------------------------------------------------------------------ which keys */
-/* Keys that rows at positions [imin, imax] may see: [0, a_end) and [b0, b_end), in tiles of KT. */
-struct KeyTiles {
-    int a_end, b0, b_end, a_tiles, n_tiles;
-};
-template <int KT>
-VB_DEVINL KeyTiles key_tiles(int imin, int imax, int window, int keep) {
-    KeyTiles t;
-    t.b_end = imax + 1;
-    if (window <= 0) { t.a_end = 0; t.b0 = 0; }
-    else {
-        t.a_end = keep < t.b_end ? keep : t.b_end;
-        t.b0 = imin - window + 1 > t.a_end ? imin - window + 1 : t.a_end;
-    }
-    t.a_tiles = (t.a_end + KT - 1) / KT;
-    t.n_tiles = t.a_tiles + (t.b_end > t.b0 ? (t.b_end - t.b0 + KT - 1) / KT : 0);
-    return t;
-}
-/* First key of tile t and how many keys it has. */
-template <int KT>
-VB_DEVINL void key_tile(const KeyTiles &k, int t, int *j0, int *n) {
-    const bool first = t < k.a_tiles;
-    const int s = first ? t * KT : k.b0 + (t - k.a_tiles) * KT, e = first ? k.a_end : k.b_end;
-    *j0 = s;
-    *n = e - s < KT ? e - s : KT;
-}
-VB_DEVINL bool key_seen(int i, int j, int window, int keep) {
-    return j <= i && (window <= 0 || i - j < window || j < keep);
 }
 
 /* ------------------------------------------------------------------ generic kernel */
@@ -367,12 +287,7 @@ __global__ void __launch_bounds__(kSaThreads) lm_attn_step_kernel(const LmAttn a
     if (writer)
         for (int c = tid; c < vdim; c += kSaThreads) kv_put(Vc + new_row * nv, vdim, c, lm_sum_batch(a.qkv, 0, nq + nk + g * vdim + c), SPLIT);
     for (int i = tid; i < half; i += kSaThreads) {
-        const float p = (float)pos, f = a.freq[i];
-        const float hi = p * f, lo = fmaf(p, f, -hi) + p * a.freq[half + i];
-        float s, c;
-        sincosf(hi, &s, &c);
-        cs[i] = (c - s * lo) * a.mag;
-        cs[half + i] = (s + c * lo) * a.mag;
+        lm_angle(pos, a.freq[i], a.freq[half + i], a.mag, &cs[i], &cs[half + i]);
     }
     sq = vb_warp_sum(sq);
     sk = vb_warp_sum(sk);
@@ -558,26 +473,6 @@ int launch_attn_step(const LmAttn &a, int splits, int lanes_h, cudaStream_t st) 
 }
 
 /* ------------------------------------------------------------------ prompts on the warp-level tensor cores */
-VB_DEVINL void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-VB_DEVINL void ldsm(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-VB_DEVINL void ldsm_t(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-/* Byte offset of the 16-byte chunk `chunk` of key row `key` in a [keys][16 * STEPS] BF16 tile; chunks are
- * XOR-swizzled by the key so that eight rows of one chunk column hit eight different banks. */
-template <int STEPS>
-VB_DEVINL uint32_t tile_off(int key, int chunk) {
-    return (uint32_t)(key * STEPS * 32 + (((chunk & ~7) | ((chunk ^ key) & 7)) << 4));
-}
-
 constexpr int kMaThreads = 256, kMaWarps = 8, kMaKeys = 32;
 
 /* Requests 32 keys of one KV head: the high and low halves of the cache rows, 16 bytes per copy,
@@ -588,23 +483,40 @@ VB_DEVINL void request_tile(unsigned char *hi_t, const float *cache, int ld, int
     for (int i = threadIdx.x; i < n * 2 * per; i += kMaThreads) {
         const int key = i / (2 * per), f = i % (2 * per), plane = f >= per ? 1 : 0, chunk = f - plane * per;
         const uint16_t *src = reinterpret_cast<const uint16_t *>(cache + (size_t)lm_ring_row(ring, j0 + key) * ld + col0) + f * 8;
-        unsigned char *dst = hi_t + plane * (kMaKeys * STEPS * 32) + tile_off<STEPS>(key, chunk);
-        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(vb_smem_u32(dst)), "l"(src) : "memory");
+        lm_cp16(hi_t + plane * (kMaKeys * STEPS * 32) + tile_off<STEPS>(key, chunk), src);
     }
 }
+/* The same out of keys and values that were read out of a latent: a head's own columns from the written-out
+ * rows, then `shared` columns (the key part all heads have in common) from the latent's cache row. */
+template <int STEPS>
+VB_DEVINL void request_wide(unsigned char *hi_t, const LmWide &w, int col0, int size, int shared, int j0, int n, const LmRing &ring) {
+    const int own = size / 8, per = own + shared / 8, row = w.rank + w.rot_dim;
+    for (int i = threadIdx.x; i < n * 2 * per; i += kMaThreads) {
+        const int key = i / (2 * per), f = i % (2 * per), plane = f >= per ? 1 : 0, chunk = f - plane * per;
+        const uint16_t *src;
+        if (chunk < own) src = w.kv + plane * w.plane + (size_t)(j0 + key - w.first) * w.ld + col0 + chunk * 8;
+        else src = reinterpret_cast<const uint16_t *>(w.cache + (size_t)lm_ring_row(ring, j0 + key) * row) + plane * row + w.rank + (chunk - own) * 8;
+        lm_cp16(hi_t + plane * (kMaKeys * STEPS * 32) + tile_off<STEPS>(key, chunk), src);
+    }
+}
+
+struct LmNotWide {};
+template <bool WIDE> struct LmWideSel { using type = LmNotWide; };
+template <> struct LmWideSel<true> { using type = LmWide; };
 
 /* cap * tanh(x / cap), the hyperbolic tangent through one exponential (absolute error about 1e-7 of cap) */
 VB_DEVINL float soft_cap(float x, float cap, float two_over_cap) {
     return cap - 2.0f * cap * __fdividef(1.0f, 1.0f + __expf(x * two_over_cap));
 }
 
-/* A CTA serves one KV head; each of its eight warps owns 16 query rows of one query head of the
+/* WIDE: every head has keys and values of its own, read out of a latent (LmWide).
+ * A CTA serves one KV head; each of its eight warps owns 16 query rows of one query head of the
  * group (consecutive (row block, head) tiles), so that the staged keys are shared by up to eight
  * warps. Every product a.b is taken as a_hi.b_hi + a_hi.b_lo + a_lo.b_hi, accumulated in fp32;
  * scores, softcap, weights and the running maximum are fp32. DK, DV: 16-wide steps of the key
  * and value sizes (padded with zeros). */
-template <int DK, int DV>
-__global__ void __launch_bounds__(kMaThreads) lm_attn_mma_kernel(const LmAttn a, int M) {
+template <int DK, int DV, bool WIDE>
+__global__ void __launch_bounds__(kMaThreads) lm_attn_mma_kernel(const LmAttn a, const typename LmWideSel<WIDE>::type wide, int M) {
     extern __shared__ __align__(128) unsigned char ma_tiles[];
     /* two buffers of K high, K low, V high, V low */
     constexpr int kTileK = kMaKeys * DK * 32, kTileV = kMaKeys * DV * 32, kBuf = 2 * (kTileK + kTileV);
@@ -627,8 +539,11 @@ __global__ void __launch_bounds__(kMaThreads) lm_attn_mma_kernel(const LmAttn a,
     const int last_row = T1 > T0 ? ((T1 - 1) / group * 16 + 15 < M - 1 ? (T1 - 1) / group * 16 + 15 : M - 1) : 0;
     const KeyTiles kt = key_tiles<kMaKeys>(pos0 + T0 / group * 16, pos0 + last_row, a.window, a.keep);
     const int w_imin = pos0 + r0, w_imax = pos0 + (r0 + 15 < M - 1 ? r0 + 15 : M - 1);
-    const float *Kc = lm_state(a.k, a.dyn), *Vc = lm_state(a.v, a.dyn);
+    const float *Kc = nullptr, *Vc = nullptr;
+    if constexpr (!WIDE) { Kc = lm_state(a.k, a.dyn); Vc = lm_state(a.v, a.dyn); }
     const int ldk = a.kv_heads * a.dim, ldv = a.kv_heads * a.vdim;
+    typename LmWideSel<WIDE>::type lw = wide;
+    if constexpr (WIDE) lw.cache += (size_t)a.dyn->slot * lw.slab;
 
     /* Q as A fragments: (row A, k 2t..), (row B, k 2t..), (row A, k 8 + 2t..), (row B, k 8 + 2t..) */
     uint32_t qh[DK][4], ql[DK][4];
@@ -639,11 +554,27 @@ __global__ void __launch_bounds__(kMaThreads) lm_attn_mma_kernel(const LmAttn a,
 #pragma unroll
             for (int rr = 0; rr < 2; rr++) {
                 const int d = ks * 16 + hf * 8 + 2 * tq;
-                const float *q = a.q + (size_t)(rr ? rowB : rowA) * a.heads * a.dim + (size_t)h * a.dim + d;
                 const bool v = rr ? validB : validA;
+                float q0 = 0.0f, q1 = 0.0f;
+                if constexpr (WIDE) {
+                    if (v && d < a.dim) {          /* dim is a multiple of 8: d and d + 1 are a rotated pair or neither is */
+                        const int row = rr ? rowB : rowA, i = (d - (a.dim - wide.rot_dim)) / 2, half = a.rot / 2;
+                        const float2 u = lm_sum2(wide.q, row, h * a.dim + d);
+                        q0 = u.x; q1 = u.y;
+                        if (d >= a.dim - wide.rot_dim && i < half) {
+                            const float c = wide.cs[(size_t)row * a.rot + i], s = wide.cs[(size_t)row * a.rot + half + i];
+                            q0 = u.x * c - u.y * s;
+                            q1 = u.y * c + u.x * s;
+                        }
+                    }
+                } else {
+                    const float *q = a.q + (size_t)(rr ? rowB : rowA) * a.heads * a.dim + (size_t)h * a.dim + d;
+                    if (v && d < a.dim) q0 = q[0];
+                    if (v && d + 1 < a.dim) q1 = q[1];
+                }
                 uint32_t h0, l0, h1, l1;
-                hilo(v && d < a.dim ? q[0] : 0.0f, h0, l0);
-                hilo(v && d + 1 < a.dim ? q[1] : 0.0f, h1, l1);
+                hilo(q0, h0, l0);
+                hilo(q1, h1, l1);
                 qh[ks][hf * 2 + rr] = h0 | (h1 << 16);
                 ql[ks][hf * 2 + rr] = l0 | (l1 << 16);
             }
@@ -658,16 +589,21 @@ __global__ void __launch_bounds__(kMaThreads) lm_attn_mma_kernel(const LmAttn a,
         int j0, n;
         key_tile<kMaKeys>(kt, t, &j0, &n);
         unsigned char *b = ma_tiles + (t & 1) * kBuf;
-        request_tile<DK>(b, Kc, ldk, g * a.dim, a.dim, j0, n, a.ring);
-        request_tile<DV>(b + 2 * kTileK, Vc, ldv, g * a.vdim, a.vdim, j0, n, a.ring);
-        asm volatile("cp.async.commit_group;" ::: "memory");
+        if constexpr (WIDE) {
+            request_wide<DK>(b, lw, g * (a.dim - lw.rot_dim), a.dim - lw.rot_dim, lw.rot_dim, j0, n, a.ring);
+            request_wide<DV>(b + 2 * kTileK, lw, lw.v0 + g * a.vdim, a.vdim, 0, j0, n, a.ring);
+        } else {
+            request_tile<DK>(b, Kc, ldk, g * a.dim, a.dim, j0, n, a.ring);
+            request_tile<DV>(b + 2 * kTileK, Vc, ldv, g * a.vdim, a.vdim, j0, n, a.ring);
+        }
+        lm_cp_commit();
     };
     if (kt.n_tiles > 0) request(0);
 
     for (int t = 0; t < kt.n_tiles; t++) {
         int j0, n;
         key_tile<kMaKeys>(kt, t, &j0, &n);
-        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        lm_cp_wait_all();
         __syncthreads();                               /* this buffer is complete, the other one is free */
         if (t + 1 < kt.n_tiles) request(t + 1);
         const uint32_t sKh = smem0 + (uint32_t)((t & 1) * kBuf), sKl = sKh + kTileK, sVh = sKl + kTileK, sVl = sVh + kTileV;
@@ -754,7 +690,11 @@ __global__ void __launch_bounds__(kMaThreads) lm_attn_mma_kernel(const LmAttn a,
     lA += __shfl_xor_sync(0xffffffffu, lA, 2);
     lB += __shfl_xor_sync(0xffffffffu, lB, 1);
     lB += __shfl_xor_sync(0xffffffffu, lB, 2);
-    const float rA = 1.0f / lA, rB = 1.0f / lB;
+    float rA = 1.0f / lA, rB = 1.0f / lB;
+    if constexpr (WIDE) {
+        if (validA) rA *= wide.gate[(size_t)rowA * a.heads + h];
+        if (validB) rB *= wide.gate[(size_t)rowB * a.heads + h];
+    }
 #pragma unroll
     for (int nt = 0; nt < 2 * DV; nt++)
 #pragma unroll
@@ -766,19 +706,19 @@ __global__ void __launch_bounds__(kMaThreads) lm_attn_mma_kernel(const LmAttn a,
         }
 }
 
-template <int DK, int DV>
-int launch_mma(const LmAttn &a, int M, cudaStream_t st) {
+template <int DK, int DV, bool WIDE>
+int launch_mma(const LmAttn &a, const typename LmWideSel<WIDE>::type &wide, int M, cudaStream_t st) {
     constexpr size_t smem = (size_t)2 * kMaKeys * 64 * (DK + DV);
     static bool attr = false;
     if (!attr) {
-        if (cudaFuncSetAttribute(lm_attn_mma_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+        if (cudaFuncSetAttribute(lm_attn_mma_kernel<DK, DV, WIDE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
             cudaGetLastError();
             return -1;
         }
         attr = true;
     }
     const int tiles = (M + 15) / 16 * (a.heads / a.kv_heads);
-    return ok(launch_pdl(lm_attn_mma_kernel<DK, DV>, dim3((tiles + kMaWarps - 1) / kMaWarps, a.kv_heads), dim3(kMaThreads), smem, st, a, M));
+    return ok(launch_pdl(lm_attn_mma_kernel<DK, DV, WIDE>, dim3((tiles + kMaWarps - 1) / kMaWarps, a.kv_heads), dim3(kMaThreads), smem, st, a, wide, M));
 }
 
 constexpr int kSplitBudget = 296;        /* two CTAs per SM */
@@ -830,8 +770,20 @@ bool lm_attn_mma_ok(int dim, int vdim) { return dim <= 128 && vdim <= 128 && dim
 
 int lm_attn_mma(const LmAttn &a, int M, cudaStream_t st) {
     const bool k4 = a.dim <= 64, v4 = a.vdim <= 64;
-    if (k4) return v4 ? launch_mma<4, 4>(a, M, st) : launch_mma<4, 8>(a, M, st);
-    return v4 ? launch_mma<8, 4>(a, M, st) : launch_mma<8, 8>(a, M, st);
+    const LmNotWide w;
+    if (k4) return v4 ? launch_mma<4, 4, false>(a, w, M, st) : launch_mma<4, 8, false>(a, w, M, st);
+    return v4 ? launch_mma<8, 4, false>(a, w, M, st) : launch_mma<8, 8, false>(a, w, M, st);
+}
+
+bool lm_attn_wide_ok(int plain, int rot_dim, int vdim) {
+    return plain + rot_dim <= 192 && vdim <= 128 && plain % 8 == 0 && rot_dim % 8 == 0 && vdim % 8 == 0;
+}
+
+int lm_attn_wide(const LmAttn &a, const LmWide &w, int M, cudaStream_t st) {
+    const bool v4 = a.vdim <= 64;
+    if (a.dim <= 64) return v4 ? launch_mma<4, 4, true>(a, w, M, st) : launch_mma<4, 8, true>(a, w, M, st);
+    if (a.dim <= 128) return v4 ? launch_mma<8, 4, true>(a, w, M, st) : launch_mma<8, 8, true>(a, w, M, st);
+    return v4 ? launch_mma<12, 4, true>(a, w, M, st) : launch_mma<12, 8, true>(a, w, M, st);
 }
 
 bool lm_attn_step_ok(const LmAttn &a) {

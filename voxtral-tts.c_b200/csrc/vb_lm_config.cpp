@@ -39,6 +39,13 @@ std::vector<LmConfig::Run> LmConfig::runs() const {
     return r;
 }
 
+int LmConfig::cache_window(int i) const {
+    int w = layers[i].mixer.mask.window;
+    for (const LmLayer &l : layers)
+        if (l.mixer.kv_from == i) w = w > 0 && l.mixer.mask.window > 0 ? std::max(w, l.mixer.mask.window) : 0;
+    return w;
+}
+
 namespace {
 
 /* Reads members of one JSON object and keeps the first complaint. */
@@ -70,12 +77,48 @@ struct Fields {
 
 constexpr int kMaxSize = 1 << 20;
 
-bool read_mixer(const Json &layer, const std::string &where, LmMixer *m, std::string *err) {
-    const Json *type = layer.get("type"), *mix = layer.get("mixer");
-    if (!type || type->kind != Json::STRING || !mix || mix->kind != Json::OBJECT) {
-        *err = "config.json: " + where + " needs 'type' and 'mixer'";
-        return false;
+bool read_mask(const Json *mix, const std::string &where, LmMask *mask, std::string *err) {
+    const Json *o = mix->get("mask");
+    if (!o) return true;
+    Fields g{o, where + ".mixer.mask", err};
+    mask->window = g.integer("size", 1, 1 << 30);
+    mask->keep_first = g.integer("keep_first", 0, 1 << 30, false, 0);
+    return g.ok;
+}
+
+bool read_rope(const Json *mix, const std::string &where, int dim, LmRope *rope, std::string *err) {
+    const Json *rot = mix->get("rot");
+    if (!rot) return true;
+    Fields g{rot, where + ".mixer.rot", err};
+    rope->dims = g.integer("dims", 0, dim);
+    rope->base = g.number("base");
+    if (g.ok && (rope->dims & 1)) g.complain("dims", "is odd");
+    if (g.ok && rope->base <= 1.0) g.complain("base", "is not above 1");
+    if (const Json *sc = rot->get("scaling")) {
+        Fields s{sc, where + ".mixer.rot.scaling", err};
+        rope->yarn = true;
+        rope->factor = s.number("factor");
+        rope->original = s.number("original");
+        rope->fast = s.number("fast");
+        rope->slow = s.number("slow");
+        if (s.ok && !(rope->factor > 0 && rope->original > 0 && rope->fast > 0 && rope->slow > 0))
+            s.complain("factor", "and its companions have to be positive");
+        if (!s.ok) return false;
     }
+    return g.ok;
+}
+
+bool mixer_of(const Json &layer, const std::string &where, const Json **type, const Json **mix, std::string *err) {
+    *type = layer.get("type");
+    *mix = layer.get("mixer");
+    if (*type && (*type)->kind == Json::STRING && *mix && (*mix)->kind == Json::OBJECT) return true;
+    *err = "config.json: " + where + " needs 'type' and 'mixer'";
+    return false;
+}
+
+bool read_mixer(const Json &layer, const std::string &where, LmMixer *m, std::string *err) {
+    const Json *type, *mix;
+    if (!mixer_of(layer, where, &type, &mix, err)) return false;
     Fields f{mix, where + ".mixer", err};
     m->heads = f.integer("heads", 1, 65535);
     m->kv_heads = f.integer("kv_heads", 1, 65535, false, m->heads);
@@ -95,35 +138,12 @@ bool read_mixer(const Json &layer, const std::string &where, LmMixer *m, std::st
     m->scale = f.number("scale");
     m->softcap = f.number("softcap", false, 0.0);
     if (f.ok && m->softcap < 0.0) f.complain("softcap", "is negative");
-    if (const Json *mask = mix->get("mask")) {
-        Fields g{mask, where + ".mixer.mask", err};
-        m->mask.window = g.integer("size", 1, 1 << 30);
-        m->mask.keep_first = g.integer("keep_first", 0, 1 << 30, false, 0);
-        if (!g.ok) return false;
-    }
-    if (const Json *rot = mix->get("rot")) {
-        Fields g{rot, where + ".mixer.rot", err};
-        m->rope.dims = g.integer("dims", 0, m->dim);
-        m->rope.base = g.number("base");
-        if (g.ok && (m->rope.dims & 1)) g.complain("dims", "is odd");
-        if (g.ok && m->rope.base <= 1.0) g.complain("base", "is not above 1");
-        if (const Json *sc = rot->get("scaling")) {
-            Fields s{sc, where + ".mixer.rot.scaling", err};
-            m->rope.yarn = true;
-            m->rope.factor = s.number("factor");
-            m->rope.original = s.number("original");
-            m->rope.fast = s.number("fast");
-            m->rope.slow = s.number("slow");
-            if (s.ok && !(m->rope.factor > 0 && m->rope.original > 0 && m->rope.fast > 0 && m->rope.slow > 0))
-                s.complain("factor", "and its companions have to be positive");
-            if (!s.ok) return false;
-        }
-        if (!g.ok) return false;
-    }
-    return f.ok;
+    return read_mask(mix, where, &m->mask, err) && read_rope(mix, where, m->dim, &m->rope, err) && f.ok;
 }
 
-bool read_kegizen(const Json &c, LmConfig *out, std::string *err) {
+/* vocab, width, norm.eps and the list of layers, each read by `layer`. */
+bool read_stack(const Json &c, LmConfig *out, std::string *err,
+                bool (*layer)(const Json &, const std::string &where, LmLayer *, std::string *err)) {
     Fields f{&c, "model", err};
     out->vocab = f.integer("vocab", 1, 1 << 26);
     out->width = f.integer("width", 1, kMaxSize);
@@ -137,21 +157,30 @@ bool read_kegizen(const Json &c, LmConfig *out, std::string *err) {
         return false;
     }
     for (size_t i = 0; i < layers->items.size(); i++) {
-        const std::string where = "layers[" + std::to_string(i) + "]";
         LmLayer l;
-        if (!read_mixer(layers->items[i], where, &l.mixer, err)) return false;
-        if (const Json *mlp = layers->items[i].get("mlp")) {
-            const Json *kind = mlp->get("kind");
-            if (kind && (kind->kind != Json::STRING || kind->text != "dense")) {
-                *err = "config.json: " + where + ".mlp.kind is not known";
-                return false;
-            }
-            Fields m{mlp, where + ".mlp", err};
-            l.ff = m.integer("ff", 1, kMaxSize);
-            if (!m.ok) return false;
-        }
+        if (!layer(layers->items[i], "layers[" + std::to_string(i) + "]", &l, err)) return false;
         out->layers.push_back(l);
     }
+    return true;
+}
+
+bool read_kegizen_layer(const Json &layer, const std::string &where, LmLayer *l, std::string *err) {
+    if (!read_mixer(layer, where, &l->mixer, err)) return false;
+    const Json *mlp = layer.get("mlp");
+    if (!mlp) return true;
+    const Json *kind = mlp->get("kind");
+    if (kind && (kind->kind != Json::STRING || kind->text != "dense")) {
+        *err = "config.json: " + where + ".mlp.kind is not known";
+        return false;
+    }
+    Fields m{mlp, where + ".mlp", err};
+    l->mlp.kind = LM_MLP_SWIGLU;
+    l->mlp.ff = m.integer("ff", 1, kMaxSize);
+    return m.ok;
+}
+
+bool read_kegizen(const Json &c, LmConfig *out, std::string *err) {
+    if (!read_stack(c, out, err, read_kegizen_layer)) return false;
     if (const Json *loop = c.get("loop")) {
         Fields l{loop, "loop", err};
         const int nl = (int)out->layers.size();
@@ -163,8 +192,65 @@ bool read_kegizen(const Json &c, LmConfig *out, std::string *err) {
     return true;
 }
 
+bool read_bupozen_layer(const Json &layer, const std::string &where, LmLayer *l, std::string *err) {
+    const Json *type, *mix;
+    if (!mixer_of(layer, where, &type, &mix, err)) return false;
+    if (type->text != "latent_attention") {
+        *err = "config.json: " + where + ".type '" + type->text + "' is not a known mixer";
+        return false;
+    }
+    LmMixer *m = &l->mixer;
+    Fields f{mix, where + ".mixer", err};
+    m->kind = LM_MIXER_LATENT;
+    m->heads = f.integer("heads", 1, 65535);
+    m->kv_heads = m->heads;
+    m->dim = f.integer("dim", 1, kMaxSize);
+    m->rot_dim = f.integer("rot_dim", 0, kMaxSize);
+    m->vdim = f.integer("vdim", 1, kMaxSize);
+    m->q_rank = f.integer("q_rank", 1, kMaxSize);
+    m->kv_rank = f.integer("kv_rank", 1, kMaxSize);
+    m->scale = f.number("scale");
+    if (mix->get("kv_from")) m->kv_from = f.integer("kv_from", 0, kMaxSize);
+    if (!f.ok || !read_mask(mix, where, &m->mask, err) || !read_rope(mix, where, m->rot_dim, &m->rope, err)) return false;
+    const Json *mlp = layer.get("mlp");
+    if (!mlp) return true;
+    const Json *kind = mlp->get("kind");
+    const bool moe = kind && kind->kind == Json::STRING && kind->text == "moe";
+    if (!moe && !(kind && kind->kind == Json::STRING && kind->text == "dense")) {
+        *err = "config.json: " + where + ".mlp.kind is not known";
+        return false;
+    }
+    l->mlp.kind = LM_MLP_RELU2;
+    Fields s{moe ? mlp->get("expert") : mlp, where + (moe ? ".mlp.expert" : ".mlp"), err};
+    l->mlp.ff = s.integer("ff", 1, kMaxSize);
+    if (!moe) return s.ok;
+    Fields r{mlp->get("router"), where + ".mlp.router", err};
+    l->mlp.experts = r.integer("experts", 1, 1 << 16);
+    l->mlp.top = r.integer("top", 1, l->mlp.experts > 0 ? l->mlp.experts : 1);
+    return s.ok && r.ok;
+}
+
+bool read_bupozen(const Json &c, LmConfig *out, std::string *err) {
+    out->block = LM_BLOCK_PARALLEL;
+    out->norm = LM_NORM_RMS;
+    if (!read_stack(c, out, err, read_bupozen_layer)) return false;
+    for (size_t i = 0; i < out->layers.size(); i++) {
+        const LmMixer &m = out->layers[i].mixer;
+        if (m.kv_from < 0) continue;
+        const LmMixer *o = m.kv_from < (int)i ? &out->layers[m.kv_from].mixer : nullptr;
+        if (!o || o->kv_from >= 0 || o->kv_rank != m.kv_rank || o->rot_dim != m.rot_dim || o->rope.dims != m.rope.dims ||
+            o->rope.base != m.rope.base) {
+            *err = "config.json: layers[" + std::to_string(i) + "].mixer.kv_from has to name an earlier layer with a latent of its own, of equal "
+                   "kv_rank, rot_dim and rotation";
+            return false;
+        }
+    }
+    return true;
+}
+
 const LmArchitecture kArchitectures[] = {
     {"Kegizen", read_kegizen},
+    {"Bupozen", read_bupozen},
 };
 
 } // namespace

@@ -20,8 +20,8 @@ VB_DEVINL float cta_sum(float v, float *red) {
 }
 
 /* One row of the residual stream per CTA, held in registers: the sublayer's output (split-K
- * partials) is normalised, added to the stream, and the new row is normalised again for the next
- * sublayer. Variances are means of squared deviations. A thread owns NV groups of VEC columns. */
+ * partials) is normalised or taken as it is, added to the stream, and the new row is normalised for
+ * the next sublayer. Variances are means of squared deviations. A thread owns NV groups of VEC columns. */
 template <int VEC, int NV>
 __global__ void __launch_bounds__(1024) lm_residual_kernel(const LmResidual a) {
     __shared__ float red[4][32];
@@ -37,7 +37,7 @@ __global__ void __launch_bounds__(1024) lm_residual_kernel(const LmResidual a) {
 #pragma unroll
         for (int j = 0; j < VEC; j++) {
             const int c = col(i) + j;
-            gp[i * VEC + j] = a.post_gain && c < W ? __ldg(a.post_gain + c) : 0.0f;
+            gp[i * VEC + j] = a.join == LM_JOIN_NORMED && c < W ? __ldg(a.post_gain + c) : 0.0f;
             gn[i * VEC + j] = a.next == LM_NEXT_NORM && c < W ? __ldg(a.next_gain + c) : 0.0f;
         }
     pdl_wait();
@@ -52,7 +52,7 @@ __global__ void __launch_bounds__(1024) lm_residual_kernel(const LmResidual a) {
             for (int j = 0; j < VEC; j++) x[i * VEC + j] = col(i) < W ? __uint_as_float((uint32_t)e0[col(i) + j] << 16) : 0.0f;
     } else {
         float r[N];
-        const bool add = a.post_gain != nullptr;
+        const bool add = a.join != LM_JOIN_REPLACE;
 #pragma unroll
         for (int i = 0; i < NV; i++) {
             const int c = col(i);
@@ -67,11 +67,30 @@ __global__ void __launch_bounds__(1024) lm_residual_kernel(const LmResidual a) {
                 x[i] = in ? lm_sum_batch(a.part, src, c) : 0.0f;
             }
         }
-        if (add) {
+        for (int k = 0; k < a.mix.top; k++) {              /* the chosen experts, weighted */
+            const float p = a.mix.weight[(size_t)src * a.mix.top + k];
+            const float *y = a.mix.y + (size_t)a.mix.at[(size_t)src * a.mix.top + k] * a.mix.ld;
+#pragma unroll
+            for (int i = 0; i < NV; i++) {
+                const int c = col(i);
+                if (c >= W) continue;
+                if constexpr (VEC == 4) {
+                    const float4 v = vb_ldcg4(y + c);
+                    x[i * 4] = fmaf(p, v.x, x[i * 4]); x[i * 4 + 1] = fmaf(p, v.y, x[i * 4 + 1]);
+                    x[i * 4 + 2] = fmaf(p, v.z, x[i * 4 + 2]); x[i * 4 + 3] = fmaf(p, v.w, x[i * 4 + 3]);
+                } else {
+                    x[i] = fmaf(p, vb_ldcg(y + c), x[i]);
+                }
+            }
+        }
+        if (a.join == LM_JOIN_ADD) {
+#pragma unroll
+            for (int i = 0; i < N; i++) x[i] = r[i] + x[i];
+        } else if (add) {
             float s = 0.0f;
 #pragma unroll
             for (int i = 0; i < N; i++) s += x[i];
-            const float mean = cta_sum(s, red[0]) * inv_w;
+            const float mean = a.rms ? 0.0f : cta_sum(s, red[0]) * inv_w;
             s = 0.0f;
 #pragma unroll
             for (int i = 0; i < N; i++) {
@@ -108,7 +127,7 @@ __global__ void __launch_bounds__(1024) lm_residual_kernel(const LmResidual a) {
         float s = 0.0f;
 #pragma unroll
         for (int i = 0; i < N; i++) s += x[i];
-        const float mean = cta_sum(s, red[2]) * inv_w;
+        const float mean = a.rms ? 0.0f : cta_sum(s, red[2]) * inv_w;
         s = 0.0f;
 #pragma unroll
         for (int i = 0; i < N; i++) {
@@ -135,11 +154,11 @@ __global__ void __launch_bounds__(1024) lm_residual_kernel(const LmResidual a) {
     }
 }
 
-__global__ void lm_pack_rows_kernel(uint16_t *dst, int Kp, int row0, int step, const uint16_t *src, int rows, int K) {
+__global__ void lm_pack_rows_kernel(uint16_t *dst, int Kp, int row0, int step, int col0, const uint16_t *src, int rows, int K) {
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i >= (size_t)rows * Kp) return;
-    const int r = (int)(i / Kp), c = (int)(i % Kp);
-    dst[(size_t)(row0 + (long long)r * step) * Kp + c] = c < K ? src[(size_t)r * K + c] : (uint16_t)0;
+    if (i >= (size_t)rows * K) return;
+    const int r = (int)(i / K), c = (int)(i % K);
+    dst[(size_t)(row0 + (long long)r * step) * Kp + col0 + c] = src[i];
 }
 
 __global__ void lm_widen_kernel(float *dst, const uint16_t *src, int n) {
@@ -164,11 +183,20 @@ __global__ void lm_fill_random_kernel(uint16_t *dst, size_t n, uint32_t seed, fl
  * levels, so that its rounding error grows with the step length and the number of steps, not with K. */
 constexpr int kFgT = 64, kFgK = 16;
 __global__ void __launch_bounds__(256)
-lm_gemm_f32_kernel(float *y, int ld_out, const float *x, int ldx, const uint16_t *W, int ldw, int M, int N, int K, int swiglu) {
+lm_gemm_f32_kernel(float *y, int ld_out, const float *x, int ldx, const uint16_t *W, int ldw, int M, int N, int K, int act,
+                   const int4 *table, int group_rows) {
     __shared__ __align__(16) float xs[kFgK][kFgT + 4], ws[kFgK][kFgT + 4];
     pdl_launch_dependents();
     pdl_wait();
-    const int n0 = blockIdx.x * kFgT, m0 = blockIdx.y * kFgT;
+    const int n0 = blockIdx.x * kFgT;
+    int m0 = blockIdx.y * kFgT;
+    if (table) {                       /* two tiles of rows per block of 128 */
+        const int4 g = __ldcg(table + (blockIdx.y >> 1));
+        m0 = g.y + (int)(blockIdx.y & 1) * kFgT;
+        M = g.y + g.z;
+        if (g.x < 0 || m0 >= M) return;
+        W += (size_t)g.x * group_rows * ldw;
+    }
     const int tid = threadIdx.x, tm = (tid >> 4) * 4, tn = (tid & 15) * 4;
     float sum[4][4] = {};
     for (int k0 = 0; k0 < K; k0 += kFgK) {
@@ -198,14 +226,16 @@ lm_gemm_f32_kernel(float *y, int ld_out, const float *x, int ldx, const uint16_t
     for (int i = 0; i < 4; i++) {
         const int m = m0 + tm + i;
         if (m >= M) break;
-        if (swiglu) {
+        if (act == LM_ACT_SWIGLU) {
             for (int j = 0; j < 4; j += 2) {
                 const int n = n0 + tn + j;
                 if (n + 1 < N) y[(size_t)m * ld_out + n / 2] = sum[i][j] / (1.0f + expf(-sum[i][j])) * sum[i][j + 1];
             }
         } else {
-            for (int j = 0; j < 4; j++)
-                if (n0 + tn + j < N) y[(size_t)m * ld_out + n0 + tn + j] = sum[i][j];
+            for (int j = 0; j < 4; j++) {
+                const float v = act == LM_ACT_RELU2 ? fmaxf(sum[i][j], 0.0f) * fmaxf(sum[i][j], 0.0f) : sum[i][j];
+                if (n0 + tn + j < N) y[(size_t)m * ld_out + n0 + tn + j] = v;
+            }
         }
     }
 }
@@ -264,10 +294,10 @@ int lm_residual(const LmResidual &a, int M, cudaStream_t st) {
     return -1;
 }
 
-int lm_pack_rows(uint16_t *dst, int Kp, int row0, int step, const uint16_t *src, int rows, int K, cudaStream_t st) {
-    const size_t n = (size_t)rows * Kp;
+int lm_pack_rows(uint16_t *dst, int Kp, int row0, int step, int col0, const uint16_t *src, int rows, int K, cudaStream_t st) {
+    const size_t n = (size_t)rows * K;
     if (n == 0) return 0;
-    lm_pack_rows_kernel<<<(unsigned)((n + 255) / 256), 256, 0, st>>>(dst, Kp, row0, step, src, rows, K);
+    lm_pack_rows_kernel<<<(unsigned)((n + 255) / 256), 256, 0, st>>>(dst, Kp, row0, step, col0, src, rows, K);
     return ok(cudaGetLastError());
 }
 
@@ -283,10 +313,11 @@ int lm_fill_random(uint16_t *dst, size_t n, uint32_t seed, float mean, float sca
     return ok(cudaGetLastError());
 }
 
-int lm_gemm_f32(float *y, int ld_out, const float *x, int ldx, const uint16_t *W, int ldw, int M, int N, int K, bool swiglu,
-                cudaStream_t st) {
+int lm_gemm_f32(float *y, int ld_out, const float *x, int ldx, const uint16_t *W, int ldw, int M, int N, int K, LmAct act,
+                cudaStream_t st, const int4 *table, int group_rows) {
     const dim3 g((N + kFgT - 1) / kFgT, (M + kFgT - 1) / kFgT);
-    return ok(launch_pdl(lm_gemm_f32_kernel, g, dim3(256), 0, st, y, ld_out, x, ldx, W, ldw, M, N, K, swiglu ? 1 : 0));
+    return ok(launch_pdl(lm_gemm_f32_kernel, g, dim3(256), 0, st, y, ld_out, x, ldx, W, ldw, M, N, K, (int)act,
+                         table, group_rows));
 }
 
 int lm_argmax_advance(LmDyn *dyn, int *tokens, int *log, int log_cap, LmPart logits, int vocab, int rows, cudaStream_t st) {

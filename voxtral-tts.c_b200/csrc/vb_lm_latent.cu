@@ -1,0 +1,687 @@
+/*
+ * vb_lm_latent.cu - decoder language models: attention over a latent cache. A token leaves one
+ * normed latent and one rotated key part, shared by all heads; keys and values are linear in the
+ * latent, so that with few rows the key matrix is applied to the query instead (absorb), all heads
+ * attend over the same cache rows (attend), and the value matrix is applied to what they read
+ * (readout, with the gate per head). Prompts write keys and values out (gather, a GEMM) and use
+ * the attention of vb_lm_attn.cu.
+ *
+ *   lm_latent_prepare  norms of both latents, rotated key part, cache append, gates, angles, routing,
+ *                      squared-ReLU columns of a feed-forward that shares the in-projection
+ *   lm_latent_attend   mma.sync on hi + lo BF16 halves (cache rows as such halves), or fp32 pipes for
+ *                      other sizes and the 32-bit mode; key splits, merged by the readout
+ */
+#include "vb_lm_attn.cuh"
+#include "vb_tc.cuh"
+
+namespace vb {
+
+namespace {
+
+inline int ok(cudaError_t e) { return e == cudaSuccess ? 0 : -1; }
+
+template <typename K> int allow_smem(K *kernel, size_t smem, size_t *set) {
+    if (smem <= *set) return 0;
+    if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+        cudaGetLastError();
+        return -1;
+    }
+    *set = smem;
+    return 0;
+}
+
+__host__ __device__ constexpr int up4(int v) { return (v + 3) & ~3; }
+constexpr size_t kSmemLimit = 216 * 1024;      /* dynamic part; a few KB are static */
+
+/* ------------------------------------------------------------------ a row's latents */
+constexpr int kLpThreads = 512, kLpWarps = kLpThreads / 32;
+
+/* The `top` largest of z[0, n), the first one on a tie, and the softmax over them: one warp. */
+VB_DEVINL void route_row(const float *z, int n, int top, int *chosen, float *weight, int lane) {
+    unsigned taken = 0;                      /* bit i: z[lane + 32 * i] */
+    float first = 0.0f, sum = 0.0f;
+    for (int k = 0; k < top; k++) {
+        float best = -INFINITY;
+        int bi = 0x7fffffff;
+        for (int i = 0, e = lane; e < n; i++, e += 32)
+            if (!((taken >> i) & 1u) && (bi == 0x7fffffff || z[e] > best)) { best = z[e]; bi = e; }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+            if (bi == 0x7fffffff || (oi != 0x7fffffff && (ov > best || (!(ov < best) && oi < bi)))) { best = ov; bi = oi; }
+        }
+        bi = __shfl_sync(0xffffffffu, bi, 0);
+        best = __shfl_sync(0xffffffffu, best, 0);
+        if ((bi & 31) == lane) taken |= 1u << (bi >> 5);
+        if (k == 0) first = best;
+        const float p = expf(best - first);
+        sum += p;
+        if (lane == 0) { chosen[k] = bi; weight[k] = p; }
+    }
+    if (lane == 0)
+        for (int k = 0; k < top; k++) weight[k] /= sum;
+}
+
+/* grid = (rows, 1 + pieces of the feed-forward columns) */
+__global__ void __launch_bounds__(kLpThreads) lm_latent_prepare_kernel(const LmLatent a) {
+    extern __shared__ __align__(16) float lp[];
+    __shared__ float red[2][kLpWarps];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int m = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    if (blockIdx.y > 0) {
+        const int c = (((int)blockIdx.y - 1) * kLpThreads + tid) * 4;
+        if (c >= a.ff) return;
+        const float4 v = lm_sum4(a.in, m, a.col_ff + c);
+        float e[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (int i = 0; i < 4; i++) { e[i] = fmaxf(e[i], 0.0f); e[i] *= e[i]; }
+        if (c + 3 < a.ff) {
+            lm_put4(a.out, m, a.ff_out + c, e);
+        } else {
+            for (int i = 0; c + i < a.ff; i++) lm_put(a.out, m, a.ff_out + c + i, e[i]);
+        }
+        return;
+    }
+    const int half = a.rot / 2, row = a.rank + a.rot_dim, nq = up4(a.q_rank), nc = a.c_gain ? up4(row) : 0;
+    float *ql = lp, *cl = ql + nq, *z = cl + nc, *cs = z + a.experts;
+    const int pos = a.dyn->pos + m;
+    for (int i = tid; i < half; i += kLpThreads) {
+        float c, s;
+        lm_angle(pos, a.freq[i], a.freq[half + i], a.mag, &c, &s);
+        cs[i] = c;
+        cs[half + i] = s;
+        a.cs[(size_t)m * a.rot + i] = c;
+        a.cs[(size_t)m * a.rot + half + i] = s;
+    }
+    /* a part that does not fill its last four columns is followed by zero ones */
+    float sq = 0.0f, sc = 0.0f;
+    for (int c = tid * 4; c < nq + nc; c += kLpThreads * 4) {
+        const bool isq = c < nq;
+        const float4 v = lm_sum4(a.in, m, isq ? c : a.col_c + c - nq);
+        *reinterpret_cast<float4 *>(lp + c) = v;
+        if (isq) {
+            sq += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        } else {
+            const int d = c - nq;
+            sc += (d < a.rank ? v.x * v.x : 0.0f) + (d + 1 < a.rank ? v.y * v.y : 0.0f) + (d + 2 < a.rank ? v.z * v.z : 0.0f) +
+                  (d + 3 < a.rank ? v.w * v.w : 0.0f);
+        }
+    }
+    for (int e = tid; e < a.experts; e += kLpThreads) z[e] = lm_sum_batch(a.in, m, a.col_router + e);
+    for (int h = tid; h < a.heads; h += kLpThreads)
+        a.gate[(size_t)m * a.heads + h] = 1.0f / (1.0f + expf(-lm_sum_batch(a.in, m, a.col_g + h)));
+    sq = vb_warp_sum(sq);
+    sc = vb_warp_sum(sc);
+    if (lane == 0) { red[0][warp] = sq; red[1][warp] = sc; }
+    __syncthreads();
+    sq = sc = 0.0f;
+#pragma unroll
+    for (int w = 0; w < kLpWarps; w++) { sq += red[0][w]; sc += red[1][w]; }
+    const float rq = 1.0f / sqrtf(sq / (float)a.q_rank + a.eps), rc = 1.0f / sqrtf(sc / (float)a.rank + a.eps);
+    if ((a.q_rank & 3) == 0) {
+        for (int c = tid * 4; c < a.q_rank; c += kLpThreads * 4) {
+            const float4 g = __ldg(reinterpret_cast<const float4 *>(a.q_gain + c));
+            const float e[4] = {ql[c] * rq * g.x, ql[c + 1] * rq * g.y, ql[c + 2] * rq * g.z, ql[c + 3] * rq * g.w};
+            lm_put4(a.q_latent, m, c, e);
+        }
+    } else {
+        for (int c = tid; c < a.q_rank; c += kLpThreads) lm_put(a.q_latent, m, c, ql[c] * rq * __ldg(a.q_gain + c));
+    }
+    if (a.c_gain) {
+        float *dst = lm_state(a.kv, a.dyn) + (size_t)lm_ring_row(a.ring, pos) * row;
+        auto value = [&](int d) {
+            if (d < a.rank) return cl[d] * rc * __ldg(a.c_gain + d);
+            const int j = d - a.rank, i = j >> 1;
+            if (j >= a.rot) return cl[d];
+            return (j & 1) ? cl[d] * cs[i] + cl[d - 1] * cs[half + i] : cl[d] * cs[i] - cl[d + 1] * cs[half + i];
+        };
+        if ((row & 3) == 0) {
+            for (int d = tid * 4; d < row; d += kLpThreads * 4)
+                kv_put4(dst, row, d, make_float4(value(d), value(d + 1), value(d + 2), value(d + 3)), a.split);
+        } else {
+            for (int d = tid; d < row; d += kLpThreads) kv_put(dst, row, d, value(d), a.split);
+        }
+    }
+    if (a.experts > 0 && warp == kLpWarps - 1)
+        route_row(z, a.experts, a.top, a.chosen + (size_t)m * a.top, a.weight + (size_t)m * a.top, lane);
+}
+
+/* ------------------------------------------------------------------ queries into the latent's space */
+constexpr int kLtThreads = 256, kLtWarps = 8;
+
+VB_DEVINL void bf16x8(const uint4 &u, float (&f)[8]) {
+    f[0] = vb_bf16_lo(u.x); f[1] = vb_bf16_hi(u.x); f[2] = vb_bf16_lo(u.y); f[3] = vb_bf16_hi(u.y);
+    f[4] = vb_bf16_lo(u.z); f[5] = vb_bf16_hi(u.z); f[6] = vb_bf16_lo(u.w); f[7] = vb_bf16_hi(u.w);
+}
+
+/* ql[m][h][r] = sum over d of q[m][h][d] * W_key[h * dim + d][r]; the rotated part follows. grid = (heads, 64-column
+ * blocks of the latent, MR-row blocks). Eight lanes share a 128-byte piece of a weight row; the weights of the first
+ * kPre steps are requested before the previous kernel has ended. */
+template <int MR>
+__global__ void __launch_bounds__(kLtThreads) lm_latent_absorb_kernel(const LmLatent a, int M) {
+    extern __shared__ __align__(16) float ab[];
+    __shared__ float red[kLtWarps][MR][64];
+    constexpr int kPre = 4;
+    const int h = blockIdx.x, kb = blockIdx.y, m0 = blockIdx.z * MR, nr = M - m0 < MR ? M - m0 : MR;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int d0 = warp * 4 + (lane >> 3), c0 = (lane & 7) * 8;
+    pdl_launch_dependents();
+    uint4 pre[kPre];
+#pragma unroll
+    for (int i = 0; i < kPre; i++) {
+        const int d = d0 + i * 32;
+        pre[i] = d < a.dim ? __ldg(reinterpret_cast<const uint4 *>(lm_weight_row(a.ukv, h * a.dim + d, kb) + c0)) : make_uint4(0u, 0u, 0u, 0u);
+    }
+    pdl_wait();
+    const int hw = a.dim + a.rot_dim, row = a.rank + a.rot_dim;
+    for (int i = tid; i < MR * a.dim; i += kLtThreads) {
+        const int r = i / a.dim, d = i % a.dim;
+        ab[i] = r < nr ? lm_sum_batch(a.q, m0 + r, h * hw + d) : 0.0f;
+    }
+    if (kb == 0) {
+        const int half = a.rot / 2;
+        for (int i = tid; i < nr * a.rot_dim; i += kLtThreads) {
+            const int r = i / a.rot_dim, j = i % a.rot_dim, m = m0 + r, k = j >> 1;
+            float v = lm_sum_batch(a.q, m, h * hw + a.dim + j);
+            if (j < a.rot) {
+                const float u = lm_sum_batch(a.q, m, h * hw + a.dim + (j ^ 1));
+                const float c = a.cs[(size_t)m * a.rot + k], s = a.cs[(size_t)m * a.rot + half + k];
+                v = (j & 1) ? v * c + u * s : v * c - u * s;
+            }
+            a.ql[((size_t)m * a.heads + h) * row + a.rank + j] = v;
+        }
+    }
+    __syncthreads();
+    float acc[MR][8];
+#pragma unroll
+    for (int r = 0; r < MR; r++)
+#pragma unroll
+        for (int j = 0; j < 8; j++) acc[r][j] = 0.0f;
+    auto add = [&](const uint4 &u, int d) {
+        float w[8];
+        bf16x8(u, w);
+#pragma unroll
+        for (int r = 0; r < MR; r++) {
+            const float q = ab[r * a.dim + d];
+#pragma unroll
+            for (int j = 0; j < 8; j++) acc[r][j] = fmaf(q, w[j], acc[r][j]);
+        }
+    };
+#pragma unroll
+    for (int i = 0; i < kPre; i++)
+        if (d0 + i * 32 < a.dim) add(pre[i], d0 + i * 32);
+    for (int d = d0 + kPre * 32; d < a.dim; d += 32)
+        add(__ldg(reinterpret_cast<const uint4 *>(lm_weight_row(a.ukv, h * a.dim + d, kb) + c0)), d);
+#pragma unroll
+    for (int r = 0; r < MR; r++)
+#pragma unroll
+        for (int j = 0; j < 8; j++) {
+            float v = acc[r][j];
+            v += __shfl_xor_sync(0xffffffffu, v, 8);
+            v += __shfl_xor_sync(0xffffffffu, v, 16);
+            if (lane < 8) red[warp][r][c0 + j] = v;
+        }
+    __syncthreads();
+    for (int i = tid; i < nr * 64; i += kLtThreads) {
+        const int r = i >> 6, c = i & 63, col = kb * 64 + c;
+        if (col >= a.rank) continue;
+        float v = 0.0f;
+#pragma unroll
+        for (int w = 0; w < kLtWarps; w++) v += red[w][r][c];
+        a.ql[((size_t)(m0 + r) * a.heads + h) * row + col] = v;
+    }
+}
+
+/* ------------------------------------------------------------------ attention over cache rows */
+constexpr int kLaPairs = kLmLatentPairs, kLaSplits = 64, kLaBudget = 148;
+
+inline int attend_tiles(int M, int heads) { return (M * heads + kLaPairs - 1) / kLaPairs; }
+inline int attend_splits(int M, int heads) {
+    const int s = kLaBudget / attend_tiles(M, heads);
+    return s < 1 ? 1 : s > kLaSplits ? kLaSplits : s;
+}
+
+/* Key tiles of pairs p0 .. p0 + np - 1 (pair = row * heads + head). */
+template <int KT>
+VB_DEVINL KeyTiles pair_tiles(const LmLatent &a, int M, int p0, int *np) {
+    const int P = M * a.heads, pos0 = a.dyn->pos;
+    *np = P - p0 < kLaPairs ? P - p0 : kLaPairs;
+    return key_tiles<KT>(pos0 + p0 / a.heads, pos0 + (p0 + *np - 1) / a.heads, a.window, 0);
+}
+
+constexpr int kLaKeys = 32;
+
+struct AttendSmem {
+    int row_bytes;               /* of a query or key row in one plane: whole 64-element groups */
+    size_t q, k, total;
+    int stages;
+};
+inline AttendSmem attend_smem(int rank, int rot_dim) {
+    AttendSmem s;
+    s.row_bytes = (rank + rot_dim + 63) / 64 * 128;
+    s.q = (size_t)2 * kLaPairs * s.row_bytes;
+    s.k = (size_t)2 * kLaKeys * s.row_bytes;
+    s.stages = s.q + 2 * s.k <= kSmemLimit ? 2 : 1;
+    s.total = s.q + s.stages * s.k;
+    return s;
+}
+
+/* A CTA attends with 16 (row, head) pairs over its share of the visible cache rows, 32 at a time. Scores: a warp takes
+ * eight keys and half of the columns; values: a warp takes every eighth 16-column step. Products a.b as
+ * a_hi.b_hi + a_hi.b_lo + a_lo.b_hi, accumulated in fp32. ND: value steps per warp. grid = (pair tiles, splits) */
+template <int ND>
+__global__ void __launch_bounds__(kLtThreads) lm_latent_attend_kernel(const LmLatent a, int M, int row_bytes, int stages) {
+    extern __shared__ __align__(128) unsigned char at_smem[];
+    __shared__ float S[2][kLaPairs][kLaKeys + 1], mx[kLaPairs], den[kLaPairs], cor[kLaPairs];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, tq = lane & 3;
+    const int q_plane = kLaPairs * row_bytes, k_plane = kLaKeys * row_bytes;
+    unsigned char *Kb = at_smem + 2 * q_plane;
+    pdl_launch_dependents();
+    for (int i = tid; i < (2 * q_plane + stages * 2 * k_plane) / 16; i += kLtThreads)
+        reinterpret_cast<uint4 *>(at_smem)[i] = make_uint4(0u, 0u, 0u, 0u);
+    pdl_wait();
+    int np;
+    const int p0 = blockIdx.x * kLaPairs, sp = blockIdx.y;
+    const KeyTiles kt = pair_tiles<kLaKeys>(a, M, p0, &np);
+    const int S_eff = (int)gridDim.y < kt.n_tiles ? (int)gridDim.y : kt.n_tiles;
+    if (sp >= S_eff) return;
+    const int t0 = (int)((long long)kt.n_tiles * sp / S_eff), t1 = (int)((long long)kt.n_tiles * (sp + 1) / S_eff);
+    const int row = a.rank + a.rot_dim, pos0 = a.dyn->pos, P = M * a.heads;
+    const float *cache = lm_state(a.kv, a.dyn);
+    __syncthreads();
+    auto swz = [&](int r, int chunk) { return (uint32_t)(r * row_bytes + (((chunk & ~7) | ((chunk ^ r) & 7)) << 4)); };
+    auto request = [&](int t) {
+        int j0, n;
+        key_tile<kLaKeys>(kt, t, &j0, &n);
+        unsigned char *b = Kb + (stages == 2 ? (t & 1) : 0) * 2 * k_plane;
+        const int per = row / 8;
+        for (int i = tid; i < n * 2 * per; i += kLtThreads) {
+            const int key = i / (2 * per), f = i % (2 * per), plane = f >= per ? 1 : 0, chunk = f - plane * per;
+            lm_cp16(b + plane * k_plane + swz(key, chunk),
+                    reinterpret_cast<const uint16_t *>(cache + (size_t)lm_ring_row(a.ring, j0 + key) * row) + f * 8);
+        }
+        lm_cp_commit();
+    };
+    request(t0);
+    for (int i = tid; i < np * (row / 8); i += kLtThreads) {
+        const int p = i / (row / 8), chunk = i % (row / 8);
+        const float *q = a.ql + (size_t)(p0 + p) * row + chunk * 8;
+        const float4 u = vb_ldcg4(q), v = vb_ldcg4(q + 4);
+        const float e[8] = {u.x, u.y, u.z, u.w, v.x, v.y, v.z, v.w};
+        uint32_t hi[8], lo[8];
+#pragma unroll
+        for (int j = 0; j < 8; j++) hilo(e[j], hi[j], lo[j]);
+        unsigned char *o = at_smem + swz(p, chunk);
+        *reinterpret_cast<uint4 *>(o) = make_uint4(hi[0] | (hi[1] << 16), hi[2] | (hi[3] << 16), hi[4] | (hi[5] << 16), hi[6] | (hi[7] << 16));
+        *reinterpret_cast<uint4 *>(o + q_plane) = make_uint4(lo[0] | (lo[1] << 16), lo[2] | (lo[3] << 16), lo[4] | (lo[5] << 16), lo[6] | (lo[7] << 16));
+    }
+    if (tid < kLaPairs) { mx[tid] = -INFINITY; den[tid] = 0.0f; }
+    float o[2 * ND][4];
+#pragma unroll
+    for (int i = 0; i < 2 * ND; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
+    const int steps = row_bytes / 32, vsteps = (a.rank + 15) / 16;
+    const int nt = warp & 3, kh = warp >> 2, mat = lane >> 3, mr = lane & 7;
+    const uint32_t sQ = vb_smem_u32(at_smem);
+
+    for (int t = t0; t < t1; t++) {
+        int j0, n;
+        key_tile<kLaKeys>(kt, t, &j0, &n);
+        if (stages == 1 && t > t0) {
+            __syncthreads();
+            request(t);
+        }
+        lm_cp_wait_all();
+        __syncthreads();
+        if (stages == 2 && t + 1 < t1) request(t + 1);
+        const uint32_t sK = vb_smem_u32(Kb + (stages == 2 ? (t & 1) : 0) * 2 * k_plane);
+        float s0[4] = {}, s1[4] = {}, s2[4] = {};
+#pragma unroll 4
+        for (int ks = kh * steps / 2; ks < (kh + 1) * steps / 2; ks++) {
+            uint32_t qh[4], ql[4], b[4];
+            const uint32_t qo = swz((lane & 7) + ((lane >> 3) & 1) * 8, ks * 2 + (lane >> 4));
+            ldsm(qh, sQ + qo);
+            ldsm(ql, sQ + q_plane + qo);
+            ldsm(b, sK + (mat >> 1) * k_plane + swz(nt * 8 + mr, ks * 2 + (mat & 1)));     /* high halves, low halves */
+            mma_bf16(s0, qh, b[0], b[1]);
+            mma_bf16(s1, qh, b[2], b[3]);
+            mma_bf16(s2, ql, b[0], b[1]);
+        }
+#pragma unroll
+        for (int c = 0; c < 4; c++) S[kh][gq + (c >> 1) * 8][nt * 8 + 2 * tq + (c & 1)] = s0[c] + (s1[c] + s2[c]);
+        __syncthreads();
+#pragma unroll
+        for (int rr = 0; rr < 2; rr++) {
+            const int p = warp * 2 + rr, pc = p0 + p < P ? p0 + p : P - 1;
+            const int i = pos0 + pc / a.heads;
+            float s = (S[0][p][lane] + S[1][p][lane]) * a.scale;
+            if (lane >= n || !key_seen(i, j0 + lane, a.window, 0)) s = -INFINITY;
+            float top = s;
+#pragma unroll
+            for (int off = 16; off > 0; off >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, off));
+            const float old = mx[p], now = fmaxf(old, top), ref = now > -INFINITY ? now : 0.0f;
+            const float w = expf(s - ref);
+            const float sum = vb_warp_sum(w);
+            S[0][p][lane] = w;
+            __syncwarp();
+            if (lane == 0) {
+                const float c = expf(old - ref);
+                cor[p] = c;
+                mx[p] = now;
+                den[p] = den[p] * c + sum;
+            }
+        }
+        __syncthreads();
+        uint32_t ph[2][4], pl[2][4];
+#pragma unroll
+        for (int kp = 0; kp < 2; kp++)
+#pragma unroll
+            for (int x = 0; x < 4; x++) {
+                const float *w = &S[0][gq + (x & 1) * 8][kp * 16 + (x >> 1) * 8 + 2 * tq];
+                uint32_t h0, l0, h1, l1;
+                hilo(w[0], h0, l0);
+                hilo(w[1], h1, l1);
+                ph[kp][x] = h0 | (h1 << 16);
+                pl[kp][x] = l0 | (l1 << 16);
+            }
+        const float cA = cor[gq], cB = cor[gq + 8];
+#pragma unroll
+        for (int i = 0; i < ND; i++) {
+            const int dp = warp + i * kLtWarps;
+            if (dp >= vsteps) break;
+#pragma unroll
+            for (int u = 0; u < 2; u++) { o[2 * i + u][0] *= cA; o[2 * i + u][1] *= cA; o[2 * i + u][2] *= cB; o[2 * i + u][3] *= cB; }
+#pragma unroll
+            for (int kp = 0; kp < 2; kp++) {
+                const uint32_t off = swz(kp * 16 + (mat & 1) * 8 + mr, dp * 2 + (mat >> 1));
+                uint32_t vh[4], vl[4];
+                ldsm_t(vh, sK + off);
+                ldsm_t(vl, sK + k_plane + off);
+                mma_bf16(o[2 * i], ph[kp], vh[0], vh[1]);
+                mma_bf16(o[2 * i + 1], ph[kp], vh[2], vh[3]);
+                mma_bf16(o[2 * i], ph[kp], vl[0], vl[1]);
+                mma_bf16(o[2 * i + 1], ph[kp], vl[2], vl[3]);
+                mma_bf16(o[2 * i], pl[kp], vh[0], vh[1]);
+                mma_bf16(o[2 * i + 1], pl[kp], vh[2], vh[3]);
+            }
+        }
+    }
+    /* (the last statistics were written before the barrier ahead of the value products) */
+    float *out = a.scratch + ((size_t)sp * P + p0) * (a.rank + 2);
+#pragma unroll
+    for (int i = 0; i < ND; i++) {
+        const int dp = warp + i * kLtWarps;
+#pragma unroll
+        for (int u = 0; u < 2; u++) {
+            const int c = dp * 16 + u * 8 + 2 * tq;
+            if (c >= a.rank) continue;
+            if (gq < np) *reinterpret_cast<float2 *>(out + (size_t)gq * (a.rank + 2) + c) = make_float2(o[2 * i + u][0], o[2 * i + u][1]);
+            if (gq + 8 < np) *reinterpret_cast<float2 *>(out + (size_t)(gq + 8) * (a.rank + 2) + c) = make_float2(o[2 * i + u][2], o[2 * i + u][3]);
+        }
+    }
+    if (tid < np) {
+        out[(size_t)tid * (a.rank + 2) + a.rank] = mx[tid];
+        out[(size_t)tid * (a.rank + 2) + a.rank + 1] = den[tid];
+    }
+}
+
+/* The same on the fp32 pipes, any sizes; cache rows in either form. */
+inline size_t attend_f32_smem(int rank, int rot_dim, int keys) {
+    const size_t row = (size_t)rank + rot_dim;
+    return sizeof(float) * (kLaPairs * row + keys * (row + 1) + kLaPairs * (size_t)rank + kLaPairs * (keys + 1) + 3 * kLaPairs);
+}
+inline int attend_f32_keys(int rank, int rot_dim) { return attend_f32_smem(rank, rot_dim, 32) <= kSmemLimit ? 32 : 8; }
+
+template <int KT>
+__global__ void __launch_bounds__(kLtThreads) lm_latent_attend_f32_kernel(const LmLatent a, int M) {
+    extern __shared__ __align__(16) float af[];
+    pdl_launch_dependents();
+    pdl_wait();
+    int np;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int p0 = blockIdx.x * kLaPairs, sp = blockIdx.y, row = a.rank + a.rot_dim, pos0 = a.dyn->pos, P = M * a.heads;
+    const KeyTiles kt = pair_tiles<KT>(a, M, p0, &np);
+    const int S_eff = (int)gridDim.y < kt.n_tiles ? (int)gridDim.y : kt.n_tiles;
+    if (sp >= S_eff) return;
+    const int t0 = (int)((long long)kt.n_tiles * sp / S_eff), t1 = (int)((long long)kt.n_tiles * (sp + 1) / S_eff);
+    float *Q = af, *K = Q + kLaPairs * row, *O = K + KT * (row + 1), *S = O + kLaPairs * a.rank, *mx = S + kLaPairs * (KT + 1),
+          *den = mx + kLaPairs, *cor = den + kLaPairs;
+    const float *cache = lm_state(a.kv, a.dyn);
+    for (int i = tid; i < np * row; i += kLtThreads) Q[i] = __ldcg(a.ql + (size_t)p0 * row + i);
+    for (int i = tid; i < np * a.rank; i += kLtThreads) O[i] = 0.0f;
+    if (tid < kLaPairs) { mx[tid] = -INFINITY; den[tid] = 0.0f; }
+    for (int t = t0; t < t1; t++) {
+        int j0, n;
+        key_tile<KT>(kt, t, &j0, &n);
+        __syncthreads();
+        for (int i = tid; i < n * row; i += kLtThreads) {
+            const int j = i / row, d = i % row;
+            K[j * (row + 1) + d] = kv_get(cache + (size_t)lm_ring_row(a.ring, j0 + j) * row, row, d, a.split);
+        }
+        __syncthreads();
+        for (int p = warp; p < np; p += kLtWarps) {
+            const int i = pos0 + (p0 + p) / a.heads;
+            float s = -INFINITY;
+            if (lane < n && key_seen(i, j0 + lane, a.window, 0)) {
+                const float *q = Q + p * row, *k = K + lane * (row + 1);
+                float e0 = 0.0f, e1 = 0.0f, e2 = 0.0f, e3 = 0.0f;
+                int d = 0;
+                for (; d + 3 < row; d += 4) {
+                    e0 = fmaf(q[d], k[d], e0);
+                    e1 = fmaf(q[d + 1], k[d + 1], e1);
+                    e2 = fmaf(q[d + 2], k[d + 2], e2);
+                    e3 = fmaf(q[d + 3], k[d + 3], e3);
+                }
+                for (; d < row; d++) e0 = fmaf(q[d], k[d], e0);
+                s = ((e0 + e1) + (e2 + e3)) * a.scale;
+            }
+            float top = s;
+#pragma unroll
+            for (int off = 16; off > 0; off >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, off));
+            const float old = mx[p], now = fmaxf(old, top), ref = now > -INFINITY ? now : 0.0f;
+            const float w = expf(s - ref);
+            const float sum = vb_warp_sum(w);
+            if (lane < KT) S[p * (KT + 1) + lane] = w;
+            __syncwarp();
+            if (lane == 0) {
+                const float c = expf(old - ref);
+                cor[p] = c;
+                mx[p] = now;
+                den[p] = den[p] * c + sum;
+            }
+        }
+        __syncthreads();
+        for (int i = tid; i < np * a.rank; i += kLtThreads) {
+            const int p = i / a.rank, d = i % a.rank;
+            float o = O[i] * cor[p];
+            for (int j = 0; j < n; j++) o = fmaf(S[p * (KT + 1) + j], K[j * (row + 1) + d], o);
+            O[i] = o;
+        }
+    }
+    __syncthreads();
+    float *out = a.scratch + ((size_t)sp * P + p0) * (a.rank + 2);
+    for (int i = tid; i < np * a.rank; i += kLtThreads) out[(size_t)(i / a.rank) * (a.rank + 2) + i % a.rank] = O[i];
+    if (tid < np) {
+        out[(size_t)tid * (a.rank + 2) + a.rank] = mx[tid];
+        out[(size_t)tid * (a.rank + 2) + a.rank + 1] = den[tid];
+    }
+}
+
+/* ------------------------------------------------------------------ values */
+/* Merges the key splits of a head (in order), applies its value matrix and its gate. grid = (heads, 32-row blocks of the
+ * value matrix, MR-row blocks). KT: keys per tile of the kernel that wrote the splits. */
+template <int MR, int KT>
+__global__ void __launch_bounds__(kLtThreads) lm_latent_readout_kernel(const LmLatent a, int M, int splits) {
+    extern __shared__ __align__(16) float ro[];                /* [MR][rank, padded to 64] */
+    __shared__ float wgt[MR][kLaSplits];
+    __shared__ int count[MR];
+    constexpr int kPre = MR == 1 ? 8 : 1;
+    const int h = blockIdx.x, m0 = blockIdx.z * MR, nr = M - m0 < MR ? M - m0 : MR;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int v = blockIdx.y * 32 + warp * 4 + (lane >> 3), c0 = (lane & 7) * 8;
+    const int kblocks = (a.rank + 63) / 64, rp = kblocks * 64;
+    const int wrow = a.heads * a.dim + h * a.vdim + (v < a.vdim ? v : 0);
+    pdl_launch_dependents();
+    uint4 pre[kPre];
+#pragma unroll
+    for (int i = 0; i < kPre; i++)
+        pre[i] = i < kblocks ? __ldg(reinterpret_cast<const uint4 *>(lm_weight_row(a.ukv, wrow, i) + c0)) : make_uint4(0u, 0u, 0u, 0u);
+    pdl_wait();
+    const int stride = a.rank + 2;
+    const size_t P = (size_t)M * a.heads;
+    if (warp < nr) {
+        const int p = (m0 + warp) * a.heads + h;
+        int np;
+        const KeyTiles kt = pair_tiles<KT>(a, M, p / kLaPairs * kLaPairs, &np);
+        const int S = splits < kt.n_tiles ? splits : kt.n_tiles;
+        float mu[2], top = -INFINITY, L = 0.0f;
+#pragma unroll
+        for (int x = 0; x < 2; x++) {
+            const int u = lane + 32 * x;
+            mu[x] = u < S ? __ldcg(a.scratch + (u * P + p) * stride + a.rank) : -INFINITY;
+            top = fmaxf(top, mu[x]);
+        }
+#pragma unroll
+        for (int off = 16; off > 0; off >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, off));
+#pragma unroll
+        for (int x = 0; x < 2; x++) {
+            const int u = lane + 32 * x;
+            mu[x] = u < S ? expf(mu[x] - top) : 0.0f;          /* a row always sees itself: top is finite */
+            if (u < S) L = fmaf(mu[x], __ldcg(a.scratch + (u * P + p) * stride + a.rank + 1), L);
+        }
+        L = vb_warp_sum(L);
+        wgt[warp][lane] = mu[0] / L;
+        wgt[warp][lane + 32] = mu[1] / L;
+        if (lane == 0) count[warp] = S;
+    }
+    __syncthreads();
+    for (int i = tid; i < nr * rp; i += kLtThreads) {
+        const int r = i / rp, c = i % rp;
+        float o = 0.0f;
+        if (c < a.rank) {
+            const float *s = a.scratch + ((size_t)(m0 + r) * a.heads + h) * stride + c;
+            const int S = count[r];
+#pragma unroll 8
+            for (int u = 0; u < S; u++) o = fmaf(wgt[r][u], __ldcg(s + u * P * stride), o);
+        }
+        ro[i] = o;
+    }
+    __syncthreads();
+    float acc[MR];
+#pragma unroll
+    for (int r = 0; r < MR; r++) acc[r] = 0.0f;
+    auto add = [&](const uint4 &u, int kb) {
+        float w[8];
+        bf16x8(u, w);
+#pragma unroll
+        for (int r = 0; r < MR; r++) {
+            if (r >= nr) break;
+            const float *x = ro + r * rp + kb * 64 + c0;
+#pragma unroll
+            for (int j = 0; j < 8; j++) acc[r] = fmaf(w[j], x[j], acc[r]);
+        }
+    };
+#pragma unroll
+    for (int i = 0; i < kPre; i++)
+        if (i < kblocks) add(pre[i], i);
+    for (int kb = kPre; kb < kblocks; kb++) add(__ldg(reinterpret_cast<const uint4 *>(lm_weight_row(a.ukv, wrow, kb) + c0)), kb);
+#pragma unroll
+    for (int r = 0; r < MR; r++) {
+#pragma unroll
+        for (int off = 4; off > 0; off >>= 1) acc[r] += __shfl_xor_sync(0xffffffffu, acc[r], off);
+        if (r < nr && (lane & 7) == 0 && v < a.vdim)
+            lm_put(a.out, m0 + r, h * a.vdim + v, acc[r] * a.gate[(size_t)(m0 + r) * a.heads + h]);
+    }
+}
+
+/* ------------------------------------------------------------------ latents of a stretch as GEMM rows */
+__global__ void lm_latent_gather_kernel(const LmLatent a, uint16_t *terms, int rows_pad, int ld, int first, int n) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int per = a.rank / 8, row = a.rank + a.rot_dim;
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= (size_t)n * 2 * per) return;
+    const int j = (int)(i / (2 * per)), f = (int)(i % (2 * per)), plane = f >= per ? 1 : 0, chunk = f - plane * per;
+    const uint16_t *src = reinterpret_cast<const uint16_t *>(lm_state(a.kv, a.dyn) + (size_t)lm_ring_row(a.ring, first + j) * row) +
+                          (size_t)plane * row + chunk * 8;
+    *reinterpret_cast<uint4 *>(terms + ((size_t)plane * rows_pad + j) * ld + chunk * 8) = __ldcg(reinterpret_cast<const uint4 *>(src));
+}
+
+template <int ND>
+int launch_attend(const LmLatent &a, int M, const AttendSmem &s, cudaStream_t st) {
+    static size_t set = 32 * 1024;
+    if (allow_smem(lm_latent_attend_kernel<ND>, s.total, &set)) return -1;
+    return ok(launch_pdl(lm_latent_attend_kernel<ND>, dim3(attend_tiles(M, a.heads), attend_splits(M, a.heads)), dim3(kLtThreads), s.total, st, a, M,
+                         s.row_bytes, s.stages));
+}
+template <int KT>
+int launch_attend_f32(const LmLatent &a, int M, cudaStream_t st) {
+    static size_t set = 32 * 1024;
+    const size_t smem = attend_f32_smem(a.rank, a.rot_dim, KT);
+    if (allow_smem(lm_latent_attend_f32_kernel<KT>, smem, &set)) return -1;
+    return ok(launch_pdl(lm_latent_attend_f32_kernel<KT>, dim3(attend_tiles(M, a.heads), attend_splits(M, a.heads)), dim3(kLtThreads), smem, st, a, M));
+}
+template <int MR, int KT>
+int launch_readout(const LmLatent &a, int M, cudaStream_t st) {
+    static size_t set = 32 * 1024;
+    const size_t smem = sizeof(float) * MR * ((a.rank + 63) / 64 * 64);
+    if (allow_smem(lm_latent_readout_kernel<MR, KT>, smem, &set)) return -1;
+    return ok(launch_pdl(lm_latent_readout_kernel<MR, KT>, dim3(a.heads, (a.vdim + 31) / 32, (M + MR - 1) / MR), dim3(kLtThreads), smem, st, a, M,
+                         attend_splits(M, a.heads)));
+}
+template <int MR>
+int launch_absorb(const LmLatent &a, int M, cudaStream_t st) {
+    static size_t set = 24 * 1024;
+    const size_t smem = sizeof(float) * MR * a.dim;
+    if (allow_smem(lm_latent_absorb_kernel<MR>, smem, &set)) return -1;
+    return ok(launch_pdl(lm_latent_absorb_kernel<MR>, dim3(a.heads, (a.rank + 63) / 64, (M + MR - 1) / MR), dim3(kLtThreads), smem, st, a, M));
+}
+
+} // namespace
+
+bool lm_latent_split_ok(int rank, int rot_dim) {
+    return rank % 8 == 0 && rot_dim % 8 == 0 && rank <= 1024 && attend_smem(rank, rot_dim).total <= kSmemLimit;
+}
+bool lm_latent_supported(int q_rank, int rank, int rot_dim) {
+    return attend_f32_smem(rank, rot_dim, attend_f32_keys(rank, rot_dim)) <= kSmemLimit &&
+           sizeof(float) * ((size_t)q_rank + rank + 2 * rot_dim + kLmMoeExperts + 16) <= kSmemLimit;
+}
+size_t lm_latent_scratch_floats(int rows, int heads, int rank) {
+    size_t n = 0;
+    for (int M = 1; M <= rows; M++) n = n > (size_t)attend_splits(M, heads) * M ? n : (size_t)attend_splits(M, heads) * M;
+    return n * heads * (rank + 2);
+}
+
+int lm_latent_prepare(const LmLatent &a, int M, cudaStream_t st) {
+    static size_t set = 40 * 1024;
+    const size_t smem = sizeof(float) * ((size_t)up4(a.q_rank) + (a.c_gain ? up4(a.rank + a.rot_dim) : 0) + a.experts + a.rot);
+    if (allow_smem(lm_latent_prepare_kernel, smem, &set)) return -1;
+    const int pieces = (a.ff + kLpThreads * 4 - 1) / (kLpThreads * 4);
+    return ok(launch_pdl(lm_latent_prepare_kernel, dim3(M, 1 + pieces), dim3(kLpThreads), smem, st, a));
+}
+
+int lm_latent_absorb(const LmLatent &a, int M, cudaStream_t st) { return M == 1 ? launch_absorb<1>(a, M, st) : launch_absorb<8>(a, M, st); }
+
+int lm_latent_attend(const LmLatent &a, int M, cudaStream_t st) {
+    if (a.split) {
+        const AttendSmem s = attend_smem(a.rank, a.rot_dim);
+        if (a.rank <= 128) return launch_attend<1>(a, M, s, st);
+        if (a.rank <= 256) return launch_attend<2>(a, M, s, st);
+        if (a.rank <= 512) return launch_attend<4>(a, M, s, st);
+        return launch_attend<8>(a, M, s, st);
+    }
+    return attend_f32_keys(a.rank, a.rot_dim) == 32 ? launch_attend_f32<32>(a, M, st) : launch_attend_f32<8>(a, M, st);
+}
+
+int lm_latent_readout(const LmLatent &a, int M, cudaStream_t st) {
+    if (a.split || attend_f32_keys(a.rank, a.rot_dim) == 32) return M == 1 ? launch_readout<1, 32>(a, M, st) : launch_readout<8, 32>(a, M, st);
+    return M == 1 ? launch_readout<1, 8>(a, M, st) : launch_readout<8, 8>(a, M, st);
+}
+
+int lm_latent_gather(const LmLatent &a, uint16_t *terms, int rows_pad, int ld, int first, int n, cudaStream_t st) {
+    const size_t items = (size_t)n * 2 * (a.rank / 8);
+    return ok(launch_pdl(lm_latent_gather_kernel, dim3((unsigned)((items + 255) / 256)), dim3(256), 0, st, a, terms, rows_pad, ld, first, n));
+}
+
+} // namespace vb

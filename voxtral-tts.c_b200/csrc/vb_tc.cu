@@ -140,6 +140,15 @@ int tc_acts(TcActs *a, uint16_t *d_buf, int rows_pad, int K) {
     return 0;
 }
 
+int tc_acts_blocks(TcActs *a, uint16_t *d_buf, int rows, int K) {
+    a->ok = false;
+    a->buf = d_buf; a->rows_pad = rows; a->K = K;
+    if (rows <= 0 || rows % 128 || (K % kTcBlockK) != 0) return -1;
+    if (make_map(&a->map_rows, d_buf, (uint64_t)2 * rows, (uint64_t)K, 128u)) return -1;
+    a->ok = true;
+    return 0;
+}
+
 int tc_pick_splits(int N, int K, int n_sm) {
     const int tiles = (N + kTcTileN - 1) / kTcTileN;
     int s = n_sm / tiles;
@@ -184,6 +193,7 @@ struct TcKernelArgs {
     int *status;
     int tile0;               /* first output tile of this launch */
     int n_tiles_launch;      /* tiles this launch covers (host side: the grid) */
+    int act_n0, out_terms_ld, out_col0;   /* row-block kernel: TC_EPI_TERMS, TC_EPI_RELU2_TERMS */
 };
 
 /* Tensor parallelism is a separate instantiation of every kernel that takes part in it, with
@@ -536,9 +546,20 @@ constexpr int kRbTmemCols = kRbTiles * kRbRows;
 constexpr int kRbSmemBytes = kRbStages * kRbStage + 1024 + 256 + 4 * kRbRows;
 static_assert(kRbSmemBytes <= 232448, "over the 227 KB a CTA may use");
 
+/* GROUPED: a row block belongs to one of several stacked weight matrices, looked up in device memory;
+ * N is the size of one of them. */
+struct TcGroupArgs {
+    const int4 *table;       /* {matrix or -1, first row, rows, unused} per row block */
+    int tiles;               /* 128-row tiles of one matrix */
+};
+struct TcNoGroupArgs {};
+template <bool GROUPED> struct TcGroupSel { using type = TcNoGroupArgs; };
+template <> struct TcGroupSel<true> { using type = TcGroupArgs; };
+
+template <bool GROUPED>
 __global__ void __launch_bounds__(kTcThreads, 1)
 vb_tc_rows_kernel(const __grid_constant__ CUtensorMap mapA, const __grid_constant__ CUtensorMap mapB,
-                  const TcKernelArgs ka) {
+                  const TcKernelArgs ka, const typename TcGroupSel<GROUPED>::type ga) {
     const int N = ka.N, K = ka.K, M = ka.M, rows_pad = ka.rows_pad, ld_out = ka.ld_out, splits = ka.splits,
               epi = ka.epi;
     float *const out = ka.out;
@@ -565,8 +586,17 @@ vb_tc_rows_kernel(const __grid_constant__ CUtensorMap mapA, const __grid_constan
     const int kblocks = K / kTcBlockK;
     const int kb0 = (int)((long long)kblocks * sp / splits), kb1 = (int)((long long)kblocks * (sp + 1) / splits);
     const int n_it = kb1 - kb0;
-    const int m0 = rb * kRbRows;
-    const int Mb = M - m0 < kRbRows ? M - m0 : kRbRows;
+    int m0 = rb * kRbRows;
+    int Mb = M - m0 < kRbRows ? M - m0 : kRbRows;
+    int w0 = t0;                 /* first weight tile of this CTA */
+    if constexpr (GROUPED) {
+        pdl_wait();              /* the table is made by an earlier kernel */
+        const int4 g = __ldcg(ga.table + rb);
+        if (g.x < 0) return;     /* the whole CTA: an unused row block */
+        m0 = g.y;
+        Mb = g.z;
+        w0 = g.x * ga.tiles + t0;
+    }
     const uint32_t stage_tx = (uint32_t)(nt * kRbStageW + kRbTerms * kRbStageX);
 
     if (threadIdx.x == 0) {
@@ -592,8 +622,8 @@ vb_tc_rows_kernel(const __grid_constant__ CUtensorMap mapA, const __grid_constan
         auto load_w = [&](int it, int s) {
             unsigned char *sa = stages + (size_t)s * kRbStage;
             for (int t = 0; t < nt; t++) {
-                if (ka.a_tiled) tma_load_2d(sa + t * kRbStageW, &mapA, 0, ((t0 + t) * kblocks + kb0 + it) * kTcTileN, &full[s]);
-                else tma_load_2d(sa + t * kRbStageW, &mapA, (kb0 + it) * kTcBlockK, (t0 + t) * kTcTileN, &full[s]);
+                if (ka.a_tiled) tma_load_2d(sa + t * kRbStageW, &mapA, 0, ((w0 + t) * kblocks + kb0 + it) * kTcTileN, &full[s]);
+                else tma_load_2d(sa + t * kRbStageW, &mapA, (kb0 + it) * kTcBlockK, (w0 + t) * kTcTileN, &full[s]);
             }
         };
         auto load_x = [&](int it, int s) {
@@ -739,6 +769,29 @@ vb_tc_rows_kernel(const __grid_constant__ CUtensorMap mapA, const __grid_constan
             } else {
                 for (int t = 0; t < nt; t++) {
                     const int n = (t0 + t) * kTcTileN + lane * 4;
+                    if ((epi == TC_EPI_TERMS || epi == TC_EPI_RELU2_TERMS) && n >= ka.act_n0) {
+                        const int col = ka.out_col0 + n - ka.act_n0;
+                        for (int mb = warp; mb < Mb; mb += 4) {
+                            const float4 v = *(const float4 *)(stg + (t * kRbRows + mb) * kTcTileN + lane * 4);
+                            float e[4] = {v.x, v.y, v.z, v.w};
+                            uint16_t q[3][4];
+#pragma unroll
+                            for (int i = 0; i < 4; i++) {
+                                if (epi == TC_EPI_RELU2_TERMS) { e[i] = fmaxf(e[i], 0.0f); e[i] *= e[i]; }
+                                vb_split3(e[i], q[0][i], q[1][i], q[2][i]);
+                            }
+#pragma unroll
+                            for (int j = 0; j < kRbTerms; j++) {
+                                uint16_t *o = ka.out_terms + ((size_t)j * ka.out_rows_pad + m0 + mb) * ka.out_terms_ld + col;
+                                if (n + 3 < N) {
+                                    *(uint2 *)o = make_uint2(q[j][0] | ((uint32_t)q[j][1] << 16), q[j][2] | ((uint32_t)q[j][3] << 16));
+                                } else {
+                                    for (int i = 0; i < 4 && n + i < N; i++) o[i] = q[j][i];
+                                }
+                            }
+                        }
+                        continue;
+                    }
                     for (int mb = warp; mb < Mb; mb += 4) {
                         float4 v = *(const float4 *)(stg + (t * kRbRows + mb) * kTcTileN + lane * 4);
                         const size_t o = ((size_t)(epi == TC_EPI_STORE ? 0 : sp) * M + m0 + mb) * ld_out + n;
@@ -778,10 +831,12 @@ vb_tc_rows_kernel(const __grid_constant__ CUtensorMap mapA, const __grid_constan
     }
 }
 
-static int launch_rows(const TcWeight &w, const TcActs &a, const TcKernelArgs &ka, cudaStream_t st) {
+template <bool GROUPED>
+static int launch_rows(const TcWeight &w, const TcActs &a, const TcKernelArgs &ka, const typename TcGroupSel<GROUPED>::type &ga,
+                       cudaStream_t st) {
     static bool attr = false;
     if (!attr) {
-        if (cudaFuncSetAttribute(vb_tc_rows_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kRbSmemBytes) !=
+        if (cudaFuncSetAttribute(vb_tc_rows_kernel<GROUPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, kRbSmemBytes) !=
             cudaSuccess) {
             cudaGetLastError();
             return -1;
@@ -790,10 +845,33 @@ static int launch_rows(const TcWeight &w, const TcActs &a, const TcKernelArgs &k
     }
     const int tiles = (ka.N + kTcTileN - 1) / kTcTileN, pairs = (tiles + kRbTiles - 1) / kRbTiles;
     const int row_blocks = (ka.M + kRbRows - 1) / kRbRows;
-    return launch_pdl(vb_tc_rows_kernel, dim3(pairs * row_blocks * ka.splits), dim3(kTcThreads), (size_t)kRbSmemBytes, st,
-                      w.map, a.map_rows, ka) == cudaSuccess
+    return launch_pdl(vb_tc_rows_kernel<GROUPED>, dim3(pairs * row_blocks * ka.splits), dim3(kTcThreads), (size_t)kRbSmemBytes, st,
+                      w.map, a.map_rows, ka, ga) == cudaSuccess
                ? 0
                : -1;
+}
+
+static bool terms_epilogue_ok(const TcGemm &g) {
+    return g.out_terms && g.act_n0 % kTcTileN == 0 && g.out_terms_ld % 4 == 0 && g.out_col0 % 4 == 0;
+}
+
+int tc_gemm_grouped(const TcWeight &w, const TcActs &a, const TcGemm &g, int n, const int4 *table, int n_blocks, cudaStream_t st) {
+    const int tiles = (n + kTcTileN - 1) / kTcTileN;
+    if (!w.ok || !w.tiled || !a.ok || w.K != a.K || n < 1 || n_blocks < 1 || !table || g.splits != 1) return -1;
+    if (w.N % (tiles * kTcTileN) || (size_t)n_blocks * kRbRows > (size_t)a.rows_pad || g.act_n0 != 0) return -1;
+    if (g.epi == TC_EPI_TERMS || g.epi == TC_EPI_RELU2_TERMS) {
+        if (!terms_epilogue_ok(g) || g.out_rows_pad < n_blocks * kRbRows) return -1;
+    } else if (g.epi != TC_EPI_STORE || !g.out || g.ld_out < n) {
+        return -1;
+    }
+    TcKernelArgs ka = {};
+    ka.a_tiled = 1;
+    ka.N = n; ka.K = w.K; ka.M = n_blocks * kRbRows; ka.rows_pad = a.rows_pad; ka.ld_out = g.ld_out; ka.splits = 1;
+    ka.epi = g.epi; ka.out = g.out; ka.out_terms = g.out_terms; ka.out_rows_pad = g.out_rows_pad; ka.status = g.status;
+    ka.out_terms_ld = g.out_terms_ld; ka.out_col0 = g.out_col0;
+    ka.n_tiles_launch = tiles;
+    const TcGroupArgs ga = {table, tiles};
+    return launch_rows<true>(w, a, ka, ga, st);
 }
 
 int tc_gemm(const TcWeight &w, const TcActs &a, const TcGemm &g, cudaStream_t st) {
@@ -802,11 +880,15 @@ int tc_gemm(const TcWeight &w, const TcActs &a, const TcGemm &g, cudaStream_t st
     if (g.epi != TC_EPI_PARTIAL && g.splits != 1) return -1;
     if ((g.epi == TC_EPI_SWIGLU || g.epi == TC_EPI_SWIGLU_TERMS) && (w.N & 1)) return -1;
     if (g.epi == TC_EPI_SWIGLU_TERMS && (!g.out_terms || g.out_rows_pad < g.M)) return -1;
+    if (g.epi == TC_EPI_TERMS || g.epi == TC_EPI_RELU2_TERMS) {
+        if (a.rows_pad < 256 || !terms_epilogue_ok(g) || g.out_rows_pad < g.M || (g.act_n0 > 0 && !g.out)) return -1;
+    }
     TcKernelArgs ka;
     ka.a_tiled = w.tiled ? 1 : 0;
     ka.N = w.N; ka.K = w.K; ka.M = g.M; ka.rows_pad = a.rows_pad; ka.ld_out = g.ld_out; ka.splits = g.splits;
     ka.epi = g.epi; ka.out = g.out; ka.bias = g.bias; ka.ssq = g.ssq; ka.ssq_chunks = g.ssq_chunks; ka.eps = g.eps;
     ka.out_terms = g.out_terms; ka.out_rows_pad = g.out_rows_pad; ka.status = g.status;
+    ka.act_n0 = g.act_n0; ka.out_terms_ld = g.out_terms_ld; ka.out_col0 = g.out_col0;
     {
         const int tiles = (w.N + kTcTileN - 1) / kTcTileN;
         ka.tile0 = g.n_tiles > 0 ? g.tile0 : 0;
@@ -826,11 +908,11 @@ int tc_gemm(const TcWeight &w, const TcActs &a, const TcGemm &g, cudaStream_t st
         /* whole-launch calls on one GPU take the row-block kernel; sliced or exchanged launches
          * (tensor parallelism) do not occur at this size */
         if (g.n_tiles == 0 && tpa.push.n_dst == 0 && tpa.wait.n == 0)
-            return launch_rows(w, a, ka, st);
+            return launch_rows<false>(w, a, ka, TcNoGroupArgs(), st);
         return launch_tc<256, 2>(w, a, ka, tpa, st);
     default:
         if (a.rows_pad > 256 && a.rows_pad % 128 == 0 && g.n_tiles == 0 && tpa.push.n_dst == 0 && tpa.wait.n == 0)
-            return launch_rows(w, a, ka, st);
+            return launch_rows<false>(w, a, ka, TcNoGroupArgs(), st);
         return -1;
     }
 }

@@ -31,7 +31,11 @@ enum TcEpilogue {
     TC_EPI_PARTIAL = 0,       /* out[split][m][n] = partial sum (fp32) */
     TC_EPI_STORE = 1,         /* splits == 1: out[m][n] = sum (+ bias[n]) */
     TC_EPI_SWIGLU = 2,        /* splits == 1, rows interleaved (gate, up): out[m][n/2] = silu(gate) * up */
-    TC_EPI_SWIGLU_TERMS = 3   /* same value, written as three BF16 terms for the next GEMM */
+    TC_EPI_SWIGLU_TERMS = 3,  /* same value, written as three BF16 terms for the next GEMM */
+    /* splits == 1, row-block kernel only: columns from act_n0 on leave as two BF16 terms, the ones before
+     * it as fp32 (out) */
+    TC_EPI_TERMS = 4,         /* the sum itself */
+    TC_EPI_RELU2_TERMS = 5    /* max(sum, 0)^2 */
 };
 
 /* One weight matrix prepared for the tensor-core path. */
@@ -96,6 +100,8 @@ struct TcGemm {
     float eps = 0.0f;
     uint16_t *out_terms = nullptr;    /* TC_EPI_SWIGLU_TERMS destination [3][out_rows_pad][N/2] */
     int out_rows_pad = 0;
+    int act_n0 = 0;                   /* TC_EPI_TERMS, TC_EPI_RELU2_TERMS (a multiple of 128) */
+    int out_terms_ld = 0, out_col0 = 0;   /* the same two: row length of out_terms, column of result act_n0 */
     int *status = nullptr;            /* device int, set non-zero when a bounded wait runs out */
     int tile0 = 0, n_tiles = 0;       /* output tiles [tile0, tile0 + n_tiles) of the weight matrix; 0 = all */
     TcPush push;
@@ -124,6 +130,13 @@ void tc_prepare(const TcActs &acts, const float *x, int ldx, int M, const float 
                 cudaStream_t st, const TcWait &wait = TcWait(), float *tap = nullptr);
 
 int tc_gemm(const TcWeight &w, const TcActs &acts, const TcGemm &g, cudaStream_t st);
+
+/* Grouped GEMM: several weight matrices of equal size stacked in one TcWeight (each padded to whole
+ * 128-row tiles), and rows sorted by matrix in blocks of 128. table[b] = {matrix or -1, first row, rows,
+ * unused} of row block b, in device memory; n_blocks bounds it. acts: tc_acts_blocks. n: rows of one
+ * matrix that are wanted. epi: TC_EPI_STORE or a *_TERMS one. */
+int tc_acts_blocks(TcActs *a, uint16_t *d_buf, int rows, int K);   /* two terms, any multiple of 128 rows */
+int tc_gemm_grouped(const TcWeight &w, const TcActs &acts, const TcGemm &g, int n, const int4 *table, int n_blocks, cudaStream_t st);
 
 void tc_reduce(float *y, const float *partials, int n_part, size_t stride, size_t count, const float *bias, int N,
                cudaStream_t st);

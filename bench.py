@@ -471,9 +471,38 @@ def lm_configs():
         if loop:
             c["loop"] = dict(zip(("start", "stop", "times"), loop))
         return c
+
+    def latent(width, ff, layers, heads, q_rank, vocab, window, experts=None):
+        """Latent attention (heads of 128 + 64, latents of 512) beside a squared-ReLU feed-forward (two matrices: half as wide
+        again as a gated one of equal weight). experts: every second layer has that many of that size, of which a token
+        uses some, and reads the latents of the layer before it."""
+        mixer = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "q_rank": q_rank, "scale": 192 ** -0.5,
+                 "mask": {"size": window}, "rot": {"dims": 64, "base": 100000.0}}
+        stack = []
+        for i in range(layers):
+            if experts and i % 2:
+                n, size, top = experts
+                stack.append({"type": "latent_attention", "mixer": {**mixer, "kv_from": i - 1},
+                              "mlp": {"kind": "moe", "expert": {"ff": size}, "router": {"experts": n, "top": top}}})
+            else:
+                stack.append({"type": "latent_attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": ff}})
+        return {"architecture": "Bupozen", "layers": stack, "norm": {"eps": 1e-5}, "vocab": vocab, "width": width}
     return {"w3072_l26": build(3072, 9216, 26, 24, 8, 32, 8, 128, 128, 8320, 1024),
             "w2048_l16_loop": build(2048, 5632, 16, 16, 8, 16, 4, 128, 128, 32768, 512, (4, 12, 2)),
-            "w4096_l8": build(4096, 14336, 8, 32, 16, 32, 8, 128, 128, 65536, 2048)}
+            "w4096_l8": build(4096, 14336, 8, 32, 16, 32, 8, 128, 128, 65536, 2048),
+            "latent_w3072_l26": latent(3072, 13824, 26, 32, 1536, 8320, 1024),
+            "latent_w2048_l16_experts": latent(2048, 8448, 16, 16, 768, 32768, 512, (64, 1024, 6)),
+            "latent_w4096_l8": latent(4096, 21504, 8, 32, 1536, 65536, 2048)}
+
+
+def lm_unread_bytes(c):
+    """Weight bytes that a token does not read: the experts that were not chosen."""
+    n = 0
+    for l in c["layers"]:
+        if (l.get("mlp") or {}).get("kind") == "moe":
+            r = l["mlp"]["router"]
+            n += (r["experts"] - r["top"]) * l["mlp"]["expert"]["ff"] * c["width"] * 2 * 2
+    return n
 
 
 def lm_bench(args):
@@ -506,7 +535,7 @@ def lm_bench(args):
         with pkg.LanguageModel(config=c, max_tokens=8192) as lm:
             m = {"runs": lm.info.runs, "weight_bytes": lm.info.weight_bytes, "state_bytes": lm.info.state_bytes_per_seq, "prefill": []}
             embed = c["vocab"] * c["width"] * 2
-            layers = lm.info.weight_bytes - 2 * embed
+            layers = lm.info.weight_bytes - 2 * embed - lm_unread_bytes(c)
             loop = c.get("loop")
             passes = lm.info.runs / len(c["layers"])
             m["bytes_per_token"] = layers * passes + embed          # head once, embedding row negligible

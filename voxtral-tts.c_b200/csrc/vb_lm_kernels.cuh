@@ -264,7 +264,7 @@ struct LmLatent {
     LmPart q;                    /* [M][heads * (dim + rot_dim)] */
     LmWeight ukv;                /* rows [heads * dim] key part, [heads * vdim] value part */
     float *ql;                   /* [M][heads][rank + rot_dim] */
-    float *scratch;              /* [key split][(row, head)][rank + 2] */
+    float *scratch;              /* what the key splits leave for the readout */
 };
 constexpr int kLmLatentRows = 16;        /* rows that take the absorbed form where the written-out one is possible */
 constexpr int kLmLatentPairs = 16;       /* (row, head) pairs per CTA */

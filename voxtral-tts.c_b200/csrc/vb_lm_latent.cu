@@ -251,7 +251,15 @@ VB_DEVINL KeyTiles pair_tiles(const LmLatent &a, int M, int p0, int *np) {
     return key_tiles<KT>(pos0 + p0 / a.heads, pos0 + (p0 + *np - 1) / a.heads, a.window, 0);
 }
 
+/* What a key split leaves: [split][pair][rank] sums of weighted rows, then [split][pair] (largest score, sum of weights). */
+VB_DEVINL float2 *attend_stats(const LmLatent &a, int splits, int P) {
+    return reinterpret_cast<float2 *>(a.scratch + (((size_t)splits * P * a.rank + 1) & ~(size_t)1));
+}
+
 constexpr int kLaKeys = 32;
+
+constexpr int kLaThreads = 512, kLaWarps = 16;
+static_assert(kLaWarps == kLaPairs, "a warp owns the softmax of one pair");
 
 struct AttendSmem {
     int row_bytes;               /* of a query or key row in one plane: whole 64-element groups */
@@ -269,18 +277,26 @@ inline AttendSmem attend_smem(int rank, int rot_dim) {
 }
 
 /* A CTA attends with 16 (row, head) pairs over its share of the visible cache rows, 32 at a time. Scores: a warp takes
- * eight keys and half of the columns; values: a warp takes every eighth 16-column step. Products a.b as
+ * eight keys and a quarter of the columns; values: a warp takes every 16th 16-column step. Products a.b as
  * a_hi.b_hi + a_hi.b_lo + a_lo.b_hi, accumulated in fp32. ND: value steps per warp. grid = (pair tiles, splits) */
 template <int ND>
-__global__ void __launch_bounds__(kLtThreads) lm_latent_attend_kernel(const LmLatent a, int M, int row_bytes, int stages) {
+__global__ void __launch_bounds__(kLaThreads) lm_latent_attend_kernel(const LmLatent a, int M, int row_bytes, int stages) {
     extern __shared__ __align__(128) unsigned char at_smem[];
-    __shared__ float S[2][kLaPairs][kLaKeys + 1], mx[kLaPairs], den[kLaPairs], cor[kLaPairs];
+    __shared__ float S[4][kLaPairs][kLaKeys + 1], mx[kLaPairs], den[kLaPairs], cor[kLaPairs];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, tq = lane & 3;
     const int q_plane = kLaPairs * row_bytes, k_plane = kLaKeys * row_bytes;
     unsigned char *Kb = at_smem + 2 * q_plane;
     pdl_launch_dependents();
-    for (int i = tid; i < (2 * q_plane + stages * 2 * k_plane) / 16; i += kLtThreads)
-        reinterpret_cast<uint4 *>(at_smem)[i] = make_uint4(0u, 0u, 0u, 0u);
+    const int row = a.rank + a.rot_dim, per = row / 8, chunks = row_bytes / 16;
+    auto swz = [&](int r, int chunk) { return (uint32_t)(r * row_bytes + (((chunk & ~7) | ((chunk ^ r) & 7)) << 4)); };
+    /* what is never loaded: columns beyond the row, in every plane */
+    for (int r = warp; r < 2 * kLaPairs + stages * 2 * kLaKeys; r += kLaWarps) {
+        const bool isq = r < 2 * kLaPairs;
+        const int k = r - 2 * kLaPairs;
+        unsigned char *plane = isq ? at_smem + (r / kLaPairs) * q_plane : Kb + (k / kLaKeys) * k_plane;
+        const int rr = isq ? r % kLaPairs : k % kLaKeys;
+        for (int c = per + lane; c < chunks; c += 32) *reinterpret_cast<uint4 *>(plane + swz(rr, c)) = make_uint4(0u, 0u, 0u, 0u);
+    }
     pdl_wait();
     int np;
     const int p0 = blockIdx.x * kLaPairs, sp = blockIdx.y;
@@ -288,34 +304,43 @@ __global__ void __launch_bounds__(kLtThreads) lm_latent_attend_kernel(const LmLa
     const int S_eff = (int)gridDim.y < kt.n_tiles ? (int)gridDim.y : kt.n_tiles;
     if (sp >= S_eff) return;
     const int t0 = (int)((long long)kt.n_tiles * sp / S_eff), t1 = (int)((long long)kt.n_tiles * (sp + 1) / S_eff);
-    const int row = a.rank + a.rot_dim, pos0 = a.dyn->pos, P = M * a.heads;
+    const int pos0 = a.dyn->pos, P = M * a.heads;
     const float *cache = lm_state(a.kv, a.dyn);
-    __syncthreads();
-    auto swz = [&](int r, int chunk) { return (uint32_t)(r * row_bytes + (((chunk & ~7) | ((chunk ^ r) & 7)) << 4)); };
     auto request = [&](int t) {
         int j0, n;
         key_tile<kLaKeys>(kt, t, &j0, &n);
         unsigned char *b = Kb + (stages == 2 ? (t & 1) : 0) * 2 * k_plane;
-        const int per = row / 8;
-        for (int i = tid; i < n * 2 * per; i += kLtThreads) {
-            const int key = i / (2 * per), f = i % (2 * per), plane = f >= per ? 1 : 0, chunk = f - plane * per;
-            lm_cp16(b + plane * k_plane + swz(key, chunk),
-                    reinterpret_cast<const uint16_t *>(cache + (size_t)lm_ring_row(a.ring, j0 + key) * row) + f * 8);
+        for (int key = warp; key < n; key += kLaWarps) {
+            const uint16_t *src = reinterpret_cast<const uint16_t *>(cache + (size_t)lm_ring_row(a.ring, j0 + key) * row);
+            for (int f = lane; f < 2 * per; f += 32) {
+                const int plane = f >= per ? 1 : 0;
+                lm_cp16(b + plane * k_plane + swz(key, f - plane * per), src + f * 8);
+            }
         }
+        /* beyond the last key: weights of zero must not meet what an earlier launch left */
+        for (int key = n + warp; key < kLaKeys; key += kLaWarps)
+            for (int f = lane; f < 2 * per; f += 32) {
+                const int plane = f >= per ? 1 : 0;
+                *reinterpret_cast<uint4 *>(b + plane * k_plane + swz(key, f - plane * per)) = make_uint4(0u, 0u, 0u, 0u);
+            }
         lm_cp_commit();
     };
     request(t0);
-    for (int i = tid; i < np * (row / 8); i += kLtThreads) {
-        const int p = i / (row / 8), chunk = i % (row / 8);
-        const float *q = a.ql + (size_t)(p0 + p) * row + chunk * 8;
-        const float4 u = vb_ldcg4(q), v = vb_ldcg4(q + 4);
-        const float e[8] = {u.x, u.y, u.z, u.w, v.x, v.y, v.z, v.w};
-        uint32_t hi[8], lo[8];
+    for (int p = warp; p < kLaPairs; p += kLaWarps) {
+        const float *q = a.ql + (size_t)(p0 + p) * row;
+        for (int chunk = lane; chunk < per; chunk += 32) {
+            uint32_t hi[8] = {}, lo[8] = {};
+            if (p < np) {
+                const float4 u = vb_ldcg4(q + chunk * 8), v = vb_ldcg4(q + chunk * 8 + 4);
+                const float e[8] = {u.x, u.y, u.z, u.w, v.x, v.y, v.z, v.w};
 #pragma unroll
-        for (int j = 0; j < 8; j++) hilo(e[j], hi[j], lo[j]);
-        unsigned char *o = at_smem + swz(p, chunk);
-        *reinterpret_cast<uint4 *>(o) = make_uint4(hi[0] | (hi[1] << 16), hi[2] | (hi[3] << 16), hi[4] | (hi[5] << 16), hi[6] | (hi[7] << 16));
-        *reinterpret_cast<uint4 *>(o + q_plane) = make_uint4(lo[0] | (lo[1] << 16), lo[2] | (lo[3] << 16), lo[4] | (lo[5] << 16), lo[6] | (lo[7] << 16));
+                for (int j = 0; j < 8; j++) hilo(e[j], hi[j], lo[j]);
+            }
+            unsigned char *o = at_smem + swz(p, chunk);
+            *reinterpret_cast<uint4 *>(o) = make_uint4(hi[0] | (hi[1] << 16), hi[2] | (hi[3] << 16), hi[4] | (hi[5] << 16), hi[6] | (hi[7] << 16));
+            *reinterpret_cast<uint4 *>(o + q_plane) =
+                make_uint4(lo[0] | (lo[1] << 16), lo[2] | (lo[3] << 16), lo[4] | (lo[5] << 16), lo[6] | (lo[7] << 16));
+        }
     }
     if (tid < kLaPairs) { mx[tid] = -INFINITY; den[tid] = 0.0f; }
     float o[2 * ND][4];
@@ -338,7 +363,7 @@ __global__ void __launch_bounds__(kLtThreads) lm_latent_attend_kernel(const LmLa
         const uint32_t sK = vb_smem_u32(Kb + (stages == 2 ? (t & 1) : 0) * 2 * k_plane);
         float s0[4] = {}, s1[4] = {}, s2[4] = {};
 #pragma unroll 4
-        for (int ks = kh * steps / 2; ks < (kh + 1) * steps / 2; ks++) {
+        for (int ks = kh * (steps / 4); ks < (kh + 1) * (steps / 4); ks++) {      /* rows are whole 64-element groups */
             uint32_t qh[4], ql[4], b[4];
             const uint32_t qo = swz((lane & 7) + ((lane >> 3) & 1) * 8, ks * 2 + (lane >> 4));
             ldsm(qh, sQ + qo);
@@ -351,11 +376,10 @@ __global__ void __launch_bounds__(kLtThreads) lm_latent_attend_kernel(const LmLa
 #pragma unroll
         for (int c = 0; c < 4; c++) S[kh][gq + (c >> 1) * 8][nt * 8 + 2 * tq + (c & 1)] = s0[c] + (s1[c] + s2[c]);
         __syncthreads();
-#pragma unroll
-        for (int rr = 0; rr < 2; rr++) {
-            const int p = warp * 2 + rr, pc = p0 + p < P ? p0 + p : P - 1;
+        {
+            const int p = warp, pc = p0 + p < P ? p0 + p : P - 1;
             const int i = pos0 + pc / a.heads;
-            float s = (S[0][p][lane] + S[1][p][lane]) * a.scale;
+            float s = ((S[0][p][lane] + S[1][p][lane]) + (S[2][p][lane] + S[3][p][lane])) * a.scale;
             if (lane >= n || !key_seen(i, j0 + lane, a.window, 0)) s = -INFINITY;
             float top = s;
 #pragma unroll
@@ -388,7 +412,7 @@ __global__ void __launch_bounds__(kLtThreads) lm_latent_attend_kernel(const LmLa
         const float cA = cor[gq], cB = cor[gq + 8];
 #pragma unroll
         for (int i = 0; i < ND; i++) {
-            const int dp = warp + i * kLtWarps;
+            const int dp = warp + i * kLaWarps;
             if (dp >= vsteps) break;
 #pragma unroll
             for (int u = 0; u < 2; u++) { o[2 * i + u][0] *= cA; o[2 * i + u][1] *= cA; o[2 * i + u][2] *= cB; o[2 * i + u][3] *= cB; }
@@ -408,22 +432,19 @@ __global__ void __launch_bounds__(kLtThreads) lm_latent_attend_kernel(const LmLa
         }
     }
     /* (the last statistics were written before the barrier ahead of the value products) */
-    float *out = a.scratch + ((size_t)sp * P + p0) * (a.rank + 2);
+    float *out = a.scratch + ((size_t)sp * P + p0) * a.rank;
 #pragma unroll
     for (int i = 0; i < ND; i++) {
-        const int dp = warp + i * kLtWarps;
+        const int dp = warp + i * kLaWarps;
 #pragma unroll
         for (int u = 0; u < 2; u++) {
             const int c = dp * 16 + u * 8 + 2 * tq;
             if (c >= a.rank) continue;
-            if (gq < np) *reinterpret_cast<float2 *>(out + (size_t)gq * (a.rank + 2) + c) = make_float2(o[2 * i + u][0], o[2 * i + u][1]);
-            if (gq + 8 < np) *reinterpret_cast<float2 *>(out + (size_t)(gq + 8) * (a.rank + 2) + c) = make_float2(o[2 * i + u][2], o[2 * i + u][3]);
+            if (gq < np) *reinterpret_cast<float2 *>(out + (size_t)gq * a.rank + c) = make_float2(o[2 * i + u][0], o[2 * i + u][1]);
+            if (gq + 8 < np) *reinterpret_cast<float2 *>(out + (size_t)(gq + 8) * a.rank + c) = make_float2(o[2 * i + u][2], o[2 * i + u][3]);
         }
     }
-    if (tid < np) {
-        out[(size_t)tid * (a.rank + 2) + a.rank] = mx[tid];
-        out[(size_t)tid * (a.rank + 2) + a.rank + 1] = den[tid];
-    }
+    if (tid < np) attend_stats(a, (int)gridDim.y, P)[(size_t)sp * P + p0 + tid] = make_float2(mx[tid], den[tid]);
 }
 
 /* The same on the fp32 pipes, any sizes; cache rows in either form. */
@@ -500,12 +521,9 @@ __global__ void __launch_bounds__(kLtThreads) lm_latent_attend_f32_kernel(const 
         }
     }
     __syncthreads();
-    float *out = a.scratch + ((size_t)sp * P + p0) * (a.rank + 2);
-    for (int i = tid; i < np * a.rank; i += kLtThreads) out[(size_t)(i / a.rank) * (a.rank + 2) + i % a.rank] = O[i];
-    if (tid < np) {
-        out[(size_t)tid * (a.rank + 2) + a.rank] = mx[tid];
-        out[(size_t)tid * (a.rank + 2) + a.rank + 1] = den[tid];
-    }
+    float *out = a.scratch + ((size_t)sp * P + p0) * a.rank;
+    for (int i = tid; i < np * a.rank; i += kLtThreads) out[i] = O[i];
+    if (tid < np) attend_stats(a, (int)gridDim.y, P)[(size_t)sp * P + p0 + tid] = make_float2(mx[tid], den[tid]);
 }
 
 /* ------------------------------------------------------------------ values */
@@ -528,27 +546,27 @@ __global__ void __launch_bounds__(kLtThreads) lm_latent_readout_kernel(const LmL
     for (int i = 0; i < kPre; i++)
         pre[i] = i < kblocks ? __ldg(reinterpret_cast<const uint4 *>(lm_weight_row(a.ukv, wrow, i) + c0)) : make_uint4(0u, 0u, 0u, 0u);
     pdl_wait();
-    const int stride = a.rank + 2;
     const size_t P = (size_t)M * a.heads;
+    const float2 *stats = attend_stats(a, splits, (int)P);
     if (warp < nr) {
         const int p = (m0 + warp) * a.heads + h;
         int np;
         const KeyTiles kt = pair_tiles<KT>(a, M, p / kLaPairs * kLaPairs, &np);
         const int S = splits < kt.n_tiles ? splits : kt.n_tiles;
+        float2 st[2];
         float mu[2], top = -INFINITY, L = 0.0f;
 #pragma unroll
         for (int x = 0; x < 2; x++) {
             const int u = lane + 32 * x;
-            mu[x] = u < S ? __ldcg(a.scratch + (u * P + p) * stride + a.rank) : -INFINITY;
-            top = fmaxf(top, mu[x]);
+            st[x] = u < S ? __ldcg(stats + u * P + p) : make_float2(-INFINITY, 0.0f);
+            top = fmaxf(top, st[x].x);
         }
 #pragma unroll
         for (int off = 16; off > 0; off >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, off));
 #pragma unroll
         for (int x = 0; x < 2; x++) {
-            const int u = lane + 32 * x;
-            mu[x] = u < S ? expf(mu[x] - top) : 0.0f;          /* a row always sees itself: top is finite */
-            if (u < S) L = fmaf(mu[x], __ldcg(a.scratch + (u * P + p) * stride + a.rank + 1), L);
+            mu[x] = expf(st[x].x - top);                       /* a row always sees itself: top is finite */
+            L = fmaf(mu[x], st[x].y, L);
         }
         L = vb_warp_sum(L);
         wgt[warp][lane] = mu[0] / L;
@@ -556,17 +574,41 @@ __global__ void __launch_bounds__(kLtThreads) lm_latent_readout_kernel(const LmL
         if (lane == 0) count[warp] = S;
     }
     __syncthreads();
-    for (int i = tid; i < nr * rp; i += kLtThreads) {
-        const int r = i / rp, c = i % rp;
-        float o = 0.0f;
-        if (c < a.rank) {
-            const float *s = a.scratch + ((size_t)(m0 + r) * a.heads + h) * stride + c;
-            const int S = count[r];
+    if ((a.rank & 3) == 0) {
+        /* four columns per item; where there are few items, neighbouring lanes share one and take every second,
+         * fourth, ... split */
+        const int nv = a.rank / 4, items = nr * nv;
+        int parts = 1;
+        while (parts < 8 && items * parts * 2 <= kLtThreads) parts *= 2;
+        for (int i0 = 0; i0 < items; i0 += kLtThreads / parts) {
+            const int i = i0 + tid / parts, part = tid % parts;
+            const bool in = i < items;
+            const int r = in ? i / nv : 0, c = in ? i % nv * 4 : 0;
+            const float *s = a.scratch + ((size_t)(m0 + r) * a.heads + h) * a.rank + c;
+            const int S = in ? count[r] : 0;
+            float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 8
-            for (int u = 0; u < S; u++) o = fmaf(wgt[r][u], __ldcg(s + u * P * stride), o);
+            for (int u = part; u < S; u += parts) {
+                const float4 t = vb_ldcg4(s + u * P * a.rank);
+                const float w = wgt[r][u];
+                o.x = fmaf(w, t.x, o.x); o.y = fmaf(w, t.y, o.y); o.z = fmaf(w, t.z, o.z); o.w = fmaf(w, t.w, o.w);
+            }
+            for (int off = 1; off < parts; off <<= 1) {
+                o.x += __shfl_xor_sync(0xffffffffu, o.x, off); o.y += __shfl_xor_sync(0xffffffffu, o.y, off);
+                o.z += __shfl_xor_sync(0xffffffffu, o.z, off); o.w += __shfl_xor_sync(0xffffffffu, o.w, off);
+            }
+            if (in && part == 0) *reinterpret_cast<float4 *>(ro + r * rp + c) = o;
         }
-        ro[i] = o;
+    } else {
+        for (int i = tid; i < nr * a.rank; i += kLtThreads) {
+            const int r = i / a.rank, c = i % a.rank, S = count[r];
+            const float *s = a.scratch + ((size_t)(m0 + r) * a.heads + h) * a.rank + c;
+            float o = 0.0f;
+            for (int u = 0; u < S; u++) o = fmaf(wgt[r][u], __ldcg(s + u * P * a.rank), o);
+            ro[r * rp + c] = o;
+        }
     }
+    for (int i = tid; i < nr * (rp - a.rank); i += kLtThreads) ro[i / (rp - a.rank) * rp + a.rank + i % (rp - a.rank)] = 0.0f;
     __syncthreads();
     float acc[MR];
 #pragma unroll
@@ -612,7 +654,7 @@ template <int ND>
 int launch_attend(const LmLatent &a, int M, const AttendSmem &s, cudaStream_t st) {
     static size_t set = 32 * 1024;
     if (allow_smem(lm_latent_attend_kernel<ND>, s.total, &set)) return -1;
-    return ok(launch_pdl(lm_latent_attend_kernel<ND>, dim3(attend_tiles(M, a.heads), attend_splits(M, a.heads)), dim3(kLtThreads), s.total, st, a, M,
+    return ok(launch_pdl(lm_latent_attend_kernel<ND>, dim3(attend_tiles(M, a.heads), attend_splits(M, a.heads)), dim3(kLaThreads), s.total, st, a, M,
                          s.row_bytes, s.stages));
 }
 template <int KT>
@@ -650,7 +692,7 @@ bool lm_latent_supported(int q_rank, int rank, int rot_dim) {
 size_t lm_latent_scratch_floats(int rows, int heads, int rank) {
     size_t n = 0;
     for (int M = 1; M <= rows; M++) n = n > (size_t)attend_splits(M, heads) * M ? n : (size_t)attend_splits(M, heads) * M;
-    return n * heads * (rank + 2);
+    return n * heads * (rank + 2) + 2;
 }
 
 int lm_latent_prepare(const LmLatent &a, int M, cudaStream_t st) {
@@ -666,10 +708,8 @@ int lm_latent_absorb(const LmLatent &a, int M, cudaStream_t st) { return M == 1 
 int lm_latent_attend(const LmLatent &a, int M, cudaStream_t st) {
     if (a.split) {
         const AttendSmem s = attend_smem(a.rank, a.rot_dim);
-        if (a.rank <= 128) return launch_attend<1>(a, M, s, st);
-        if (a.rank <= 256) return launch_attend<2>(a, M, s, st);
-        if (a.rank <= 512) return launch_attend<4>(a, M, s, st);
-        return launch_attend<8>(a, M, s, st);
+        if (a.rank <= 256) return launch_attend<1>(a, M, s, st);
+        return a.rank <= 512 ? launch_attend<2>(a, M, s, st) : launch_attend<4>(a, M, s, st);
     }
     return attend_f32_keys(a.rank, a.rot_dim) == 32 ? launch_attend_f32<32>(a, M, st) : launch_attend_f32<8>(a, M, st);
 }

@@ -290,7 +290,7 @@ __global__ void __launch_bounds__(kLaThreads) lm_latent_attend_kernel(const LmLa
     const int row = a.rank + a.rot_dim, per = row / 8, chunks = row_bytes / 16;
     auto swz = [&](int r, int chunk) { return (uint32_t)(r * row_bytes + (((chunk & ~7) | ((chunk ^ r) & 7)) << 4)); };
     /* what is never loaded: columns beyond the row, in every plane */
-    for (int r = warp; r < 2 * kLaPairs + stages * 2 * kLaKeys; r += kLaWarps) {
+    for (int r = warp; per < chunks && r < 2 * kLaPairs + stages * 2 * kLaKeys; r += kLaWarps) {
         const bool isq = r < 2 * kLaPairs;
         const int k = r - 2 * kLaPairs;
         unsigned char *plane = isq ? at_smem + (r / kLaPairs) * q_plane : Kb + (k / kLaKeys) * k_plane;

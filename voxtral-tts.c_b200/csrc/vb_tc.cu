@@ -545,6 +545,9 @@ constexpr int kRbStage = kRbTiles * kRbStageW + kRbTerms * kRbStageX;
 constexpr int kRbTmemCols = kRbTiles * kRbRows;
 constexpr int kRbSmemBytes = kRbStages * kRbStage + 1024 + 256 + 4 * kRbRows;
 static_assert(kRbSmemBytes <= 232448, "over the 227 KB a CTA may use");
+/* The epilogue of a CTA (128 rows x 256 results) is bound by instruction latency: with four warps it took as
+ * long as 16 k-blocks. Sixteen share it: two per 32 TMEM lanes and tile, each half of the rows. */
+constexpr int kRbEpiWarps = 16, kRbEpi = 32 * kRbEpiWarps, kRbThreads = kRbEpi + 64;
 
 /* GROUPED: a row block belongs to one of several stacked weight matrices, looked up in device memory;
  * N is the size of one of them. */
@@ -557,7 +560,7 @@ template <bool GROUPED> struct TcGroupSel { using type = TcNoGroupArgs; };
 template <> struct TcGroupSel<true> { using type = TcGroupArgs; };
 
 template <bool GROUPED>
-__global__ void __launch_bounds__(kTcThreads, 1)
+__global__ void __launch_bounds__(kRbThreads, 1)
 vb_tc_rows_kernel(const __grid_constant__ CUtensorMap mapA, const __grid_constant__ CUtensorMap mapB,
                   const TcKernelArgs ka, const typename TcGroupSel<GROUPED>::type ga) {
     const int N = ka.N, K = ka.K, M = ka.M, rows_pad = ka.rows_pad, ld_out = ka.ld_out, splits = ka.splits,
@@ -616,7 +619,7 @@ vb_tc_rows_kernel(const __grid_constant__ CUtensorMap mapA, const __grid_constan
     tc_fence_after();
     const uint32_t tmem = *(volatile uint32_t *)tmem_slot;
 
-    if (warp == 4 && lane == 0) {
+    if (warp == kRbEpiWarps && lane == 0) {
         /* ---- TMA producer: weights first (they depend on nothing), activation terms after the
          * predecessor kernel has finished ---- */
         auto load_w = [&](int it, int s) {
@@ -652,7 +655,7 @@ vb_tc_rows_kernel(const __grid_constant__ CUtensorMap mapA, const __grid_constan
             load_x(it, s);
             issued = it + 1;
         }
-    } else if (warp == 5 && lane == 0) {
+    } else if (warp == kRbEpiWarps + 1 && lane == 0) {
         /* ---- MMA issuer ---- */
         const uint32_t idesc = umma_idesc_bf16(kRbRows);
         for (int it = 0; it < n_it; it++) {
@@ -678,16 +681,16 @@ vb_tc_rows_kernel(const __grid_constant__ CUtensorMap mapA, const __grid_constan
             umma_commit(&empty[s]);
         }
         umma_commit(accum);
-    } else if (warp < 4) {
+    } else if (warp < kRbEpiWarps) {
         /* ---- epilogue: TMEM -> registers -> global ---- */
         pdl_wait();
         if (ka.ssq) {
-            for (int m = threadIdx.x; m < Mb; m += 128) {
+            for (int m = threadIdx.x; m < Mb; m += kRbEpi) {
                 float t = 0.0f;
                 for (int c = 0; c < ka.ssq_chunks; c++) t += __ldcg(ka.ssq + (m0 + m) * ka.ssq_chunks + c);
                 rscale[m] = 1.0f / sqrtf(t / (float)K + ka.eps);
             }
-            vb_named_bar(1, 128);
+            vb_named_bar(1, kRbEpi);
         }
         bool ok = vb_mbar_wait(accum, 0u, abort_flag);
         if (!ok) {
@@ -702,20 +705,22 @@ vb_tc_rows_kernel(const __grid_constant__ CUtensorMap mapA, const __grid_constan
              * lane = output column, one 4-byte store per activation row - took 23 us per CTA
              * for 128 KB of results: five times the main loop's share. */
             float *stg = (float *)stages;                       /* [tile][128 rows m][128 columns n] */
-            for (int t = 0; t < nt; t++) {
+            constexpr int kParts = kRbEpiWarps / (4 * kRbTiles);    /* warps per 32 lanes and tile */
+            const int lq = warp & 3, t = (warp >> 2) % kRbTiles, part = (warp >> 2) / kRbTiles;
+            if (t < nt) {
 #pragma unroll 1
-                for (int c0 = 0; c0 < Mb; c0 += 16) {
+                for (int c0 = part * 16; c0 < Mb; c0 += 16 * kParts) {
                     uint32_t r[16];
-                    tmem_ld16(tmem + ((uint32_t)(warp * 32) << 16) + (uint32_t)(t * kRbRows + c0), r);
+                    tmem_ld16(tmem + ((uint32_t)(lq * 32) << 16) + (uint32_t)(t * kRbRows + c0), r);
 #pragma unroll
                     for (int i = 0; i < 16; i++) {
                         float v = __uint_as_float(r[i]);
                         if (ka.ssq && c0 + i < Mb) v *= rscale[c0 + i];
-                        stg[(t * kRbRows + c0 + i) * kTcTileN + warp * 32 + lane] = v;
+                        stg[(t * kRbRows + c0 + i) * kTcTileN + lq * 32 + lane] = v;
                     }
                 }
             }
-            vb_named_bar(1, 128);
+            vb_named_bar(1, kRbEpi);
             if (epi == TC_EPI_SWIGLU || epi == TC_EPI_SWIGLU_TERMS) {
                 /* a lane turns 8 staged values (4 (gate, up) pairs) into 4 results; the 32 lanes
                  * cover the 128 results of the CTA's two tiles for one activation row */
@@ -723,7 +728,7 @@ vb_tc_rows_kernel(const __grid_constant__ CUtensorMap mapA, const __grid_constan
                 const int col = (t0 + tt) * (kTcTileN / 2) + (lane & 15) * 4;       /* first result column */
                 const size_t ko = (size_t)(N >> 1);
                 if (tt < nt && 2 * col + 7 < N) {
-                    for (int mb = warp; mb < Mb; mb += 4) {
+                    for (int mb = warp; mb < Mb; mb += kRbEpiWarps) {
                         const float4 a = *(const float4 *)(stg + (tt * kRbRows + mb) * kTcTileN + n8);
                         const float4 b = *(const float4 *)(stg + (tt * kRbRows + mb) * kTcTileN + n8 + 4);
                         float res[4];
@@ -747,7 +752,7 @@ vb_tc_rows_kernel(const __grid_constant__ CUtensorMap mapA, const __grid_constan
                     }
                 } else if (tt < nt) {
                     /* ragged edge of the matrix: element by element */
-                    for (int mb = warp; mb < Mb; mb += 4) {
+                    for (int mb = warp; mb < Mb; mb += kRbEpiWarps) {
                         for (int i = 0; i < 4; i++) {
                             if (2 * (col + i) + 1 >= N) break;
                             const float g = stg[(tt * kRbRows + mb) * kTcTileN + n8 + 2 * i];
@@ -771,7 +776,7 @@ vb_tc_rows_kernel(const __grid_constant__ CUtensorMap mapA, const __grid_constan
                     const int n = (t0 + t) * kTcTileN + lane * 4;
                     if ((epi == TC_EPI_TERMS || epi == TC_EPI_RELU2_TERMS) && n >= ka.act_n0) {
                         const int col = ka.out_col0 + n - ka.act_n0;
-                        for (int mb = warp; mb < Mb; mb += 4) {
+                        for (int mb = warp; mb < Mb; mb += kRbEpiWarps) {
                             const float4 v = *(const float4 *)(stg + (t * kRbRows + mb) * kTcTileN + lane * 4);
                             float e[4] = {v.x, v.y, v.z, v.w};
                             uint16_t q[3][4];
@@ -792,7 +797,7 @@ vb_tc_rows_kernel(const __grid_constant__ CUtensorMap mapA, const __grid_constan
                         }
                         continue;
                     }
-                    for (int mb = warp; mb < Mb; mb += 4) {
+                    for (int mb = warp; mb < Mb; mb += kRbEpiWarps) {
                         float4 v = *(const float4 *)(stg + (t * kRbRows + mb) * kTcTileN + lane * 4);
                         const size_t o = ((size_t)(epi == TC_EPI_STORE ? 0 : sp) * M + m0 + mb) * ld_out + n;
                         if (n + 3 < N && (ld_out & 3) == 0) {
@@ -814,7 +819,7 @@ vb_tc_rows_kernel(const __grid_constant__ CUtensorMap mapA, const __grid_constan
 
     tc_fence_before();
     __syncthreads();
-    if (warp == 4 && lane == 0 && *(volatile int *)abort_flag) {
+    if (warp == kRbEpiWarps && lane == 0 && *(volatile int *)abort_flag) {
         /* abort path: let copies already in flight land before the shared memory goes away */
         const int first_it = issued > kRbStages ? issued - kRbStages : 0;
         for (int it = first_it; it < issued; it++) {
@@ -845,7 +850,7 @@ static int launch_rows(const TcWeight &w, const TcActs &a, const TcKernelArgs &k
     }
     const int tiles = (ka.N + kTcTileN - 1) / kTcTileN, pairs = (tiles + kRbTiles - 1) / kRbTiles;
     const int row_blocks = (ka.M + kRbRows - 1) / kRbRows;
-    return launch_pdl(vb_tc_rows_kernel<GROUPED>, dim3(pairs * row_blocks * ka.splits), dim3(kTcThreads), (size_t)kRbSmemBytes, st,
+    return launch_pdl(vb_tc_rows_kernel<GROUPED>, dim3(pairs * row_blocks * ka.splits), dim3(kRbThreads), (size_t)kRbSmemBytes, st,
                       w.map, a.map_rows, ka, ga) == cudaSuccess
                ? 0
                : -1;

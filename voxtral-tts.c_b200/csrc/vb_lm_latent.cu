@@ -34,46 +34,53 @@ __host__ __device__ constexpr int up4(int v) { return (v + 3) & ~3; }
 constexpr size_t kSmemLimit = 216 * 1024;      /* dynamic part; a few KB are static */
 
 /* ------------------------------------------------------------------ a row's latents */
-constexpr int kLpThreads = 512, kLpWarps = kLpThreads / 32;
+constexpr int kLpThreads = 512, kLpWarps = kLpThreads / 32;      /* at most: as many as a row has float4 columns */
 
-/* The `top` largest of z[0, n), the first one on a tie, and the softmax over them: one warp. */
-VB_DEVINL void route_row(const float *z, int n, int top, int *chosen, float *weight, int lane) {
+/* The `top` largest of z[0, n), the first one on a tie, and the softmax over them: one warp. `pick` holds `top` indexes. */
+VB_DEVINL void route_row(float *z, int n, int top, int *pick, int *chosen, float *weight, int lane) {
     unsigned taken = 0;                      /* bit i: z[lane + 32 * i] */
     float first = 0.0f, sum = 0.0f;
     for (int k = 0; k < top; k++) {
-        float best = -INFINITY;
+        /* floats as unsigned integers of the same order, so that a warp reduces them in one instruction */
+        unsigned best = 0u;
         int bi = 0x7fffffff;
-        for (int i = 0, e = lane; e < n; i++, e += 32)
-            if (!((taken >> i) & 1u) && (bi == 0x7fffffff || z[e] > best)) { best = z[e]; bi = e; }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-            const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-            if (bi == 0x7fffffff || (oi != 0x7fffffff && (ov > best || (!(ov < best) && oi < bi)))) { best = ov; bi = oi; }
+        for (int i = 0, e = lane; e < n; i++, e += 32) {
+            const unsigned u = __float_as_uint(z[e]), key = u & 0x80000000u ? ~u : u | 0x80000000u;
+            if (!((taken >> i) & 1u) && (bi == 0x7fffffff || key > best)) { best = key; bi = e; }
         }
-        bi = __shfl_sync(0xffffffffu, bi, 0);
-        best = __shfl_sync(0xffffffffu, best, 0);
+        const unsigned all = __reduce_max_sync(0xffffffffu, best);
+        bi = __reduce_min_sync(0xffffffffu, best == all ? bi : 0x7fffffff);
         if ((bi & 31) == lane) taken |= 1u << (bi >> 5);
-        if (k == 0) first = best;
-        const float p = expf(best - first);
+        const float v = z[bi];
+        if (k == 0) first = v;
+        const float p = expf(v - first);
         sum += p;
-        if (lane == 0) { chosen[k] = bi; weight[k] = p; }
+        __syncwarp();
+        if (lane == 0) { pick[k] = bi; z[bi] = p; }      /* this place is not looked at again */
     }
-    if (lane == 0)
-        for (int k = 0; k < top; k++) weight[k] /= sum;
+    __syncwarp();
+    for (int k = lane; k < top; k += 32) {
+        chosen[k] = pick[k];
+        weight[k] = z[pick[k]] / sum;
+    }
 }
 
-/* grid = (rows, 1 + pieces of the feed-forward columns) */
-__global__ void __launch_bounds__(kLpThreads) lm_latent_prepare_kernel(const LmLatent a) {
+/* grid = (rows, 1 + pieces of the feed-forward columns). ONE: the in-projection is not split (many rows), which leaves
+ * registers for more CTAs per SM. */
+template <bool ONE>
+__global__ void __launch_bounds__(kLpThreads, ONE ? 3 : 1) lm_latent_prepare_kernel(const LmLatent a) {
     extern __shared__ __align__(16) float lp[];
     __shared__ float red[2][kLpWarps];
     pdl_launch_dependents();
     pdl_wait();
+    const int threads = blockDim.x, warps = threads >> 5;
     const int m = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    auto sum4 = [&](int c) { return ONE ? vb_ldcg4(a.in.p + (size_t)m * a.in.ld + c) : lm_sum4(a.in, m, c); };
+    auto sum1 = [&](int c) { return ONE ? vb_ldcg(a.in.p + (size_t)m * a.in.ld + c) : lm_sum_batch(a.in, m, c); };
     if (blockIdx.y > 0) {
-        const int c = (((int)blockIdx.y - 1) * kLpThreads + tid) * 4;
+        const int c = (((int)blockIdx.y - 1) * threads + tid) * 4;
         if (c >= a.ff) return;
-        const float4 v = lm_sum4(a.in, m, a.col_ff + c);
+        const float4 v = sum4(a.col_ff + c);
         float e[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
         for (int i = 0; i < 4; i++) { e[i] = fmaxf(e[i], 0.0f); e[i] *= e[i]; }
@@ -87,19 +94,11 @@ __global__ void __launch_bounds__(kLpThreads) lm_latent_prepare_kernel(const LmL
     const int half = a.rot / 2, row = a.rank + a.rot_dim, nq = up4(a.q_rank), nc = a.c_gain ? up4(row) : 0;
     float *ql = lp, *cl = ql + nq, *z = cl + nc, *cs = z + a.experts;
     const int pos = a.dyn->pos + m;
-    for (int i = tid; i < half; i += kLpThreads) {
-        float c, s;
-        lm_angle(pos, a.freq[i], a.freq[half + i], a.mag, &c, &s);
-        cs[i] = c;
-        cs[half + i] = s;
-        a.cs[(size_t)m * a.rot + i] = c;
-        a.cs[(size_t)m * a.rot + half + i] = s;
-    }
     /* a part that does not fill its last four columns is followed by zero ones */
     float sq = 0.0f, sc = 0.0f;
-    for (int c = tid * 4; c < nq + nc; c += kLpThreads * 4) {
+    for (int c = tid * 4; c < nq + nc; c += threads * 4) {
         const bool isq = c < nq;
-        const float4 v = lm_sum4(a.in, m, isq ? c : a.col_c + c - nq);
+        const float4 v = sum4(isq ? c : a.col_c + c - nq);
         *reinterpret_cast<float4 *>(lp + c) = v;
         if (isq) {
             sq += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
@@ -109,25 +108,32 @@ __global__ void __launch_bounds__(kLpThreads) lm_latent_prepare_kernel(const LmL
                   (d + 3 < a.rank ? v.w * v.w : 0.0f);
         }
     }
-    for (int e = tid; e < a.experts; e += kLpThreads) z[e] = lm_sum_batch(a.in, m, a.col_router + e);
-    for (int h = tid; h < a.heads; h += kLpThreads)
-        a.gate[(size_t)m * a.heads + h] = 1.0f / (1.0f + expf(-lm_sum_batch(a.in, m, a.col_g + h)));
+    for (int e = tid; e < a.experts; e += threads) z[e] = sum1(a.col_router + e);
+    for (int h = tid; h < a.heads; h += threads)
+        a.gate[(size_t)m * a.heads + h] = 1.0f / (1.0f + expf(-sum1(a.col_g + h)));
+    for (int i = tid; i < half; i += threads) {
+        float c, s;
+        lm_angle(pos, a.freq[i], a.freq[half + i], a.mag, &c, &s);
+        cs[i] = c;
+        cs[half + i] = s;
+        a.cs[(size_t)m * a.rot + i] = c;
+        a.cs[(size_t)m * a.rot + half + i] = s;
+    }
     sq = vb_warp_sum(sq);
     sc = vb_warp_sum(sc);
     if (lane == 0) { red[0][warp] = sq; red[1][warp] = sc; }
     __syncthreads();
     sq = sc = 0.0f;
-#pragma unroll
-    for (int w = 0; w < kLpWarps; w++) { sq += red[0][w]; sc += red[1][w]; }
+    for (int w = 0; w < warps; w++) { sq += red[0][w]; sc += red[1][w]; }
     const float rq = 1.0f / sqrtf(sq / (float)a.q_rank + a.eps), rc = 1.0f / sqrtf(sc / (float)a.rank + a.eps);
     if ((a.q_rank & 3) == 0) {
-        for (int c = tid * 4; c < a.q_rank; c += kLpThreads * 4) {
+        for (int c = tid * 4; c < a.q_rank; c += threads * 4) {
             const float4 g = __ldg(reinterpret_cast<const float4 *>(a.q_gain + c));
             const float e[4] = {ql[c] * rq * g.x, ql[c + 1] * rq * g.y, ql[c + 2] * rq * g.z, ql[c + 3] * rq * g.w};
             lm_put4(a.q_latent, m, c, e);
         }
     } else {
-        for (int c = tid; c < a.q_rank; c += kLpThreads) lm_put(a.q_latent, m, c, ql[c] * rq * __ldg(a.q_gain + c));
+        for (int c = tid; c < a.q_rank; c += threads) lm_put(a.q_latent, m, c, ql[c] * rq * __ldg(a.q_gain + c));
     }
     if (a.c_gain) {
         float *dst = lm_state(a.kv, a.dyn) + (size_t)lm_ring_row(a.ring, pos) * row;
@@ -138,14 +144,14 @@ __global__ void __launch_bounds__(kLpThreads) lm_latent_prepare_kernel(const LmL
             return (j & 1) ? cl[d] * cs[i] + cl[d - 1] * cs[half + i] : cl[d] * cs[i] - cl[d + 1] * cs[half + i];
         };
         if ((row & 3) == 0) {
-            for (int d = tid * 4; d < row; d += kLpThreads * 4)
+            for (int d = tid * 4; d < row; d += threads * 4)
                 kv_put4(dst, row, d, make_float4(value(d), value(d + 1), value(d + 2), value(d + 3)), a.split);
         } else {
-            for (int d = tid; d < row; d += kLpThreads) kv_put(dst, row, d, value(d), a.split);
+            for (int d = tid; d < row; d += threads) kv_put(dst, row, d, value(d), a.split);
         }
     }
-    if (a.experts > 0 && warp == kLpWarps - 1)
-        route_row(z, a.experts, a.top, a.chosen + (size_t)m * a.top, a.weight + (size_t)m * a.top, lane);
+    if (a.experts > 0 && warp == warps - 1)
+        route_row(z, a.experts, a.top, reinterpret_cast<int *>(cs + a.rot), a.chosen + (size_t)m * a.top, a.weight + (size_t)m * a.top, lane);
 }
 
 /* ------------------------------------------------------------------ queries into the latent's space */
@@ -650,6 +656,17 @@ __global__ void lm_latent_gather_kernel(const LmLatent a, uint16_t *terms, int r
     *reinterpret_cast<uint4 *>(terms + ((size_t)plane * rows_pad + j) * ld + chunk * 8) = __ldcg(reinterpret_cast<const uint4 *>(src));
 }
 
+template <bool ONE>
+int launch_prepare(const LmLatent &a, int M, cudaStream_t st) {
+    static size_t set = 40 * 1024;
+    const int columns = up4(a.q_rank) + (a.c_gain ? up4(a.rank + a.rot_dim) : 0);
+    const size_t smem = sizeof(float) * ((size_t)columns + a.experts + a.rot + a.top);
+    if (allow_smem(lm_latent_prepare_kernel<ONE>, smem, &set)) return -1;
+    const int threads = columns >= kLpThreads * 4 ? kLpThreads : columns <= 512 ? 128 : (columns / 4 + 31) / 32 * 32;
+    const int pieces = (a.ff + threads * 4 - 1) / (threads * 4);
+    return ok(launch_pdl(lm_latent_prepare_kernel<ONE>, dim3(M, 1 + pieces), dim3(threads), smem, st, a));
+}
+
 template <int ND>
 int launch_attend(const LmLatent &a, int M, const AttendSmem &s, cudaStream_t st) {
     static size_t set = 32 * 1024;
@@ -687,7 +704,7 @@ bool lm_latent_split_ok(int rank, int rot_dim) {
 }
 bool lm_latent_supported(int q_rank, int rank, int rot_dim) {
     return attend_f32_smem(rank, rot_dim, attend_f32_keys(rank, rot_dim)) <= kSmemLimit &&
-           sizeof(float) * ((size_t)q_rank + rank + 2 * rot_dim + kLmMoeExperts + 16) <= kSmemLimit;
+           sizeof(float) * ((size_t)q_rank + rank + 2 * rot_dim + 2 * kLmMoeExperts + 16) <= kSmemLimit;
 }
 size_t lm_latent_scratch_floats(int rows, int heads, int rank) {
     size_t n = 0;
@@ -695,13 +712,7 @@ size_t lm_latent_scratch_floats(int rows, int heads, int rank) {
     return n * heads * (rank + 2) + 2;
 }
 
-int lm_latent_prepare(const LmLatent &a, int M, cudaStream_t st) {
-    static size_t set = 40 * 1024;
-    const size_t smem = sizeof(float) * ((size_t)up4(a.q_rank) + (a.c_gain ? up4(a.rank + a.rot_dim) : 0) + a.experts + a.rot);
-    if (allow_smem(lm_latent_prepare_kernel, smem, &set)) return -1;
-    const int pieces = (a.ff + kLpThreads * 4 - 1) / (kLpThreads * 4);
-    return ok(launch_pdl(lm_latent_prepare_kernel, dim3(M, 1 + pieces), dim3(kLpThreads), smem, st, a));
-}
+int lm_latent_prepare(const LmLatent &a, int M, cudaStream_t st) { return a.in.n == 1 ? launch_prepare<true>(a, M, st) : launch_prepare<false>(a, M, st); }
 
 int lm_latent_absorb(const LmLatent &a, int M, cudaStream_t st) { return M == 1 ? launch_absorb<1>(a, M, st) : launch_absorb<8>(a, M, st); }
 

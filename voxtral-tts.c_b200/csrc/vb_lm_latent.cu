@@ -712,7 +712,9 @@ size_t lm_latent_scratch_floats(int rows, int heads, int rank) {
     return n * heads * (rank + 2) + 2;
 }
 
-int lm_latent_prepare(const LmLatent &a, int M, cudaStream_t st) { return a.in.n == 1 ? launch_prepare<true>(a, M, st) : launch_prepare<false>(a, M, st); }
+int lm_latent_prepare(const LmLatent &a, int M, cudaStream_t st) {
+    return a.in.n == 1 && M > 64 ? launch_prepare<true>(a, M, st) : launch_prepare<false>(a, M, st);
+}
 
 int lm_latent_absorb(const LmLatent &a, int M, cudaStream_t st) { return M == 1 ? launch_absorb<1>(a, M, st) : launch_absorb<8>(a, M, st); }
 

@@ -94,6 +94,17 @@ __global__ void __launch_bounds__(kLpThreads, ONE ? 3 : 1) lm_latent_prepare_ker
     const int half = a.rot / 2, row = a.rank + a.rot_dim, nq = up4(a.q_rank), nc = a.c_gain ? up4(row) : 0;
     float *ql = lp, *cl = ql + nq, *z = cl + nc, *cs = z + a.experts;
     const int pos = a.dyn->pos + m;
+    auto angles = [&]() {
+        for (int i = tid; i < half; i += threads) {
+            float c, s;
+            lm_angle(pos, a.freq[i], a.freq[half + i], a.mag, &c, &s);
+            cs[i] = c;
+            cs[half + i] = s;
+            a.cs[(size_t)m * a.rot + i] = c;
+            a.cs[(size_t)m * a.rot + half + i] = s;
+        }
+    };
+    if (!ONE) angles();
     /* a part that does not fill its last four columns is followed by zero ones */
     float sq = 0.0f, sc = 0.0f;
     for (int c = tid * 4; c < nq + nc; c += threads * 4) {
@@ -111,20 +122,15 @@ __global__ void __launch_bounds__(kLpThreads, ONE ? 3 : 1) lm_latent_prepare_ker
     for (int e = tid; e < a.experts; e += threads) z[e] = sum1(a.col_router + e);
     for (int h = tid; h < a.heads; h += threads)
         a.gate[(size_t)m * a.heads + h] = 1.0f / (1.0f + expf(-sum1(a.col_g + h)));
-    for (int i = tid; i < half; i += threads) {
-        float c, s;
-        lm_angle(pos, a.freq[i], a.freq[half + i], a.mag, &c, &s);
-        cs[i] = c;
-        cs[half + i] = s;
-        a.cs[(size_t)m * a.rot + i] = c;
-        a.cs[(size_t)m * a.rot + half + i] = s;
-    }
+    if (ONE) angles();
     sq = vb_warp_sum(sq);
     sc = vb_warp_sum(sc);
     if (lane == 0) { red[0][warp] = sq; red[1][warp] = sc; }
     __syncthreads();
     sq = sc = 0.0f;
-    for (int w = 0; w < warps; w++) { sq += red[0][w]; sc += red[1][w]; }
+#pragma unroll
+    for (int w = 0; w < kLpWarps; w++)
+        if (w < warps) { sq += red[0][w]; sc += red[1][w]; }
     const float rq = 1.0f / sqrtf(sq / (float)a.q_rank + a.eps), rc = 1.0f / sqrtf(sc / (float)a.rank + a.eps);
     if ((a.q_rank & 3) == 0) {
         for (int c = tid * 4; c < a.q_rank; c += threads * 4) {

@@ -83,14 +83,14 @@ def test_mechanism(lm_mod, tmp_path, name):
                 lm.release(s)
 
 
-@pytest.mark.parametrize("width,vocab,eps", [(64, 50, 1e-3), (130, 333, 1e-6), (77, 31, 1e-5)])
-def test_stream_sizes(lm_mod, tmp_path, width, vocab, eps):
-    c = Case(lm_mod, tmp_path, config([latent(ff=0, window=9), latent(ff=50), latent(ff=20, experts=5)], width=width, vocab=vocab, eps=eps), seed=2)
-    toks = tokens(c.cfg, 70, 5)
+@pytest.mark.parametrize("width,vocab,eps,n", [(64, 50, 1e-3, 70), (130, 333, 1e-6, 70), (77, 31, 1e-5, 70), (400, 90, 1e-5, 300), (633, 70, 1e-4, 270)])
+def test_stream_sizes(lm_mod, tmp_path, width, vocab, eps, n):
+    c = Case(lm_mod, tmp_path, config([latent(ff=0, window=9), latent(ff=350), latent(ff=170, experts=5)], width=width, vocab=vocab, eps=eps), seed=2)
+    toks = tokens(c.cfg, n, 5)
     want = plain.forward(c.w, c.cfg, toks)[0]
     for dtype in DTYPES:
         with c.open(dtype) as lm:
-            for sizes in ([70], [30, 1, 3]):
+            for sizes in ([n], [30, 1, 3]):
                 s = lm.open()
                 assert error(feed(lm, s, toks, sizes), want) < LIMIT[dtype], (dtype, sizes)
                 lm.release(s)
